@@ -40,7 +40,7 @@ constexpr int RPT_MAX = 16;     // rows per thread in the value phase
 // Heads wider than 256 (one cached latent as key and value of many query heads): a CTA takes at most RWIDE query rows,
 // which is what its threads' value accumulators and its shared memory hold at those widths.
 constexpr int RWIDE = 32;
-constexpr int D_MAX = 512;
+constexpr int D_MAX = 640, DV_MAX = 512;
 __host__ __device__ __forceinline__ int q_rows_alloc(int d, int dv) { return d > 256 || dv > 256 ? RWIDE : RMAX; }
 
 template <typename T> struct Pad;            // padding of a key row in shared memory, in elements
@@ -70,6 +70,7 @@ attn_tile_kernel(const AttnParams p) {
     // key head and value head; with v_all the CTA applies its weights to all v_rep value heads in turn (VR of them)
     const int VR = p.v_all ? p.v_rep : 1;
     const int kvh = p.v_all ? blockIdx.y : blockIdx.y / p.v_rep;
+    const int kph = kvh / p.kv_div;              // the pool's head: several groups of query heads may share one
     const int vh = p.v_all ? 0 : (p.v_rep > 1 ? blockIdx.y - kvh * p.v_rep : kvh);
     const int tile = blockIdx.x / p.n_splits, split = blockIdx.x - tile * p.n_splits;
     const int slot = p.row_slot[b];
@@ -107,6 +108,10 @@ attn_tile_kernel(const AttnParams p) {
     float* l_s = alpha_s + RMAX;                                      // [RMAX]
     T* v_s = reinterpret_cast<T*>(l_s + RMAX);                        // [VR][KT][dv]
     T* k_s = v_s + VR * KT * dv;                                      // [KT][d + KPAD]
+    // values that are the keys' leading columns are read from the keys' rows
+    const bool v_in_k = p.v_ld != dv;
+    if (v_in_k) { k_s = v_s; }
+    const int vstride = v_in_k ? kstride : dv;
 
     __shared__ int row_s[KT];                    // per token of the tile: its row in the pools, -1 outside [lo, hi)
     __shared__ int vrow_s[KT];
@@ -138,7 +143,7 @@ attn_tile_kernel(const AttnParams p) {
 
     constexpr int EPC = 16 / sizeof(T);          // elements per 16-byte chunk
     const int cpr = d / EPC;                      // chunks per key row
-    const int cprv = dv / EPC;                    // chunks per value row
+    const int cprv = v_in_k ? 0 : dv / EPC;       // chunks per value row
     const int bs = p.block_size;
 
     for (int t0 = t_begin; t0 < hi; t0 += KT) {
@@ -156,8 +161,8 @@ attn_tile_kernel(const AttnParams p) {
                 const int blk = p.block_table[(size_t)slot * p.max_blocks + t / bs];
                 if (blk < 0 || blk >= p.num_blocks) set_status(p.status, STATUS_BAD_BLOCK);
                 else {
-                    base = (blk * p.n_kv + kvh) * bs + (t % bs);          // the token's row in the key pool
-                    vbase = (blk * p.n_kv + vh) * bs + (t % bs);          // and in the value pool
+                    base = (blk * p.n_kv_pool + kph) * bs + (t % bs);     // the token's row in the key pool
+                    vbase = (blk * p.n_kv_pool + (p.v_rep > 1 ? vh : kph)) * bs + (t % bs);   // and in the value pool
                 }
             }
             row_s[tid] = base;
@@ -177,7 +182,7 @@ attn_tile_kernel(const AttnParams p) {
                         const int tt = c / per_tok, cc = c - tt * per_tok;
                         const int base = row_s[tt];
                         if (base >= 0) {
-                            const int cv = cc - cpr, j = cv >= 0 ? cv / cprv : 0;       // value head j's row: j * bs rows on
+                            const int cv = cc - cpr, j = cv > 0 ? cv / cprv : 0;       // value head j's row: j * bs rows on
                             x4[u] = cc >= cpr ? *reinterpret_cast<const uint4*>(vp + ((size_t)vrow_s[tt] + (size_t)j * bs) * dv +
                                                                                 (cv - j * cprv) * EPC)
                                               : *reinterpret_cast<const uint4*>(kp + (size_t)base * d + cc * EPC);
@@ -282,7 +287,7 @@ attn_tile_kernel(const AttnParams p) {
             }
             for (int tt = 0; tt < KT; ++tt) {
                 float vf[4];
-                load_chunk4<T>(v_s + tt * dv + dc * 4, vf);
+                load_chunk4<T>(v_s + tt * vstride + dc * 4, vf);
 #pragma unroll
                 for (int i = 0; i < RPT_MAX; ++i) {
                     const int r = rg + i * RG;
@@ -411,10 +416,14 @@ __global__ void attn_combine_kernel(const float* __restrict__ part_m, const floa
 }
 
 template <typename T>
-static size_t attn_smem_bytes(int d, int dv, int vr = 1) {
+static size_t attn_smem_bytes(int d, int dv, int vr = 1, bool v_in_k = false) {
     return (size_t)(q_rows_alloc(d, dv) * d + RMAX * KT + 2 * RMAX) * sizeof(float) +
-           (size_t)(vr * KT * dv + KT * (d + Pad<T>::v)) * sizeof(T);
+           (size_t)((v_in_k ? 0 : vr * KT * dv) + KT * (d + Pad<T>::v)) * sizeof(T);
 }
+
+}  // namespace fd
+extern "C" int fd_attn_simt_qt(int G);
+namespace fd {
 
 template <typename T>
 static int launch_attn(const AttnParams& p0, int n_rows, int max_q_len, cudaStream_t stream) {
@@ -422,7 +431,18 @@ static int launch_attn(const AttnParams& p0, int n_rows, int max_q_len, cudaStre
     // few query rows and repeated value heads: one CTA per key head takes all value heads, if their tiles fit
     p.v_all = p.v_rep > 1 && p.QT * p.G * p.v_rep <= RMAX && p.d <= 256 && p.dv <= 256 &&
               attn_smem_bytes<T>(p.d, p.dv, p.v_rep) <= 160 * 1024;
-    const size_t smem = attn_smem_bytes<T>(p.d, p.dv, p.v_all ? p.v_rep : 1);
+    if (p.v_rep == 1) {             // a group larger than a CTA takes: several smaller ones on the same pool head
+        const int most = p.d > 256 || p.dv > 256 ? RWIDE : RMAX;
+        if (p.G > most) {
+            int g = most;
+            while (p.G % g) --g;
+            p.kv_div = p.G / g; p.n_kv *= p.kv_div; p.G = g;
+            p.QT = fd_attn_simt_qt(g);
+            if (p.QT > most / g) p.QT = most / g;
+            if (p.QT > max_q_len) p.QT = max_q_len;
+        }
+    }
+    const size_t smem = attn_smem_bytes<T>(p.d, p.dv, p.v_all ? p.v_rep : 1, p.v_ld != p.dv);
     auto k = attn_tile_kernel<T>;
     static size_t configured = 0;
     if (smem > configured) {
@@ -473,7 +493,7 @@ static int attention_impl(const void* q, const void* k_pool, const void* v_pool,
                           int n_splits, int split_len, float* scratch, int* counters, int* status, int use_mma,
                           cudaStream_t stream, const void* prefetch = nullptr, unsigned long long prefetch_bytes = 0,
                           float softcap = 0.f, int keep_first = 0, const float* sink = nullptr, int v_rep = 1,
-                          int out_f32 = 0, int ext_mma = 0) {
+                          int out_f32 = 0, int ext_mma = 0, int v_ld = 0) {
     if (n_rows == 0 || T == 0) return 0;
     FD_REQUIRE(softcap >= 0.f && keep_first >= 0 && v_rep >= 1 && (v_rep == 1 || v_rep == n_kv), -2,
                "attention: soft cap %g, %d kept first keys, weights applied to %d value heads of %d", softcap, keep_first,
@@ -482,14 +502,17 @@ static int attention_impl(const void* q, const void* k_pool, const void* v_pool,
     if (ext) use_mma = 0;
     // of the options the tensor-core decode kernel has the keyless term: a decode step that asks for nothing else runs there
     const bool sink_only = sink != nullptr && !(softcap > 0.f) && !(keep_first > 0 && window > 0) && v_rep == 1 && !out_f32;
+    if (v_ld <= 0) v_ld = dv;
+    FD_REQUIRE(v_ld == dv || (v_ld == d && dv <= d && k_pool == v_pool && v_rep == 1), -2,
+               "attention: value rows of %d in rows of %d", dv, v_ld);
+    if (v_ld != dv) { use_mma = 0; ext_mma = 0; }     // values inside the keys' rows: the CUDA-core kernel here
     const bool decode_mma = (use_mma != 0 || (sink_only && ext_mma != 0)) && dtype == 1 && max_q_len == 1 && dv == d;
     FD_REQUIRE(n_kv > 0 && n_q % n_kv == 0, -2, "attention: %d query heads are not a multiple of %d KV heads", n_q, n_kv);
     const int G = n_q / n_kv;
     FD_REQUIRE(d % 8 == 0 && d >= 8 && d <= D_MAX, -2, "attention: head size %d must be a multiple of 8 in [8, %d]", d, D_MAX);
-    FD_REQUIRE(dv % 8 == 0 && dv >= 8 && dv <= D_MAX, -2, "attention: value head size %d must be a multiple of 8 in [8, %d]", dv, D_MAX);
-    FD_REQUIRE((d <= 256 && dv <= 256) || G <= RWIDE, -2, "attention: heads wider than 256 take groups of up to %d query heads, got %d", RWIDE, G);
+    FD_REQUIRE(dv % 8 == 0 && dv >= 8 && dv <= DV_MAX, -2, "attention: value head size %d must be a multiple of 8 in [8, %d]", dv, DV_MAX);
+    FD_REQUIRE(v_rep == 1 || (d <= 256 && dv <= 256 && G <= RMAX) || G <= RWIDE, -2, "attention: repeated value heads take groups of up to %d query heads, got %d", RWIDE, G);
     FD_REQUIRE(chunk >= 0 && window >= 0, -2, "attention: chunk %d and window %d must not be negative", chunk, window);
-    FD_REQUIRE(G <= RMAX, -2, "attention: group size %d exceeds %d", G, RMAX);
     FD_REQUIRE(block_size > 0, -2, "attention: block size %d", block_size);
     FD_REQUIRE(n_splits >= 1 && n_splits <= COMBINE_MAX_SPLITS, -2, "attention: n_splits=%d (1..%d)", n_splits, COMBINE_MAX_SPLITS);
     FD_REQUIRE(n_splits == 1 || (split_len > 0 && split_len % KT == 0), -2,
@@ -513,12 +536,12 @@ static int attention_impl(const void* q, const void* k_pool, const void* v_pool,
     p.row_q_len = row_q_len; p.row_ctx_len = row_ctx_len; p.status = status;
     p.counters = nullptr;
     p.max_blocks = max_blocks; p.num_blocks = num_blocks; p.block_size = block_size;
-    p.n_q = n_q; p.n_kv = n_kv; p.G = G; p.d = d; p.dv = dv; p.chunk = chunk;
+    p.n_q = n_q; p.n_kv = n_kv; p.G = G; p.d = d; p.dv = dv; p.v_ld = v_ld; p.chunk = chunk;
     p.n_kv_pool = n_kv; p.kv_div = 1;
     p.softcap = softcap; p.keep_first = keep_first; p.sink = sink; p.v_rep = v_rep; p.out_f32 = out_f32; p.v_all = 0;
     if (dv != d) use_mma = 0;          // the tensor-core kernels keep keys and values of one size
-    int qt = fd_attn_simt_qt(G);
-    if ((d > 256 || dv > 256) && qt > RWIDE / G) qt = RWIDE / G;
+    int qt = G <= RMAX ? fd_attn_simt_qt(G) : 1;
+    if ((d > 256 || dv > 256) && qt > RWIDE / G) qt = RWIDE / G > 0 ? RWIDE / G : 1;
     if (qt > max_q_len) qt = max_q_len;
     p.QT = qt; p.n_splits = n_splits; p.split_len = split_len; p.window = window; p.scale = scale;
 
@@ -648,19 +671,20 @@ extern "C" int fd_attention_mma_sync(const void* q, const void* k_pool, const vo
 // v_rep == n_kv: every query head's weights are applied to all value heads and out is [T, n_q, n_kv, dv] (scratch for
 // the split form: fd_attn_scratch_floats(T, n_q * n_kv, dv, n_splits)); out_f32: out is float.  Decode steps in bfloat16
 // whose only option is the keyless term run on the tensor-core decode kernel when use_mma is set and it takes the sizes
-// (counters: as for fd_attention, the kernel then merges its own splits).
+// (counters: as for fd_attention, the kernel then merges its own splits).  v_ld: 0, or d when v_pool is k_pool and the
+// values are the first dv columns of the keys' rows.
 extern "C" int fd_attention_ext(const void* q, const void* k_pool, const void* v_pool, void* out, int dtype,
                                 const int* block_table, int max_blocks, int num_blocks, int block_size,
                                 const int* tok_row, const int* row_slot, const int* row_q_start,
                                 const int* row_q_len, const int* row_ctx_len, int n_rows, int T,
                                 int max_q_len, int n_q, int n_kv, int d, float scale, int window, int dv, int chunk,
                                 int n_splits, int split_len, float* scratch, int* status, float softcap, int keep_first,
-                                const float* sink, int v_rep, int out_f32, int use_mma, int* counters,
+                                const float* sink, int v_rep, int out_f32, int use_mma, int* counters, int v_ld,
                                 cudaStream_t stream) {
     return attention_impl(q, k_pool, v_pool, out, dtype, block_table, max_blocks, num_blocks, block_size, tok_row,
                           row_slot, row_q_start, row_q_len, row_ctx_len, n_rows, T, max_q_len, n_q, n_kv, d, scale,
                           window, dv, chunk, n_splits, split_len, scratch, counters, status, 0, stream, nullptr, 0,
-                          softcap, keep_first, sink, v_rep, out_f32, use_mma);
+                          softcap, keep_first, sink, v_rep, out_f32, use_mma, v_ld);
 }
 
 // o [T, n_q, n_kv, dv] float, mix [n_q, n_q] float; out (dtype 0 float32, 1 bfloat16): pointer to the first output

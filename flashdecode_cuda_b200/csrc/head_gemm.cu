@@ -2,6 +2,10 @@
 //
 //     out[t, h, n] = sum_k a[t, h, k] * w[h, n, k]        a [T, heads, K], w [heads, N, K], out [T, heads, N]
 //
+// The heads of a and of out may lie in longer places (strides a_hs, o_hs); out may be multiplied by sigmoid(gate[t, h, n]).
+// rope_heads turns a part of every head at the token's position (dimension 2i paired with 2i + 1), in place or into
+// another array: the rotated part of a latent attention's queries, which passes its per-head product by.
+//
 // (a per-head change of basis: a latent-attention mixer folds every head's key
 // expansion into its queries this way, and expands every head's attended latent
 // into values).  CUDA cores, float accumulation, k ascending in one fmaf chain
@@ -13,18 +17,25 @@ namespace fd {
 
 constexpr int HG_MT = 32, HG_NT = 64, HG_KT = 32, HG_THREADS = 256;
 
+// Where the heads lie: row and head strides of a, of out and of the gate (null: none), in elements.
+struct HeadStrides {
+    int a_ld, a_hs, o_ld, o_hs, g_ld, g_hs;
+};
+
+__device__ __forceinline__ float hg_sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
+
 template <typename T>
 __global__ void __launch_bounds__(HG_THREADS)
-head_gemm_kernel(const T* __restrict__ a, const T* __restrict__ w, T* __restrict__ out, int T_rows, int heads, int N,
-                 int K) {
+head_gemm_kernel(const T* __restrict__ a, const T* __restrict__ w, T* __restrict__ out, const T* __restrict__ gate,
+                 const HeadStrides st, int T_rows, int heads, int N, int K) {
     __shared__ float a_s[HG_MT][HG_KT + 1];
     __shared__ float b_s[HG_NT][HG_KT + 1];
     const int h = blockIdx.z;
     const int m0 = blockIdx.y * HG_MT, n0 = blockIdx.x * HG_NT;
     const int tid = threadIdx.x;
-    const T* ah = a + (size_t)h * K;                 // row stride heads * K
+    const T* ah = a + (size_t)h * st.a_hs;
     const T* wh = w + (size_t)h * N * K;
-    const size_t lda = (size_t)heads * K, ldo = (size_t)heads * N;
+    const size_t lda = st.a_ld, ldo = st.o_ld;
     const int ty = tid / 16, tx = tid % 16;          // rows 2 ty, 2 ty + 1; columns tx + 16 j
     float acc[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
     for (int k0 = 0; k0 < K; k0 += HG_KT) {
@@ -56,7 +67,10 @@ head_gemm_kernel(const T* __restrict__ a, const T* __restrict__ w, T* __restrict
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int c = n0 + tx + 16 * j;
-            if (c < N) out[(size_t)r * ldo + (size_t)h * N + c] = from_float<T>(acc[i][j]);
+            if (c >= N) continue;
+            float v = acc[i][j];
+            if (gate != nullptr) v *= hg_sigmoid(to_float(gate[(size_t)r * st.g_ld + (size_t)h * st.g_hs + c]));
+            out[(size_t)r * ldo + (size_t)h * st.o_hs + c] = from_float<T>(v);
         }
     }
 }
@@ -66,14 +80,15 @@ head_gemm_kernel(const T* __restrict__ a, const T* __restrict__ w, T* __restrict
 template <int MAXT>
 __global__ void __launch_bounds__(256)
 head_gemv_kernel(const __nv_bfloat16* __restrict__ a, const __nv_bfloat16* __restrict__ w, __nv_bfloat16* __restrict__ out,
-                 int T_rows, int heads, int N, int K) {
+                 const __nv_bfloat16* __restrict__ gate, const HeadStrides st, int T_rows, int heads, int N, int K) {
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int col = blockIdx.x * 8 + warp;
     if (col >= heads * N) return;
     const int h = col / N;
     const __nv_bfloat16* wr = w + (size_t)col * K;
-    const __nv_bfloat16* ah = a + (size_t)h * K;
-    const size_t lda = (size_t)heads * K;
+    const __nv_bfloat16* ah = a + (size_t)h * st.a_hs;
+    const size_t lda = st.a_ld;
+    const int n = col - h * N;
     float acc[MAXT];
 #pragma unroll
     for (int t = 0; t < MAXT; ++t) acc[t] = 0.f;
@@ -96,9 +111,41 @@ head_gemv_kernel(const __nv_bfloat16* __restrict__ a, const __nv_bfloat16* __res
 #pragma unroll
     for (int t = 0; t < MAXT; ++t) {
         if (t < T_rows) {
-            const float v = warp_sum(acc[t]);
-            if (lane == 0) out[(size_t)t * heads * N + col] = __float2bfloat16_rn(v);
+            float v = warp_sum(acc[t]);
+            if (lane == 0) {
+                if (gate != nullptr) v *= hg_sigmoid(__bfloat162float(gate[(size_t)t * st.g_ld + (size_t)h * st.g_hs + n]));
+                out[(size_t)t * st.o_ld + (size_t)h * st.o_hs + n] = __float2bfloat16_rn(v);
+            }
         }
+    }
+}
+
+// dst[t, h, 0 .. places) = rot(src[t, h, 0 .. nr)), zeros after it; src and dst may be the same memory (places == nr then).
+template <typename T>
+__global__ void rope_heads_kernel(const T* src, int s_ld, int s_hs, T* dst, int d_ld, int d_hs,
+                                  const float* __restrict__ cos_t, const float* __restrict__ sin_t, int table_len,
+                                  const int* __restrict__ tok_pos, int heads, int nr, int places, int* status) {
+    const int t = blockIdx.x;
+    const int pos = tok_pos[t];
+    if (pos < 0 || pos >= table_len) {
+        if (threadIdx.x == 0) set_status(status, STATUS_BAD_POSITION);
+        return;
+    }
+    const int half = nr >> 1, pp = places >> 1;
+    const float* c = cos_t + (size_t)pos * half;
+    const float* s = sin_t + (size_t)pos * half;
+    for (int e = threadIdx.x; e < heads * pp; e += blockDim.x) {
+        const int h = e / pp, i = e - h * pp;
+        T a = from_float<T>(0.f), b = a;
+        if (i < half) {
+            const T* x = src + (size_t)t * s_ld + (size_t)h * s_hs + 2 * i;
+            const float u = to_float(x[0]), v = to_float(x[1]);
+            a = from_float<T>(u * c[i] - v * s[i]);
+            b = from_float<T>(v * c[i] + u * s[i]);
+        }
+        T* o = dst + (size_t)t * d_ld + (size_t)h * d_hs + 2 * i;
+        o[0] = a;
+        o[1] = b;
     }
 }
 
@@ -106,23 +153,43 @@ head_gemv_kernel(const __nv_bfloat16* __restrict__ a, const __nv_bfloat16* __res
 
 using namespace fd;
 
-extern "C" int fd_head_gemm(const void* a, const void* w, void* out, int dtype, int T, int heads, int N, int K,
-                            cudaStream_t stream) {
+// a: [T, heads, K] with row stride a_ld and head stride a_hs (elements); out likewise; gate (or null): sigmoid(gate) times out.
+extern "C" int fd_head_gemm(const void* a, int a_ld, int a_hs, const void* w, void* out, int o_ld, int o_hs, const void* gate,
+                            int g_ld, int g_hs, int dtype, int T, int heads, int N, int K, cudaStream_t stream) {
     if (T == 0) return 0;
     FD_REQUIRE(heads > 0 && heads <= 65535 && N > 0 && K > 0, -2, "head_gemm: %d heads, N %d, K %d", heads, N, K);
-    if (dtype == 1 && T <= 16 && K % 8 == 0 && (uintptr_t)a % 16 == 0 && (uintptr_t)w % 16 == 0) {
+    const HeadStrides st = {a_ld, a_hs, o_ld, o_hs, g_ld, g_hs};
+    if (dtype == 1 && T <= 16 && K % 8 == 0 && a_ld % 8 == 0 && a_hs % 8 == 0 && (uintptr_t)a % 16 == 0 && (uintptr_t)w % 16 == 0) {
         const dim3 g((unsigned)((heads * (long long)N + 7) / 8));
         if (T <= 8)
             return launch("head_gemm", head_gemv_kernel<8>, g, dim3(256), 0, stream, dim3(1, 1, 1), (const __nv_bfloat16*)a,
-                          (const __nv_bfloat16*)w, (__nv_bfloat16*)out, T, heads, N, K);
+                          (const __nv_bfloat16*)w, (__nv_bfloat16*)out, (const __nv_bfloat16*)gate, st, T, heads, N, K);
         return launch("head_gemm", head_gemv_kernel<16>, g, dim3(256), 0, stream, dim3(1, 1, 1), (const __nv_bfloat16*)a,
-                      (const __nv_bfloat16*)w, (__nv_bfloat16*)out, T, heads, N, K);
+                      (const __nv_bfloat16*)w, (__nv_bfloat16*)out, (const __nv_bfloat16*)gate, st, T, heads, N, K);
     }
     dim3 grid((N + HG_NT - 1) / HG_NT, (T + HG_MT - 1) / HG_MT, heads);
     FD_REQUIRE(grid.y <= 65535, -2, "head_gemm: %d rows are too many", T);
     if (dtype == 0)
-        return launch("head_gemm", head_gemm_kernel<float>, grid, dim3(HG_THREADS), 0, stream, dim3(1, 1, 1),
-                      (const float*)a, (const float*)w, (float*)out, T, heads, N, K);
+        return launch("head_gemm", head_gemm_kernel<float>, grid, dim3(HG_THREADS), 0, stream, dim3(1, 1, 1), (const float*)a,
+                      (const float*)w, (float*)out, (const float*)gate, st, T, heads, N, K);
     return launch("head_gemm", head_gemm_kernel<__nv_bfloat16>, grid, dim3(HG_THREADS), 0, stream, dim3(1, 1, 1),
-                  (const __nv_bfloat16*)a, (const __nv_bfloat16*)w, (__nv_bfloat16*)out, T, heads, N, K);
+                  (const __nv_bfloat16*)a, (const __nv_bfloat16*)w, (__nv_bfloat16*)out, (const __nv_bfloat16*)gate, st, T, heads,
+                  N, K);
+}
+
+// src / dst: pointers to the first rotated dimension of the first head; cos_t / sin_t [table_len, nr / 2].
+extern "C" int fd_rope_heads(const void* src, int s_ld, int s_hs, void* dst, int d_ld, int d_hs, int dtype, const float* cos_t,
+                             const float* sin_t, int table_len, const int* tok_pos, int T, int heads, int nr, int places,
+                             int* status, cudaStream_t stream) {
+    if (T == 0 || nr == 0) return 0;
+    FD_REQUIRE(heads > 0 && nr > 0 && nr % 2 == 0 && places >= nr && places % 2 == 0, -2, "rope_heads: %d of %d dimensions", nr, places);
+    FD_REQUIRE(src != dst || places == nr, -2, "rope_heads: in place there is nothing to fill up");
+    const int work = heads * places / 2;
+    const dim3 block(work >= 256 ? 256 : (work + 31) / 32 * 32);
+    if (dtype == 0)
+        return launch("rope_heads", rope_heads_kernel<float>, dim3(T), block, 0, stream, dim3(1, 1, 1), (const float*)src, s_ld,
+                      s_hs, (float*)dst, d_ld, d_hs, cos_t, sin_t, table_len, tok_pos, heads, nr, places, status);
+    return launch("rope_heads", rope_heads_kernel<__nv_bfloat16>, dim3(T), block, 0, stream, dim3(1, 1, 1),
+                  (const __nv_bfloat16*)src, s_ld, s_hs, (__nv_bfloat16*)dst, d_ld, d_hs, cos_t, sin_t, table_len, tok_pos,
+                  heads, nr, places, status);
 }

@@ -3,7 +3,8 @@
 //   S_t = diag(a_t) S_(t-1) + b_t v_t^T,      o_t = S_t^T q_t          S [d, dv] per sequence and head
 //
 //  * mode 0 (constant decay): a_t = decay[h] for every channel, b_t = rot(k_t) * k_scale, q_t = rot(q_t); rot turns
-//    the first `rot` dimensions of a head at the token's position, dimension i paired with i + rot/2.
+//    the first `rot` dimensions of a head at the token's position, dimension i paired with i + rot/2.  With `silu` set (and
+//    rot 0) q, k and v pass silu on their way in.
 //  * mode 1 (forget gate): a_t = f_t = lower + (1 - lower) * sigmoid(z_t) per channel, b_t = 1 - f_t,
 //    q_t = silu(zq_t); z and zq are columns of the projection.
 //  * mode 2 (decay per key channel): a_t = sigmoid(z_t)^(1/tau) per channel with z a float array of its own (the output
@@ -32,6 +33,7 @@
 //
 //  * low_rank_expand: a narrow vector per token times a matrix [N, R] plus a bias, as floats (the pre-activation of a
 //    decay that comes through a narrow projection);
+//  * row_norm_gate: one norm over a token's heads side by side, times a weight per channel, times sigmoid(gate).
 //  * head_norm_gate: y = o / sqrt(mean(o^2) + eps) per token and head (over dv), times an optional weight [dv], times
 //    an optional silu(gate) read from a column range of a packed projection, times a constant; written with a row
 //    stride and a column offset of its own so that several mixers can fill one buffer.
@@ -55,6 +57,7 @@ struct ScanParams {
     float q_scale, inv_tau;            // (mode 2)
     const float* cos_t; const float* sin_t; int table_len, rot;
     float k_scale;
+    int silu;                          // (mode 0) q, k and v pass silu
     const int* row_slot; const int* row_q_start; const int* row_q_len; const int* row_ctx_len;
     int H, d, dv, mode, write_state, DS, TC;
     int* status;
@@ -64,6 +67,8 @@ struct ScanParams {
     float* seg_state; float* seg_decay;
     float* prep; float* prep_v; int dvp;      // the preparing kernel's q, b (and a) [T, H, NA * CS] and v [T, H, dvp]
 };
+
+__device__ __forceinline__ float scan_silu(float z) { return z / (1.f + expf(-z)); }
 
 // Segment s of step row r has the slot q_start / seg_len + r + s: slots of different rows never meet, and a step of T
 // tokens and n rows needs at most T / seg_len + n + 1 of them.
@@ -124,6 +129,9 @@ __device__ __forceinline__ void stage_tokens(const ScanParams& p, int h, int tok
             if (i >= d) {
                 at[0] = 0.f; at[CS] = 0.f;
                 if (p.mode != 0) at[2 * CS] = 0.f;
+            } else if (p.mode == 0 && p.silu) {
+                at[0] = scan_silu(xq[u]);
+                at[CS] = scan_silu(xk[u]) * p.k_scale;
             } else if (p.mode == 0) {
                 at[0] = xq[u] * cc[u] + yq[u] * ss[u];              // first half: x c - y s; second half: x c + y s
                 at[CS] = (xk[u] * cc[u] + yk[u] * ss[u]) * p.k_scale;
@@ -169,7 +177,8 @@ scan_prepare_kernel(const ScanParams p) {
     for (int idx = threadIdx.x; idx < n * p.dvp; idx += PREP_THREADS) {
         const int tt = idx / p.dvp, c = idx - tt * p.dvp;
         const size_t tok = q_start + t0 + tt;
-        p.prep_v[(tok * p.H + h) * p.dvp + c] = c < p.dv ? to_float(proj[tok * p.ld + p.v_col + h * p.dv + c]) : 0.f;
+        const float v = c < p.dv ? to_float(proj[tok * p.ld + p.v_col + h * p.dv + c]) : 0.f;
+        p.prep_v[(tok * p.H + h) * p.dvp + c] = p.silu ? scan_silu(v) : v;
     }
 }
 
@@ -249,7 +258,8 @@ linear_scan_kernel(const ScanParams p) {
             for (int idx = tid; idx < n * VT; idx += SCAN_THREADS) {
                 const int tt = idx / VT, c = idx - tt * VT;
                 const int vc = tile * VT + c;
-                sm[TC * TS + idx] = vc < dv ? to_float(proj[(size_t)(q_start + c0 + tt) * p.ld + p.v_col + h * dv + vc]) : 0.f;
+                const float v = vc < dv ? to_float(proj[(size_t)(q_start + c0 + tt) * p.ld + p.v_col + h * dv + vc]) : 0.f;
+                sm[TC * TS + idx] = p.silu ? scan_silu(v) : v;
             }
             __syncthreads();
         } else {
@@ -388,6 +398,24 @@ __global__ void head_norm_gate_kernel(const float* __restrict__ o, const float* 
 }
 
 
+// A CTA per token: y = o / sqrt(mean(o^2) + eps) * w over ALL n values of the row, times sigmoid(gate).
+constexpr int ROW_GATE_THREADS = 256;
+template <typename T>
+__global__ void __launch_bounds__(ROW_GATE_THREADS)
+row_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ w, const T* __restrict__ gate, int ldg,
+                     T* __restrict__ out, int n, float eps) {
+    __shared__ float red[33];
+    const size_t t = blockIdx.x;
+    const float* x = o + t * n;
+    float ss = 0.f;
+    for (int j = threadIdx.x; j < n; j += blockDim.x) ss = fmaf(x[j], x[j], ss);
+    const float rs = 1.f / sqrtf(block_sum(ss, red) / (float)n + eps);
+    for (int j = threadIdx.x; j < n; j += blockDim.x) {
+        const float z = to_float(gate[t * ldg + j]);
+        out[t * n + j] = from_float<T>(x[j] * rs * w[j] / (1.f + expf(-z)));
+    }
+}
+
 // out[t, c] = bias[c] + sum_r w[c, r] * x[t, x_col + r]: a narrow vector per token (R <= EXPAND_MAX_R columns of a wider
 // matrix) expanded to N channels, float sums in the order r = 0, 1, ... from the bias on, whatever else the step holds.
 // A CTA of two warps takes 64 channels and up to EXPAND_TOK tokens, so that a decode step still spreads over dozens of
@@ -514,6 +542,7 @@ extern "C" long long fd_linear_scan_scratch_floats(int T, int n_rows, int H, int
 // at k_col - H * d columns each - and v at v_col (H * dv columns).  state [slots, H, d, dv] and out [T, H * dv] float.
 // mode 0: decay [H], cos_t / sin_t [table_len, rot / 2] (unused when rot == 0), k_scale.  mode 1: lower [H * d].
 // mode 2: gate [T, gate_ld] float (the decay's pre-activation, H * d columns from the pointer on), q_scale, inv_tau.
+// silu (mode 0, rot 0): q, k and v pass silu.
 // max_q_len: the longest portion of the step; with scratch memory (fd_linear_scan_scratch_floats floats for the step's T
 // tokens) portions longer than two segments run in segments side by side, otherwise each in one CTA per head and tile.
 extern "C" int fd_linear_scan(const void* proj, int ld, int dtype, int q_col, int k_col, int v_col, float* state,
@@ -521,7 +550,7 @@ extern "C" int fd_linear_scan(const void* proj, int ld, int dtype, int q_col, in
                               const float* sin_t, int table_len, int rot, float k_scale, const int* row_slot,
                               const int* row_q_start, const int* row_q_len, const int* row_ctx_len, int n_rows, int H,
                               int d, int dv, int write_state, int* status, int T, int max_q_len, float* scratch,
-                              long long scratch_floats, const float* gate, int gate_ld, float q_scale, float inv_tau,
+                              long long scratch_floats, const float* gate, int gate_ld, float q_scale, float inv_tau, int silu,
                               cudaStream_t stream) {
     if (n_rows == 0) return 0;
     FD_REQUIRE(H > 0 && d > 0 && dv > 0 && d <= 256, -2, "linear_scan: %d heads of %d x %d (d at most 256)", H, d, dv);
@@ -535,6 +564,8 @@ extern "C" int fd_linear_scan(const void* proj, int ld, int dtype, int q_col, in
     p.proj = proj; p.ld = ld; p.q_col = q_col; p.k_col = k_col; p.v_col = v_col; p.state = state; p.out = out;
     p.decay = decay; p.lower = lower; p.cos_t = cos_t; p.sin_t = sin_t; p.table_len = table_len;
     p.rot = mode == 0 ? rot : 0; p.k_scale = k_scale;
+    p.silu = mode == 0 && silu;
+    FD_REQUIRE(!p.silu || p.rot == 0, -2, "linear_scan: silu on q, k and v goes without a rotation");
     p.gate = gate; p.gate_ld = gate_ld; p.q_scale = q_scale; p.inv_tau = inv_tau;
     p.row_slot = row_slot; p.row_q_start = row_q_start; p.row_q_len = row_q_len; p.row_ctx_len = row_ctx_len;
     p.H = H; p.d = d; p.dv = dv; p.mode = mode; p.write_state = write_state; p.status = status;
@@ -572,6 +603,20 @@ extern "C" int fd_head_norm_gate(const float* o, const float* w, const void* gat
                       (const float*)gate, ldg, (float*)out, ld_out, (int)pairs, H, dv, eps, scale);
     return launch("head_norm_gate", head_norm_gate_kernel<bf16>, grid, dim3(128), 0, stream, dim3(1, 1, 1), o, w,
                   (const bf16*)gate, ldg, (bf16*)out, ld_out, (int)pairs, H, dv, eps, scale);
+}
+
+// o [T, n] float; w [n] float; gate: pointer to the first gate column of a packed projection with row stride ldg (dtype as
+// out); out [T, n].
+extern "C" int fd_row_norm_gate(const float* o, const float* w, const void* gate, int ldg, void* out, int dtype, int T, int n,
+                                float eps, cudaStream_t stream) {
+    if (T == 0) return 0;
+    FD_REQUIRE(n > 0, -2, "row_norm_gate: rows of %d", n);
+    const dim3 block(n >= 1024 ? ROW_GATE_THREADS : 128);
+    if (dtype == 0)
+        return launch("row_norm_gate", row_norm_gate_kernel<float>, dim3(T), block, 0, stream, dim3(1, 1, 1), o, w,
+                      (const float*)gate, ldg, (float*)out, n, eps);
+    return launch("row_norm_gate", row_norm_gate_kernel<bf16>, dim3(T), block, 0, stream, dim3(1, 1, 1), o, w,
+                  (const bf16*)gate, ldg, (bf16*)out, n, eps);
 }
 
 // x: pointer to the first of the R columns of a matrix [T, ldx] of `dtype` (0 float32, 1 bfloat16); w [N, R] of the same

@@ -267,7 +267,8 @@ class Model:
                 li = groups[gi]["n_layers"]
                 groups[gi]["n_layers"] += 1
             st = {}
-            for s in (mixer.state_requests() if mixer is not None else []):
+            extra = getattr(self.blocks[run.layer], "extra_state_requests", list)()
+            for s in (mixer.state_requests() if mixer is not None else []) + extra:
                 key = f"run{i}.{s.name}"
                 states.append(StateSpec(key, tuple(s.shape), s.dtype))
                 st[s.name] = key

@@ -97,13 +97,14 @@ def _declare(L: ctypes.CDLL) -> None:
         "fd_attention": [P, P, P, P, I, P, I, I, I, P, P, P, P, P, I, I, I, I, I, I, F, I, I, I, I, I, P, P, P, P, c_ulonglong, P],
         "fd_attention_mma_sync": [P, P, P, P, I, P, I, I, I, P, P, P, P, P, I, I, I, I, I, I, F, I, I, I, I, I, P, P, P, P],
         "fd_conv_rope_append": [P, I, I, P, P, P, P, P, I, I, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, P, I, P, P, F, I, I, P],
-        "fd_attention_ext": [P, P, P, P, I, P, I, I, I, P, P, P, P, P, I, I, I, I, I, I, F, I, I, I, I, I, P, P, F, I, P, I, I, I, P, P],
+        "fd_attention_ext": [P, P, P, P, I, P, I, I, I, P, P, P, P, P, I, I, I, I, I, I, F, I, I, I, I, I, P, P, F, I, P, I, I, I, P, I, P],
         "fd_attn_head_mix": [P, P, P, I, I, I, I, I, I, F, P],
         "fd_add_dyn_tanh": [P, I, P, I, P, P, F, P, I, P, I, I, P],
         "fd_quad_exp_act": [P, P, I, P, LL, P],
         "fd_scale_f32": [P, LL, F, P],
         "fd_axpy_f32": [P, P, I, LL, F, I, P],
-        "fd_linear_scan": [P, I, I, I, I, I, P, P, I, P, P, P, P, I, I, F, P, P, P, P, I, I, I, I, I, P, I, I, P, LL, P, I, F, F, P],
+        "fd_linear_scan": [P, I, I, I, I, I, P, P, I, P, P, P, P, I, I, F, P, P, P, P, I, I, I, I, I, P, I, I, P, LL, P, I, F, F, I, P],
+        "fd_row_norm_gate": [P, P, P, I, P, I, I, I, F, P],
         "fd_head_norm_gate": [P, P, P, I, P, I, I, I, I, I, F, F, P],
         "fd_low_rank_expand": [P, I, P, P, P, I, I, I, I, P],
         "fd_conv_state_update": [P, I, I, P, P, P, P, I, I, I, P],
@@ -117,8 +118,11 @@ def _declare(L: ctypes.CDLL) -> None:
         "fd_lanes_norm": [P, I, I, LL, P, P, P, P, I, P, P, F, P, I, P, I, I, I, P],
         "fd_lanes_fill": [P, P, I, I, I, P],
         "fd_lanes_sum": [P, I, P, P, P, P, P, I, I, I, P],
-        "fd_norm_append": [P, I, P, I, P, P, F, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, P, I, I, P, P],
-        "fd_head_gemm": [P, P, P, I, I, I, I, I, P],
+        "fd_norm_append": [P, I, P, I, P, P, F, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, P, I, I, P, P, I, I, I, P, I, P, P],
+        "fd_head_gemm": [P, I, I, P, P, I, I, P, I, I, I, I, I, I, I, P],
+        "fd_rope_heads": [P, I, I, P, I, I, I, P, P, I, P, I, I, I, I, P, P],
+        "fd_post_norm": [P, I, P, P, I, P, I, F, P, I, P, LL, I, I, P, P, I, P, I, F, P, P, I, P, P, P, I, I, P],
+        "fd_stream_conv": [P, P, P, P, I, P, P, P, I, I, I, P],
         "fd_moe_align": [P, I, I, P, P, P, P, I, I, P],
         "fd_moe_gemm": [P, P, P, I, I, P, P, P, I, I, I, I, I, F, I, P],
         "fd_add_cast": [P, I, P, P, I, I, I, F, P],
@@ -329,18 +333,24 @@ def norm_append(proj: torch.Tensor, q_out: Optional[torch.Tensor], q_weight: Opt
                 k_weight: Optional[torch.Tensor], eps: float, tok_row: torch.Tensor, tok_pos: torch.Tensor,
                 row_slot: torch.Tensor, k_pool: torch.Tensor, v_pool: Optional[torch.Tensor], block_table: torch.Tensor,
                 n_kv: int, write_kv: bool, status: torch.Tensor, k_rows: Optional[torch.Tensor] = None,
-                q_count: int = 0, k_count: int = 0) -> None:
+                q_count: int = 0, k_count: int = 0, cos: Optional[torch.Tensor] = None, sin: Optional[torch.Tensor] = None,
+                rot: int = 0, rot_places: int = 0, r_rows: Optional[torch.Tensor] = None) -> None:
     """``proj`` [T, >= nq + nk + nv] = [q | k | v]: q (normed over all its nq columns with ``q_weight``, or as it is) to
     ``q_out`` [T, nq]; k (normed over all its nk columns with ``k_weight``, or as it is) and v to the pools at each
     token's position.  ``v_pool`` None: nothing but the keys is kept.  ``q_out`` None: the rows hold no q.  ``k_rows``
     [T, nk]: receives the (normed) k once more as plain rows.  ``q_count`` / ``k_count``: how many of q's and k's
     columns are real where heads are zero-padded to multiples of 8 (the norms' means run over these; 0: all).  Norm
-    weights float32."""
+    weights float32.  ``rot`` > 0 (one key head, keys only): the ``rot`` columns after k are one rotated part per position
+    (pairs 2i, 2i + 1; ``cos`` / ``sin`` [positions, rot / 2]), which follows k in the pool's rows in ``rot_places`` places
+    (zeros behind it) and goes to ``r_rows`` [T, >= rot] once more."""
     T, ld = proj.shape
     nq = 0 if q_out is None else q_out.shape[1]
     num_blocks, kvh, block_size, d = k_pool.shape
+    d -= rot_places
     nk = n_kv * d
     nv = 0 if v_pool is None else n_kv * v_pool.shape[-1]
+    assert rot == 0 or (cos.dtype == sin.dtype == torch.float32 and cos.shape == sin.shape and cos.shape[1] == rot // 2)
+    assert r_rows is None or (r_rows.shape[0] == T and r_rows.dtype == proj.dtype)
     assert kvh == n_kv and proj.dtype == k_pool.dtype and proj.is_contiguous() and (q_out is None or q_out.dtype == proj.dtype)
     assert k_rows is None or (k_rows.shape == (T, nk) and k_rows.dtype == proj.dtype and k_rows.is_contiguous())
     assert q_weight is None or (q_weight.dtype == torch.float32 and q_weight.numel() == nq)
@@ -348,24 +358,104 @@ def norm_append(proj: torch.Tensor, q_out: Optional[torch.Tensor], q_weight: Opt
     _check(lib().fd_norm_append(_ptr(proj), ld, _ptr(q_out), _dt(proj.dtype), _ptr(q_weight), _ptr(k_weight), float(eps),
                                 _ptr(tok_row), _ptr(tok_pos), _ptr(row_slot), _ptr(k_pool), _ptr(v_pool),
                                 _ptr(block_table), block_table.shape[1], num_blocks, block_size, T, nq, nk, nv, n_kv,
-                                int(write_kv), _ptr(k_rows), int(q_count), int(k_count), _ptr(status), _stream()))
+                                int(write_kv), _ptr(k_rows), int(q_count), int(k_count), _ptr(cos), _ptr(sin),
+                                cos.shape[0] if rot else 0, int(rot), int(rot_places), _ptr(r_rows),
+                                r_rows.shape[1] if r_rows is not None else 0, _ptr(status), _stream()))
 
 
 HEAD_GEMM_LIBRARY_ROWS = 64      # from this many rows on, the per-head products of bfloat16 steps go to the library's batched product
 
 
-def head_gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
-    """out[t, h, :] = w[h] a[t, h, :]: a [T, heads * K], w [heads, N, K], out [T, heads * N]; float accumulation.
-    float32: the library's own CUDA-core kernel with k ascending (no bit of a row depends on the step's other rows);
-    bfloat16: a warp per output column for steps of up to 16 rows, cuBLAS's strided batched product for prompts."""
+def head_gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, a_size: int = 0, out_size: int = 0,
+              gate: Optional[torch.Tensor] = None, gate_col: int = 0) -> None:
+    """out[t, h, :N] = w[h] a[t, h, :K]: a [T, heads * a_size], w [heads, N, K], out [T, heads * out_size]; ``a_size`` /
+    ``out_size``: the places a head has there (0: K and N; the places behind are neither read nor written).  ``gate``: out is
+    multiplied by sigmoid of its columns ``gate_col + h * N + n``.  Float accumulation.  float32: the library's own CUDA-core
+    kernel with k ascending (no bit of a row depends on the step's other rows); bfloat16: a warp per output column for
+    steps of up to 16 rows, cuBLAS's strided batched product for prompts (without a gate)."""
     heads, N, Kd = w.shape
     T = a.shape[0]
-    assert a.shape == (T, heads * Kd) and out.shape == (T, heads * N) and a.dtype == w.dtype == out.dtype
+    a_size, out_size = a_size or Kd, out_size or N
+    assert a.shape == (T, heads * a_size) and out.shape == (T, heads * out_size) and a.dtype == w.dtype == out.dtype
+    assert a_size >= Kd and out_size >= N
     assert a.is_contiguous() and w.is_contiguous() and out.is_contiguous()
-    if a.dtype == torch.bfloat16 and T >= HEAD_GEMM_LIBRARY_ROWS:
-        torch.bmm(a.view(T, heads, Kd).transpose(0, 1), w.transpose(1, 2), out=out.view(T, heads, N).transpose(0, 1))
+    assert gate is None or (gate.shape[0] == T and gate.dtype == a.dtype and gate_col + heads * N <= gate.shape[1])
+    if a.dtype == torch.bfloat16 and T >= HEAD_GEMM_LIBRARY_ROWS and gate is None:
+        torch.bmm(a.view(T, heads, a_size)[:, :, :Kd].transpose(0, 1), w.transpose(1, 2),
+                  out=out.view(T, heads, out_size)[:, :, :N].transpose(0, 1))
         return
-    _check(lib().fd_head_gemm(_ptr(a), _ptr(w), _ptr(out), _dt(a.dtype), T, heads, N, Kd, _stream()))
+    _check(lib().fd_head_gemm(_ptr(a), heads * a_size, a_size, _ptr(w), _ptr(out), heads * out_size, out_size,
+                              _col_ptr(gate, gate_col) if gate is not None else None, gate.shape[1] if gate is not None else 0,
+                              N, _dt(a.dtype), T, heads, N, Kd, _stream()))
+
+
+def rope_heads(src: torch.Tensor, src_size: int, src_off: int, dst: torch.Tensor, dst_size: int, dst_off: int,
+               cos: torch.Tensor, sin: torch.Tensor, tok_pos: torch.Tensor, n_heads: int, rot: int, places: int,
+               status: torch.Tensor) -> None:
+    """The ``rot`` dimensions from ``src_off`` on of every head of ``src`` [T, heads * src_size], turned at each token's
+    position (pairs 2i, 2i + 1), to the ``places`` from ``dst_off`` on of every head of ``dst`` (zeros behind them); src
+    and dst may be the same array."""
+    T = src.shape[0]
+    assert src.shape == (T, n_heads * src_size) and dst.shape == (T, n_heads * dst_size) and src.dtype == dst.dtype
+    assert src_off + rot <= src_size and dst_off + places <= dst_size and cos.shape[1] == rot // 2
+    _check(lib().fd_rope_heads(_col_ptr(src, src_off), n_heads * src_size, src_size, _col_ptr(dst, dst_off),
+                               n_heads * dst_size, dst_size, _dt(src.dtype), _ptr(cos), _ptr(sin), cos.shape[0],
+                               _ptr(tok_pos), T, n_heads, rot, places, _ptr(status), _stream()))
+
+
+def post_norm(y, weight: Optional[torch.Tensor], groups: int, eps: float, resid: torch.Tensor, out: Optional[torch.Tensor],
+              rows: Optional[torch.Tensor] = None, n_out: Optional[int] = None, write_resid: bool = True,
+              history: Optional[torch.Tensor] = None, n_history: int = 0, put_history: int = -1,
+              depth_weights: Optional[torch.Tensor] = None, out_weight: Optional[torch.Tensor] = None, out_groups: int = 1,
+              out_eps: float = 0.0, conv_weight: Optional[torch.Tensor] = None, conv_state: Optional[torch.Tensor] = None,
+              tok_row: Optional[torch.Tensor] = None, row_slot: Optional[torch.Tensor] = None) -> None:
+    """Completes a float32 stream ``resid`` [T, H] whose sub-layers' norms sit on their outputs, and makes the next input:
+
+        x = resid[r] + norm(y[r])                                  norm: ``groups`` RMS norms side by side, times weight
+        history[put_history][r] = x                                (optional)
+        x = sum_j depth_weights[j] history[j][r] + depth_weights[n_history] x          (optional, j < n_history)
+        resid[r] = x                                               (``write_resid``)
+        out[j] = x, or norm(x) with ``out_weight``, or x + conv(x) with ``conv_weight`` [taps, H] (single-token steps;
+                 ``conv_state`` [slots, taps - 1, H] is moved on)
+
+    for row j (or rows[j]).  ``y``: [T, H], or the unsummed rows of a routed feed-forward (an object with ``y``, ``wts``,
+    ``pair_pos``), or None (nothing pending).  Everything is float32 until the store to ``out``."""
+    T, H = resid.shape
+    wts = pair_pos = None
+    top = 0
+    if y is not None and not isinstance(y, torch.Tensor):
+        y, wts, pair_pos = y.y, y.wts, y.pair_pos
+        top = wts.shape[1]
+        assert wts.dtype == torch.float32 and wts.shape[0] == T and pair_pos.dtype == torch.int32 and pair_pos.numel() == T * top
+    elif y is not None:
+        assert y.shape == (T, H)
+    assert resid.dtype == torch.float32 and (y is None or (y.shape[-1] == H and weight.numel() == H))
+    for t in (weight, depth_weights, out_weight, history, conv_weight, conv_state):
+        assert t is None or t.dtype == torch.float32
+    assert history is None or (history.shape[1:] == (T, H) and n_history <= history.shape[0] and put_history < history.shape[0])
+    assert depth_weights is None or depth_weights.numel() == n_history + 1
+    assert conv_weight is None or (conv_weight.shape[1] == H and (conv_state is None or conv_state.shape[1:] == (conv_weight.shape[0] - 1, H)))
+    if n_out is None:
+        n_out = rows.numel() if rows is not None else T
+    assert out is None or (out.shape[-1] == H and out.numel() >= n_out * H)
+    _check(lib().fd_post_norm(_ptr(y), _dt(y.dtype) if y is not None else 0, _ptr(wts), _ptr(pair_pos), top, _ptr(weight),
+                              int(groups), float(eps), _ptr(resid), int(write_resid), _ptr(history), T * H, int(n_history),
+                              int(put_history), _ptr(depth_weights), _ptr(out), _dt(out.dtype) if out is not None else 0,
+                              _ptr(out_weight), int(out_groups), float(out_eps), _ptr(conv_weight), _ptr(conv_state),
+                              conv_weight.shape[0] if conv_weight is not None else 0, _ptr(tok_row), _ptr(row_slot),
+                              _ptr(rows), n_out, H, _stream()))
+
+
+def stream_conv(x: torch.Tensor, weight: torch.Tensor, state: Optional[torch.Tensor], out: torch.Tensor,
+                tok_row: torch.Tensor, row_slot: torch.Tensor, row_q_start: torch.Tensor) -> None:
+    """out[t] = x[t] + sum_k weight[k] * x[t - taps + 1 + k] per channel: x float32 [T, H], weight float32 [taps, H];
+    inputs before a row's first token of the step come from ``state`` [slots, taps - 1, H] (float32)."""
+    T, H = x.shape
+    taps = weight.shape[0]
+    assert x.dtype == weight.dtype == torch.float32 and out.shape == (T, H) and weight.shape[1] == H
+    assert taps == 1 or (state.dtype == torch.float32 and state.shape[1:] == (taps - 1, H))
+    _check(lib().fd_stream_conv(_ptr(x), _ptr(weight), _ptr(state), _ptr(out), _dt(out.dtype), _ptr(tok_row), _ptr(row_slot),
+                                _ptr(row_q_start), T, H, taps, _stream()))
 
 
 def rope_append(qkv: torch.Tensor, q_out: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor,
@@ -701,7 +791,7 @@ def attention_ext(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, o
                   window: int = 0, n_splits: int = 1, split_len: int = 0,
                   scratch: Optional[torch.Tensor] = None, status: Optional[torch.Tensor] = None, chunk: int = 0,
                   softcap: float = 0.0, keep_first: int = 0, sink: Optional[torch.Tensor] = None,
-                  all_value_heads: bool = False, tensor_cores: bool = True) -> None:
+                  all_value_heads: bool = False, tensor_cores: bool = True, value_dim: int = 0) -> None:
     """Attention with more options, on the CUDA cores; prompt steps in bfloat16 whose key and value heads both have 64
     or 128 dimensions run on the tensor cores unless ``tensor_cores`` is False, and so do decode steps in bfloat16 whose
     only option is ``sink`` (the split-keys decode kernel, at the sizes it takes).  ``softcap`` > 0: the scaled scores
@@ -709,10 +799,12 @@ def attention_ext(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, o
     visible.  ``sink`` [n_q] float32: exp(sink[h]) is one more term of head h's softmax denominator; it has
     no key and no value.  ``all_value_heads``: every query head's weights are applied to each of the ``n_kv``
     value heads; ``out`` is then float32 [T, n_q, n_kv, dv] (for ``attn_head_mix``).  Otherwise ``out`` is
-    [T, n_q * dv] in q's dtype, or float32 if it is given so."""
+    [T, n_q * dv] in q's dtype, or float32 if it is given so.  ``value_dim`` (with ``v_pool`` the same memory as
+    ``k_pool``): the values are the first so many columns of the keys."""
     T = q.shape[0]
     num_blocks, _, block_size, _ = k_pool.shape
-    v_dim = v_pool.shape[-1]
+    assert not value_dim or v_pool.data_ptr() == k_pool.data_ptr()
+    v_dim = value_dim or v_pool.shape[-1]
     v_rep = n_kv if all_value_heads else 1
     assert q.dtype == k_pool.dtype == v_pool.dtype and k_pool.shape[-1] == head_dim
     assert out.dtype in (q.dtype, torch.float32) and out.numel() == T * n_q * v_rep * v_dim
@@ -731,7 +823,7 @@ def attention_ext(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, o
         n_rows, T, max_q_len, n_q, n_kv, head_dim, float(scale), int(window), int(v_dim), int(chunk), n_splits,
         split_len, _ptr(scratch), _ptr(status), float(softcap), int(keep_first), _ptr(sink), v_rep,
         int(out.dtype == torch.float32 and q.dtype != torch.float32 or all_value_heads), int(tensor_cores),
-        _ptr(_counters(q.device, n_rows * n_q)) if fused else None, _stream()))
+        _ptr(_counters(q.device, n_rows * n_q)) if fused else None, k_pool.shape[-1] if value_dim else 0, _stream()))
 
 
 def _col_ptr(t: torch.Tensor, first_col: int) -> int:
@@ -795,14 +887,15 @@ def linear_scan(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, state: t
                 lower: Optional[torch.Tensor] = None, cos: Optional[torch.Tensor] = None,
                 sin: Optional[torch.Tensor] = None, rot_dims: int = 0, k_scale: float = 1.0, max_q_len: int = 0,
                 scratch: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, gate_col: int = 0,
-                q_scale: float = 1.0, tau: float = 1.0) -> None:
+                q_scale: float = 1.0, tau: float = 1.0, silu: bool = False) -> None:
     """The recurrence S_t = diag(a_t) S_(t-1) + b_t v_t^T, o_t = S_t^T q_t per sequence and head over the step's
     tokens, from ``state`` [slots, heads, head_dim, v_head_dim] (float32, updated when ``write_state``) to ``out``
     [T, heads * v_head_dim] (float32).  q, k and v are column ranges of ``proj`` [T, ld].  ``SCAN_DECAY``: a = decay[h],
     b = rotated k times ``k_scale``, q rotated (the first ``rot_dims`` dimensions, i paired with i + rot_dims / 2).
     ``SCAN_GATED``: the k columns hold the gate's pre-activation z; a = lower + (1 - lower) sigmoid(z), b = 1 - a,
     q = silu of the q columns.  ``SCAN_CHANNEL_DECAY``: a = sigmoid(z)^(1 / tau) per key channel with z the columns
-    ``gate_col ...`` of ``gate`` [T, ldg] (float32), b = the k columns, q = the q columns times ``q_scale``.  With ``scratch`` (float32, ``linear_scan_scratch_floats`` elements) and ``max_q_len`` (the
+    ``gate_col ...`` of ``gate`` [T, ldg] (float32), b = the k columns, q = the q columns times ``q_scale``.
+    ``silu`` (``SCAN_DECAY`` without a rotation): q, k and v pass silu on their way in.  With ``scratch`` (float32, ``linear_scan_scratch_floats`` elements) and ``max_q_len`` (the
     longest portion of the step), portions longer than two segments are cut into segments that run side by side."""
     T = proj.shape[0]
     assert state.dtype == out.dtype == torch.float32 and state.shape[1:] == (n_heads, head_dim, v_head_dim)
@@ -827,7 +920,7 @@ def linear_scan(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, state: t
                                 _ptr(scratch) if scratch is not None else None,
                                 scratch.numel() if scratch is not None else 0,
                                 _col_ptr(gate, gate_col) if gate is not None else None,
-                                gate.shape[1] if gate is not None else 0, float(q_scale), 1.0 / float(tau), _stream()))
+                                gate.shape[1] if gate is not None else 0, float(q_scale), 1.0 / float(tau), int(silu), _stream()))
 
 
 def linear_scan_segment() -> int:
@@ -851,6 +944,16 @@ def low_rank_expand(x: torch.Tensor, first_col: int, w: torch.Tensor, bias: Opti
     assert bias is None or (bias.dtype == torch.float32 and bias.numel() == N)
     _check(lib().fd_low_rank_expand(_col_ptr(x, first_col), x.shape[1], _ptr(w), _ptr(bias), _ptr(out), _dt(x.dtype),
                                     T, N, R, _stream()))
+
+
+def row_norm_gate(o: torch.Tensor, weight: torch.Tensor, gate: torch.Tensor, gate_col: int, out: torch.Tensor, eps: float) -> None:
+    """out[t] = o[t] / sqrt(mean(o[t]^2) + eps) * weight * sigmoid(gate[t, gate_col ...]): one norm over the whole row.  ``o``
+    float32 [T, n], ``weight`` float32 [n], ``gate`` a packed projection [T, ldg] in out's dtype, ``out`` [T, n]."""
+    T, n = o.shape
+    assert o.dtype == weight.dtype == torch.float32 and out.shape == (T, n) and weight.numel() == n
+    assert gate.dtype == out.dtype and gate.shape[0] == T and gate_col + n <= gate.shape[1]
+    _check(lib().fd_row_norm_gate(_ptr(o), _ptr(weight), _col_ptr(gate, gate_col), gate.shape[1], _ptr(out), _dt(out.dtype), T,
+                                  n, float(eps), _stream()))
 
 
 def head_norm_gate(o: torch.Tensor, out: torch.Tensor, first_col: int, n_heads: int, v_head_dim: int, eps: float,

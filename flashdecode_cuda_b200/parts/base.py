@@ -154,6 +154,10 @@ class Block(Part):
     # True: ``forward`` takes the incoming ``delta`` as float32 partial sums [parts, T, H] too
     accepts_parts = False
 
+    def extra_state_requests(self) -> List[StateSpec]:
+        """Per-sequence state that the layer keeps beside its mixer's (under other names)."""
+        return []
+
     def stream_state(self, resid: torch.Tensor, delta) -> torch.Tensor:
         """The residual stream [T, H] (float32, a new tensor) as it stands once ``delta``, what this block's ``forward``
         returned, has been added: what a per-layer trace records.  A block whose stream or delta has another form

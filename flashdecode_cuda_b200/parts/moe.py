@@ -2,6 +2,7 @@
 
 from __future__ import annotations
 
+from dataclasses import dataclass
 from typing import Dict, List, Optional
 
 import torch
@@ -23,6 +24,14 @@ ROUTE_FUSED_MAX_WEIGHTS = 65536
 # kernel where it takes the sizes (expert matrices of at least 256 rows), else the mma.sync kernel; "mma": the
 # mma.sync kernel always (tests run both).
 GROUPED_GEMM = "auto"
+
+
+@dataclass
+class PendingExperts:
+    """The chosen experts' rows of a step before they are summed: out[t] = sum_c wts[t, c] * y[pair_pos[t, c]]."""
+    y: torch.Tensor                 # [grouped rows, H]
+    wts: torch.Tensor               # [T, top] float32
+    pair_pos: torch.Tensor          # [T * top] int32; -1: nothing
 
 
 @register_part("feed_forward", "routed_experts")
@@ -50,6 +59,8 @@ class RoutedExperts(FeedForward):
     ``<prefix>.e<i>.up`` [ff, hidden], ``<prefix>.e<i>.down`` [hidden, ff], ``<prefix>.router``,
     ``<prefix>.correction``, ``<prefix>.shared.up`` / ``.down``.
     """
+
+    offers_pairs = True         # ``forward(..., pairs_ok=True)``
 
     def __init__(self, prefix: str, hidden_size: int, n_experts: int, top: int, expert_ff: int, n_identity: int = 0,
                  shared_ff: Optional[int] = None, correction: bool = True, expert_act: str = "relu2",
@@ -145,7 +156,9 @@ class RoutedExperts(FeedForward):
         shared = ws.get("moe_shared_out", (T, H), x.dtype)
         return matmul(h, self.s_down, None, shared, target_ctas=4 * self.rt.sm_count, status=self.rt.status)
 
-    def forward(self, ctx, x: torch.Tensor, parts_ok: bool = False) -> torch.Tensor:
+    def forward(self, ctx, x: torch.Tensor, parts_ok: bool = False, pairs_ok: bool = False):
+        """[T, H]; with ``pairs_ok``, where nothing but experts with weights can be chosen, their rows unsummed
+        (``PendingExperts``) for a consumer that sums them itself."""
         T, ws, H, top = ctx.T, ctx.ws, self.hidden_size, self.top
         # the shared expert depends on nothing of the routing.  (On a second stream beside the routed experts it gained
         # 4 % in a 2,048-token prompt step at width 2,048, lost 10 % at width 1,024, where the host sets the pace, and
@@ -202,6 +215,8 @@ class RoutedExperts(FeedForward):
                 else:
                     K.moe_gemm(x, self.w_up, act, False, sorted_pair, tile_expert, n_tiles, top, mt)
                 K.moe_gemm(act, self.w_down, y, True, sorted_pair, tile_expert, n_tiles, top, mt)
+        if pairs_ok and shared is None and self.n_identity == 0:
+            return PendingExperts(y, wts, pair_pos)
         out = ws.get("ffn_out", (T, H), x.dtype)
         K.moe_combine(y, x, shared, ids, wts, pair_pos, out, self.E)
         return out

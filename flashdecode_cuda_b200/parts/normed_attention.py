@@ -1,6 +1,6 @@
-"""Attention mixers without a rotation: grouped-query attention whose q and k are normed over their whole
-projection, with a sliding window; and latent attention, which keeps one low-rank vector per position and makes
-every head's keys and values from it."""
+"""Attention mixers over normed projections: grouped-query attention whose q and k are normed over their whole
+projection, with a sliding window; and latent attention, which keeps one low-rank vector (and by option one small
+rotated key part) per position and makes every head's keys and values from it."""
 
 from __future__ import annotations
 
@@ -56,6 +56,15 @@ def _pad_heads(w: torch.Tensor, n_heads: int, size: int, padded: int) -> torch.T
     out = w.new_zeros((n_heads, padded) + tuple(w.shape[1:]))
     out[:, :size] = w.view((n_heads, size) + tuple(w.shape[1:]))
     return out.view((n_heads * padded,) + tuple(w.shape[1:]))
+
+
+def _pad_cols(w: torch.Tensor, size: int, padded: int) -> torch.Tensor:
+    """w [N, size] -> [N, padded]: zero columns at the end."""
+    if size == padded:
+        return w.contiguous()
+    out = w.new_zeros((w.shape[0], padded))
+    out[:, :size] = w
+    return out
 
 
 @register_part("mixer", "qk_normed_attention")
@@ -146,85 +155,133 @@ class LatentAttention(Mixer):
     """For the mixer's input h [T, hidden], with ``n_heads`` heads, ``head_dim`` query/key and ``v_head_dim`` value
     dimensions per head and a latent of ``kv_rank`` dimensions:
 
-        q   = W_q h                                        (no rotated part)
-        c   = (W_dkv h) / sqrt(mean((W_dkv h)^2) + eps) * w_c           the latent: all that is cached
+        q   = W_q h                                        or, with ``q_rank``, W_uq norm(W_dq h): through a latent of its own
+        c   = (W_dkv h) / sqrt(mean((W_dkv h)^2) + eps) * w_c           the latent: cached
         k_h = U_h c,  v_h = V_h c                          (U = ``.uk`` [heads * head_dim, kv_rank], V = ``.uv``, head by head)
         a_h = softmax over the visible keys j of (q_h . k_h[j]) * scale
         out = W_o [a_1 V-values ... ]
 
-    computed without ever expanding the cached positions: (q_h . U_h c) = (U_h^T q_h) . c, so the queries are taken
-    into the latent's basis (one small product per head), attention runs over the cached latents as ONE key/value head
-    of size ``kv_rank`` that all query heads share and that serves as key and as value, and V_h is applied to each
+    ``rot_dim`` > 0: a head's query has ``rot_dim`` more dimensions and W_dkv as many more rows, one key part k_r for all
+    heads; both are turned at their positions (``position``: pairs 2i, 2i + 1), q_h . k_h gains q_r,h . k_r, and k_r is cached
+    beside c.  ``sink``: exp(``.sink``[h]) is one more term of head h's denominator, without key or value.  ``gate``: the
+    concatenated heads are multiplied by sigmoid(W_g h).
+
+    Computed without ever expanding the cached positions: (q_h . U_h c) = (U_h^T q_h) . c, so the queries are taken
+    into the latent's basis (one small product per head), attention runs over the cached rows [c ; k_r] as ONE key/value
+    head that all query heads share and whose first ``kv_rank`` dimensions are the values, and V_h is applied to each
     head's attended latent afterwards.  Visible keys: j <= i, and with a ``window`` only i - j < window.
 
     Whole prompts in bfloat16 (a step whose sequences all start at their first token) take the other order where that
-    reaches a faster attention kernel: k_h and v_h of the step's own tokens are expanded by one product into pages of the
-    workspace, and attention runs over them with a key/value head per query head (``expands``); the cache still
-    receives the latents only.  Tensors ``<prefix>.q``, ``.dkv``, ``.dkv.norm``, ``.uk``, ``.uv``, ``.o``.
+    reaches a faster attention kernel: k_h and v_h of the step's own tokens are expanded by one product, and attention runs
+    over them with a key/value head per query head (``expands``); the cache still receives [c ; k_r] only.  Tensors
+    ``<prefix>.q`` (or ``.dq``, ``.dq.norm``, ``.uq``), ``.dkv``, ``.dkv.norm``, ``.uk``, ``.uv``, ``.sink``, ``.g``, ``.o``.
     """
 
     def __init__(self, prefix: str, hidden_size: int, n_heads: int, head_dim: int, v_head_dim: int, kv_rank: int,
-                 scale: float, eps: float, window: Optional[int] = None):
+                 scale: float, eps: float, window: Optional[int] = None, q_rank: Optional[int] = None, rot_dim: int = 0,
+                 position=None, sink: bool = False, gate: bool = False):
         _head_sizes_ok(prefix, latent_size=kv_rank)
-        if n_heads < 1 or n_heads > (64 if _up8(kv_rank) <= 256 else 32) or head_dim < 1 or v_head_dim < 1:
-            raise ValueError(f"{prefix}: {n_heads} heads of {head_dim} / {v_head_dim}: the attention kernel takes up to 64 "
-                             f"query heads on the one latent (32 on a latent wider than 256)")
+        if n_heads < 1 or head_dim < 1 or v_head_dim < 1 or (q_rank is not None and q_rank < 1):
+            raise ValueError(f"{prefix}: {n_heads} heads of {head_dim} / {v_head_dim}, query latent {q_rank}")
+        if rot_dim < 0 or rot_dim % 2 or (rot_dim and position is None) or _up8(kv_rank) + _up8(rot_dim) > 640:
+            raise ValueError(f"{prefix}: a rotated part of {rot_dim} dimensions beside a latent of {kv_rank}: it must be even "
+                             f"and both together at most 640")
         self.prefix, self.hidden_size = prefix, hidden_size
-        self.n_q, self.d, self.dv, self.r_true = n_heads, head_dim, v_head_dim, kv_rank
+        self.n_q, self.d, self.dv, self.r_true, self.rot = n_heads, head_dim, v_head_dim, kv_rank, rot_dim
         self.r = _up8(kv_rank)                     # the latent as the kernels see it: zero-padded to a multiple of 8
+        self.rp = _up8(rot_dim)                    # ... and the rotated part
+        self.q_rank, self.position, self.has_sink, self.has_gate = q_rank, position, bool(sink), bool(gate)
         self.scale, self.eps, self.window = float(scale), float(eps), window
 
     def tensor_specs(self) -> List[TensorSpec]:
         p, H = self.prefix, self.hidden_size
-        r = self.r_true
-        return [TensorSpec(f"{p}.q", (self.n_q * self.d, H), init="unit"),
-                TensorSpec(f"{p}.dkv", (r, H), init="unit"),
-                TensorSpec(f"{p}.dkv.norm", (r,), "vector", init="norm"),
-                TensorSpec(f"{p}.uk", (self.n_q * self.d, r), init="unit"),
-                TensorSpec(f"{p}.uv", (self.n_q * self.dv, r), init="unit"),
-                TensorSpec(f"{p}.o", (H, self.n_q * self.dv), init="unit")]
+        r, nq = self.r_true, self.n_q * (self.d + self.rot)
+        if self.q_rank is None:
+            specs = [TensorSpec(f"{p}.q", (nq, H), init="unit")]
+        else:
+            specs = [TensorSpec(f"{p}.dq", (self.q_rank, H), init="unit"),
+                     TensorSpec(f"{p}.dq.norm", (self.q_rank,), "vector", init="norm"),
+                     TensorSpec(f"{p}.uq", (nq, self.q_rank), init="unit")]
+        specs += [TensorSpec(f"{p}.dkv", (r + self.rot, H), init="unit"),
+                  TensorSpec(f"{p}.dkv.norm", (r,), "vector", init="norm"),
+                  TensorSpec(f"{p}.uk", (self.n_q * self.d, r), init="unit"),
+                  TensorSpec(f"{p}.uv", (self.n_q * self.dv, r), init="unit")]
+        if self.has_sink:
+            specs.append(TensorSpec(f"{p}.sink", (self.n_q,), "vector", init="sink"))
+        if self.has_gate:
+            specs.append(TensorSpec(f"{p}.g", (self.n_q * self.dv, H), init="unit"))
+        return specs + [TensorSpec(f"{p}.o", (H, self.n_q * self.dv), init="unit")]
 
     def kv_request(self) -> KVRequest:
-        return KVRequest(1, self.r, self.window, None, None, keys_only=True)
+        return KVRequest(1, self.r + self.rp, self.window, None, None, keys_only=True)
 
     def bind(self, tensors: Dict[str, torch.Tensor], rt: Runtime) -> None:
         self.rt = rt
-        p = self.prefix
+        p, n = self.prefix, self.n_q
         pad = lambda w: _pad_heads(w, 1, self.r_true, self.r)            # zero rows up to the padded latent size
-        self.w_in = torch.cat([tensors.pop(f"{p}.q"), pad(tensors.pop(f"{p}.dkv"))], dim=0).contiguous()     # [q | latent]
+        # Sizes of a head's parts in the activations.
+        self.dx, self.rx, self.vx = self.d, self.rot, self.dv
+        self.kx = self.dx + self.rx
+        w_q = tensors.pop(f"{p}.q" if self.q_rank is None else f"{p}.uq")
+        dkv = tensors.pop(f"{p}.dkv")
+        qr = self.qr = 0 if self.q_rank is None else _up8(self.q_rank)
+        first = w_q if self.q_rank is None else _pad_heads(tensors.pop(f"{p}.dq"), 1, self.q_rank, qr)
+        mats = [first, pad(dkv[:self.r_true]), _pad_heads(dkv[self.r_true:], 1, self.rot, self.rp)]     # [q | latent | k_r | gate]
+        self.gate_col = sum(m.shape[0] for m in mats)
+        if self.has_gate:
+            mats.append(_pad_heads(tensors.pop(f"{p}.g"), n, self.dv, self.vx))
+        self.w_in = torch.cat(mats, dim=0).contiguous()
+        self.w_uq = self.q_norm = None
+        if self.q_rank is not None:
+            self.w_uq = _pad_cols(w_q, self.q_rank, qr)
+            self.q_norm = _pad_heads(tensors[f"{p}.dq.norm"].float(), 1, self.q_rank, qr).contiguous()
         self.c_norm = pad(tensors[f"{p}.dkv.norm"].float()).contiguous()
         # per head: U_h^T [kv_rank, head_dim] takes a query into the latent's basis; V_h [v_head_dim, kv_rank]
-        uk, uv = tensors.pop(f"{p}.uk"), tensors.pop(f"{p}.uv")
-        if self.r != self.r_true:
-            uk, uv = pad(uk.t().contiguous()).t().contiguous(), pad(uv.t().contiguous()).t().contiguous()
-        self.w_qc = uk.view(self.n_q, self.d, self.r).transpose(1, 2).contiguous()
-        self.w_cv = uv.view(self.n_q, self.dv, self.r).contiguous()
+        uk = _pad_cols(_pad_heads(tensors.pop(f"{p}.uk"), n, self.d, self.dx), self.r_true, self.r)
+        uv = _pad_cols(_pad_heads(tensors.pop(f"{p}.uv"), n, self.dv, self.vx), self.r_true, self.r)
+        self.w_qc = uk.view(n, self.dx, self.r).transpose(1, 2).contiguous()
+        self.w_cv = uv.view(n, self.vx, self.r).contiguous()
         self.w_o = tensors[f"{p}.o"]
+        self.sink = tensors[f"{p}.sink"].float().contiguous() if self.has_sink else None
         # which attention kernel each order reaches (3 tcgen05, 2 mma.sync, 1 mma.sync at wide heads, 0 CUDA cores)
         rank = lambda size: {128: 3, 64: 2, 192: 1, 256: 1}.get(size, 0)
         latent, expanded = rank(self.r), (rank(self.d) if self.d == self.dv else 0)
-        self.expands = rt.dtype == torch.bfloat16 and (expanded > latent or (expanded == latent and expanded > 1
-                                                                              and 2 * self.r > self.d + self.dv))
+        self.expands = rt.dtype == torch.bfloat16 and not (self.rot or self.has_sink or self.has_gate or qr) and \
+            (expanded > latent or (expanded == latent and expanded > 1 and 2 * self.r > self.d + self.dv))
         self.w_kv = torch.cat([uk, uv], dim=0).contiguous() if self.expands else None      # [heads (d + dv), kv_rank]
 
     def weight_bytes(self) -> int:
         # (the expansion matrix is a second copy of .uk and .uv in another order: a step reads one of the two)
-        return sum(w.numel() * w.element_size() for w in (self.w_in, self.w_qc, self.w_cv, self.w_o))
+        mats = [self.w_in, self.w_qc, self.w_cv, self.w_o] + ([self.w_uq] if self.w_uq is not None else [])
+        return sum(w.numel() * w.element_size() for w in mats)
 
     def first_weights(self) -> Optional[torch.Tensor]:
         return self.w_in
 
+    def _append(self, ctx, proj: torch.Tensor, first: torch.Tensor, lc: LayerCache, **rows) -> None:
+        """The query latent normed (or the queries as they are) to ``first``, [c ; k_r] to the cache."""
+        rope = self.position if self.rot else None
+        K.norm_append(proj, first, self.q_norm, self.c_norm, self.eps, ctx.tok_row, ctx.tok_pos, ctx.row_slot, lc.k_pool,
+                      None, lc.group.table, 1, lc.writes, self.rt.status, q_count=self.q_rank or 0, k_count=self.r_true,
+                      cos=rope.cos if rope else None, sin=rope.sin if rope else None, rot=self.rot, rot_places=self.rp, **rows)
+
+    def _queries(self, ctx, first: torch.Tensor) -> torch.Tensor:
+        if self.w_uq is None:
+            return first
+        q = ctx.ws.get("lat_q", (ctx.T, self.n_q * self.kx), first.dtype)
+        return matmul(first, self.w_uq, None, q, target_ctas=4 * self.rt.sm_count, status=self.rt.status)
+
     def forward(self, ctx, x: torch.Tensor, lc: LayerCache) -> torch.Tensor:
-        T, ws, rt = ctx.T, ctx.ws, self.rt
+        T, ws, rt, n = ctx.T, ctx.ws, self.rt, self.n_q
         proj = ws.get("lat_proj", (T, self.w_in.shape[0]), x.dtype)
         matmul(x, self.w_in, None, proj, status=rt.status)
-        q = ws.get("lat_q", (T, self.n_q * self.d), x.dtype)
+        first = ws.get("lat_q_in", (T, self.qr or n * self.kx), x.dtype)
         out = ws.get("mixer_out", (T, self.hidden_size), x.dtype)
         if self.expands and ctx.max_q_len > 1 and not any(ctx.h_ctx_len):
             # whole prompts: expand the step's own keys and values and attend over them
             c = ws.get("lat_c", (T, self.r), x.dtype)
-            K.norm_append(proj, q, None, self.c_norm, self.eps, ctx.tok_row, ctx.tok_pos, ctx.row_slot, lc.k_pool, None,
-                          lc.group.table, 1, lc.writes, rt.status, k_rows=c, k_count=self.r_true)
+            self._append(ctx, proj, first, lc, k_rows=c)
+            q = self._queries(ctx, first)
             kv = ws.get("lat_kv", (T, self.w_kv.shape[0]), x.dtype)
             matmul(c, self.w_kv, None, kv, status=rt.status)
             bs = lc.group.block_size
@@ -243,15 +300,26 @@ class LatentAttention(Mixer):
                         ctx.n_rows, ctx.max_q_len, self.n_q, self.n_q, self.d, self.scale, self.window or 0, 1, 0, None,
                         rt.status)
             return matmul(av, self.w_o, None, out, target_ctas=4 * rt.sm_count, status=rt.status)
-        K.norm_append(proj, q, None, self.c_norm, self.eps, ctx.tok_row, ctx.tok_pos, ctx.row_slot, lc.k_pool, None,
-                      lc.group.table, 1, lc.writes, rt.status, k_count=self.r_true)
-        qc = ws.get("lat_qc", (T, self.n_q * self.r), x.dtype)
-        K.head_gemm(q, self.w_qc, qc)
-        ac = ws.get("lat_ac", (T, self.n_q * self.r), x.dtype)
-        n_splits, split_len, scratch = decode_splits(ctx, self.n_q, 1, self.r, x.dtype, rt, self.r)
-        K.attention(qc, lc.k_pool, lc.k_pool, ac, lc.group.table, ctx.tok_row, ctx.row_slot, ctx.row_q_start,
-                    ctx.row_q_len, ctx.row_ctx_len, ctx.n_rows, ctx.max_q_len, self.n_q, 1, self.r, self.scale,
-                    self.window or 0, n_splits, split_len, scratch, rt.status)
-        v = ws.get("lat_v", (T, self.n_q * self.dv), x.dtype)
-        K.head_gemm(ac, self.w_cv, v)
-        return matmul(v, self.w_o, None, out, target_ctas=4 * rt.sm_count, status=rt.status)
+        self._append(ctx, proj, first, lc)
+        q = self._queries(ctx, first)
+        size = self.r + self.rp
+        qc = ws.get("lat_qc", (T, n * size), x.dtype)
+        K.head_gemm(q, self.w_qc, qc, a_size=self.kx, out_size=size)
+        if self.rot:
+            K.rope_heads(q, self.kx, self.dx, qc, size, self.r, self.position.cos, self.position.sin, ctx.tok_pos, n, self.rot,
+                         self.rp, rt.status)
+        ac = ws.get("lat_ac", (T, n * self.r), x.dtype)
+        n_splits, split_len, scratch = decode_splits(ctx, n, 1, self.r, x.dtype, rt, size if not self.rot else 0)
+        args = (qc, lc.k_pool, lc.k_pool, ac, lc.group.table, ctx.tok_row, ctx.row_slot, ctx.row_q_start, ctx.row_q_len,
+                ctx.row_ctx_len, ctx.n_rows, ctx.max_q_len, n, 1, size, self.scale, self.window or 0, n_splits, split_len,
+                scratch, rt.status)
+        if self.rot or self.has_sink:
+            K.attention_ext(*args, sink=self.sink, value_dim=self.r if self.rot else 0)
+        else:
+            K.attention(*args)
+        v = ws.get("lat_v", (T, n * self.vx), x.dtype)
+        gated = self.has_gate and (T < K.HEAD_GEMM_LIBRARY_ROWS or x.dtype != torch.bfloat16)
+        K.head_gemm(ac, self.w_cv, v, gate=proj if gated else None, gate_col=self.gate_col)
+        if self.has_gate and not gated:
+            K.gate_mul(v, proj, self.gate_col, v)
+        return matmul(v, self.w_o, None, out, target_ctas=4 * rt.sm_count, status=rt.status, upcoming=ctx.upcoming)

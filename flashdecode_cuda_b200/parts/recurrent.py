@@ -1,5 +1,5 @@
 """Mixers that carry a matrix state per head instead of keys: linear attention with a constant decay per head
-(retention) and with a forget gate per channel that also decides what is written (a gated linear recurrence)."""
+(retention, lightning attention) and with a forget gate per channel that also decides what is written (a gated linear recurrence)."""
 
 from __future__ import annotations
 
@@ -107,6 +107,57 @@ class Retention(_StateMixer):
                       sin=rope.sin if self.rot_dims else None, rot_dims=self.rot_dims, k_scale=self.d ** -0.5,
                       max_q_len=ctx.max_q_len, scratch=self.scan_scratch(ctx))
         K.head_norm_gate(o, act, act_col, self.n_heads, self.dv, self.eps, None, proj, col0 + 2 * nk + nv, scale)
+        return act
+
+
+@register_part("mixer", "lightning_attention")
+class LightningAttention(_StateMixer):
+    """Linear attention with a constant decay per head.  For the mixer's input h [T, hidden], per head with the decay g_h:
+
+        q = silu(W_q h);  k = silu(W_k h);  v = silu(W_v h)                 (no biases, no other scale)
+        S_t = g_h S_(t-1) + k_t v_t^T;   o_t = S_t^T q_t
+        out = W_o ( norm(o) * sigmoid(W_g h) )           norm over the heads side by side, weight [heads * v_head_dim]
+
+    The state starts at zero and is carried in float32 per cache slot; silu, decay, state, output, norm and gate are
+    float32 in both dtypes.  Tensors ``<prefix>.q`` / ``.k`` / ``.v`` / ``.g`` / ``.norm`` / ``.o``."""
+
+    shares_products = False
+
+    def __init__(self, prefix: str, hidden_size: int, n_heads: int, head_dim: int, v_head_dim: int,
+                 decay: Sequence[float], eps: float):
+        if len(decay) != n_heads:
+            raise ValueError(f"{prefix}: {len(decay)} decays for {n_heads} heads")
+        if head_dim > 256 or min(n_heads, head_dim, v_head_dim) < 1:
+            raise ValueError(f"{prefix}: heads of {head_dim} x {v_head_dim}: the recurrence takes key sizes up to 256")
+        self.prefix, self.hidden_size = prefix, hidden_size
+        self.n_heads, self.d, self.dv = n_heads, head_dim, v_head_dim
+        self.decay, self.eps = [float(g) for g in decay], float(eps)
+
+    def tensor_specs(self) -> List[TensorSpec]:
+        p, H = self.prefix, self.hidden_size
+        nk, nv = self.n_heads * self.d, self.n_heads * self.dv
+        return [TensorSpec(f"{p}.q", (nk, H), init="unit"), TensorSpec(f"{p}.k", (nk, H), init="unit"),
+                TensorSpec(f"{p}.v", (nv, H), init="unit"), TensorSpec(f"{p}.g", (nv, H), init="unit"),
+                TensorSpec(f"{p}.norm", (nv,), "vector", init="norm"), TensorSpec(f"{p}.o", (H, nv), init="unit")]
+
+    def bind(self, tensors: Dict[str, torch.Tensor], rt: Runtime) -> None:
+        self.rt = rt
+        p = self.prefix
+        self.w_in = torch.cat([tensors.pop(f"{p}.{n}") for n in "qkvg"], dim=0).contiguous()
+        self.b_in = None
+        self.norm_w = tensors.pop(f"{p}.norm").float().contiguous()
+        self.w_o = tensors[f"{p}.o"]
+        self.decay_dev = torch.tensor(self.decay, dtype=torch.float32, device=rt.device)
+
+    def inner(self, ctx, proj: torch.Tensor, col0: int, lc: LayerCache, act: torch.Tensor, act_col: int = 0,
+              scale: float = 1.0) -> torch.Tensor:
+        nk, nv = self.n_heads * self.d, self.n_heads * self.dv
+        o = ctx.ws.get("scan_out", (ctx.T, nv), torch.float32)
+        K.linear_scan(proj, col0, col0 + nk, col0 + 2 * nk, lc.states["state"], o, K.SCAN_DECAY, ctx.row_slot,
+                      ctx.row_q_start, ctx.row_q_len, ctx.row_ctx_len, ctx.n_rows, self.n_heads, self.d, self.dv,
+                      lc.writes, self.rt.status, decay=self.decay_dev, max_q_len=ctx.max_q_len,
+                      scratch=self.scan_scratch(ctx), silu=True)
+        K.row_norm_gate(o, self.norm_w, proj, col0 + 2 * nk + nv, act, self.eps)
         return act
 
 

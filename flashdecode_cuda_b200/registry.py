@@ -7,8 +7,10 @@
   chosen through this table.
 * ``PARTS``: (kind, name) -> the class that implements a part.  Kinds are
   ``embedding``, ``position``, ``norm``, ``mixer``, ``feed_forward``, ``block``,
-  ``head``, ``stream_op``, ``table`` (a lookup table several parts share) and
-  ``side_input`` (what a layer adds from the token itself).  A blueprint names parts by (kind, name); nothing else in the
+  ``head``, ``stream_op``, ``table`` (a lookup table several parts share),
+  ``side_input`` (what a layer adds from the token itself), ``input_conv`` (a
+  convolution over time of what a mixer reads) and ``depth_average`` (an average
+  over the layers' results so far).  A blueprint names parts by (kind, name); nothing else in the
   engine knows a part's class.
 
 A new architecture or part is added by calling ``register_architecture`` /
@@ -22,7 +24,7 @@ from dataclasses import dataclass
 from typing import Callable, Dict, Tuple, Type
 
 PART_KINDS = ("embedding", "position", "norm", "mixer", "feed_forward", "block", "head", "stream_op", "table",
-              "side_input")
+              "side_input", "input_conv", "depth_average")
 
 
 @dataclass(frozen=True)

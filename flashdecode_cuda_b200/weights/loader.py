@@ -129,6 +129,11 @@ def random_tensor(spec: TensorSpec, seed: int, dtype: torch.dtype, device="cpu")
             t = 2.0 + t
         elif spec.init == "unit_rows":          # rows of a lookup table whose entries multiply activations: about one
             pass
+        elif spec.init == "conv_small":          # a convolution that is added to its own input
+            t = 0.2 * t
+        elif spec.init == "depth":               # an average over depth: about the last entry
+            t = 0.1 * t
+            t[-1] += 1.0
         elif spec.init in ("normal", "bias", "embedding"):
             t = 0.02 * t
         else:
