@@ -29,7 +29,9 @@ benchmark configuration says; the library's own default of 64 is measured
 beside it (``points.decode_b8_block64``, ``points.prefill_block64_ms``).
 
 ``--compare nizazen`` does the same for the Nizazen design (eight layers that alternate windowed and latent attention,
-dense and routed feed-forwards, on a residual stream of several lanes).  ``--compare botusun`` measures the Botusun design (six
+dense and routed feed-forwards, on a residual stream of several lanes).  ``--compare gulozen`` measures the Gulozen design (eight layers: latent
+attention with a rotated key part and lightning attention, routed feed-forwards, norms on the outputs, an average over the
+depth) beside the Nizazen design at equal sizes.  ``--compare botusun`` measures the Botusun design (six
 layers, two of them twice: linear attention with a decay per key channel and windowed attention over convolved, normed keys, dense and routed
 feed-forwards, a contribution of the token itself after every layer) beside the Revelix design at equal sizes.  ``--compare revelix`` for the Revelix design (eight layers that alternate retention and attention beside a gated
 recurrence, each with a dense feed-forward).  ``--compare lonasun`` leaves all of that aside and measures the Lonasun design beside the Qwen2 dense decoder of the
@@ -414,9 +416,44 @@ def botusun_configs(sz: dict):
     return botu, reve
 
 
+GULOZEN_SIZES = {
+    # width, heads, own key dimensions, rotated ones, value dimensions, query latent, latent, experts, choices, expert ff; heads
+    # and head size of the lightning layers, taps, norm groups
+    "w1024": dict(width=1024, heads=8, dim=128, rot=64, vdim=128, q_rank=512, rank=256, experts=16, top=4, ff=512, l_heads=8,
+                  l_dim=128, taps=4, groups=4),
+    "w2048": dict(width=2048, heads=16, dim=128, rot=64, vdim=128, q_rank=768, rank=512, experts=32, top=6, ff=768, l_heads=16,
+                  l_dim=128, taps=4, groups=4),
+    "w2048-d64": dict(width=2048, heads=32, dim=64, rot=64, vdim=64, q_rank=768, rank=256, experts=64, top=8, ff=512, l_heads=16,
+                      l_dim=128, taps=3, groups=2),
+}
+
+
+def gulozen_configs(sz: dict):
+    """(Gulozen config dictionary, Nizazen config dictionary) of equal width, layers, heads, head sizes, latent and routed
+    feed-forwards.  Gulozen: eight layers, six of latent attention and two of lightning attention, each with a mixture of
+    experts.  Beside it the closest design the library has: Nizazen with eight layers of latent attention without a rotated
+    part, each with a mixture of as many experts of the same size, on a stream of two lanes."""
+    lat = {"dim": sz["dim"], "heads": sz["heads"], "kv_rank": sz["rank"], "q_rank": sz["q_rank"], "rot_dim": sz["rot"],
+           "rot": {"base": 1000000.0, "dims": sz["rot"], "scaling": {"factor": 8.0, "original": 1024, "fast": 32.0, "slow": 1.0}},
+           "scale": (sz["dim"] + sz["rot"]) ** -0.5, "vdim": sz["vdim"]}
+    h = sz["l_heads"]
+    lin = {"decay": [1.0 - 2.0 ** (-5 - 5 * i / max(h - 1, 1)) for i in range(h)], "dim": sz["l_dim"], "heads": h, "vdim": sz["l_dim"]}
+    moe = {"expert": {"ff": sz["ff"]}, "kind": "moe", "router": {"experts": sz["experts"], "top": sz["top"]}}
+    kinds = [("latent_attention", lat), ("latent_attention", lat), ("lightning", lin), ("latent_attention", lat)]
+    gulo = {"architecture": "Gulozen", "vocab": COMPARE_VOCAB, "width": sz["width"], "norm": {"eps": 1e-5, "groups": sz["groups"]},
+            "canon": {"taps": sz["taps"]}, "embedding": {"scale": 8.0},
+            "layers": [{"type": t, "mixer": m, "mlp": moe} for t, m in kinds * 2]}
+    nlat = {"dim": sz["dim"], "heads": sz["heads"], "kv_rank": sz["rank"], "scale": sz["dim"] ** -0.5, "vdim": sz["vdim"]}
+    nmoe = {"expert": {"ff": sz["ff"], "limit": 7.0}, "kind": "moe", "router": {"experts": sz["experts"], "top": sz["top"]}}
+    niza = {"architecture": "Nizazen", "vocab": COMPARE_VOCAB, "width": sz["width"], "norm": {"eps": 1e-5}, "streams": 2,
+            "logit_softcap": 30.0, "layers": [{"type": "latent_attention", "mixer": nlat, "mlp": nmoe} for _ in range(8)]}
+    return gulo, niza
+
+
 # design -> (sizes, function of a size that gives both configurations, the key of the model that stands beside it)
 COMPARISONS = {"lonasun": (COMPARE_SIZES, compare_configs, "qwen2"), "nizazen": (NIZAZEN_SIZES, nizazen_configs, "qwen2"),
-               "revelix": (REVELIX_SIZES, revelix_configs, "qwen2"), "botusun": (REVELIX_SIZES, botusun_configs, "revelix")}
+               "revelix": (REVELIX_SIZES, revelix_configs, "qwen2"), "botusun": (REVELIX_SIZES, botusun_configs, "revelix"),
+               "gulozen": (GULOZEN_SIZES, gulozen_configs, "nizazen")}
 
 
 def compare_one(cfgd: dict, pk: dict, batch: int, context: int, prompt: int, steps: int, warmup: int, seed: int) -> dict:
@@ -544,7 +581,7 @@ def compare_main(args) -> int:
                 a, b = entry[design][phase]["parts"][part], entry[beside][phase]["parts"][part]
                 entry["ratios"][f"{phase}_{part}_frac"] = [a["frac"], b["frac"], round(a["frac"] / b["frac"], 3)]
         sizes[name] = entry
-    print(json.dumps({"compare": design, "beside": {"qwen2": "Qwen2ForCausalLM", "revelix": "Revelix"}[beside], "dtype": "bf16", "data": "synthetic: random weights",
+    print(json.dumps({"compare": design, "beside": {"qwen2": "Qwen2ForCausalLM", "revelix": "Revelix", "nizazen": "Nizazen"}[beside], "dtype": "bf16", "data": "synthetic: random weights",
                       "peaks": pk, "batch": args.batch, "prompt": 2048, "context": 2048, "block_size": LIB_BLOCK_SIZE,
                       "clocks": clocks.stop(), "sizes": sizes}))
     return 0
@@ -760,7 +797,7 @@ def main() -> int:
     ap.add_argument("--no-fp32", action="store_true", help="skip the float32 point (slow at the larger presets)")
     ap.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"],
                     help="float32: the main run through the true 32-bit path (with --no-points)")
-    ap.add_argument("--compare", default="", choices=["", "lonasun", "nizazen", "revelix", "botusun"],
+    ap.add_argument("--compare", default="", choices=["", "lonasun", "nizazen", "revelix", "botusun", "gulozen"],
                     help="measure this design beside the closest dense model at equal sizes instead of the default run")
     ap.add_argument("--compare-sizes", default="", help="with --compare: names of the sizes to run, with commas (default: all)")
     ap.add_argument("--device", default="cuda", choices=["cuda", "cpu"],

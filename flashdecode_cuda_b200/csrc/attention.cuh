@@ -39,6 +39,11 @@ struct AttnParams {
                                // n_kv heads); out is then [T, n_q, v_rep, dv]
     int v_all;                 // set by the CUDA-core launcher: a CTA takes a key head and all v_rep value heads, not one
     int out_f32;               // out is float whatever the type of q and the pools
+    // whole prompts over plain rows only (attention_prefill_tcgen05.cu): slabs of 64 key dimensions that are a head's own, and
+    // the heads' output gate, [T, gate_ld], or null
+    int dense_kn;
+    const __nv_bfloat16* gate;
+    int gate_ld;
     // decode steps on the tensor cores only: memory that a later kernel streams (the next part's first weights), or
     // null; every CTA asks L2 for its share once its own keys and values are through
     const unsigned char* pf_ptr;
@@ -50,6 +55,9 @@ struct AttnParams {
 int launch_attn_decode_mma(const AttnParams& p, int n_rows, cudaStream_t stream);
 // prompt steps (several new tokens per row) on the tensor cores; same return convention
 int launch_attn_prefill_mma(const AttnParams& p, int n_rows, int max_q_len, cudaStream_t stream);
+// decode steps and later portions of prompts over one cached row per position that is every head's key and, its first dv
+// dimensions, every head's value (n_kv 1, bfloat16)
+int launch_attn_latent_mma(const AttnParams& p, const int* tok_row, int T, cudaStream_t stream);
 // prompt steps with capped scores, kept first keys, a keyless softmax term or repeated value heads (head sizes 64 and 128)
 int launch_attn_prefill_mma_ext(const AttnParams& p, int n_rows, int max_q_len, cudaStream_t stream);
 // the same on the tcgen05 tensor cores (head size 128, block sizes 8..128 that divide 128)

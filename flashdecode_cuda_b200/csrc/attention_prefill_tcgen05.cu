@@ -1,4 +1,5 @@
-// Prompt attention on the 5th-generation tensor cores (head size 128, bfloat16):
+// Prompt attention on the 5th-generation tensor cores (bfloat16; from the paged cache at head size 128, and from plain
+// rows - the second form of reading, below - at key sizes of 64, 128 or 192 and value sizes of 64 or 128):
 // causal, grouped-query, paged, variable lengths, optional window, continuing a
 // cached prefix.  A CTA takes 256 consecutive query tokens of one sequence and
 // one query head as two query tiles of 128 rows, and walks the keys in tiles of
@@ -36,6 +37,12 @@
 // heads, so no long tile starts in a late wave.  A prompt so short that this
 // grid leaves SMs empty runs a second form of the kernel (SPLIT below): 128
 // queries per CTA, their key tiles dealt to the two groups of softmax warps.
+//
+// DENSE: the keys and values of whole prompts as plain rows, one per token of the step, before anything is paged: kv
+// [T, heads * (64 KN + 64 VS)] holds every head's own key dimensions and its value (a latent attention's expanded keys and
+// values, as the product left them), rot [T, 64 (KS - KN)] a key part that all heads share.  A key tile is then KS + VS
+// boxes of 64 tokens x 64 dimensions.  KS and VS are the key's and the value's dimensions in units of 64.  The epilogue can
+// multiply the heads by sigmoid(gate).
 #include <cuda.h>
 #include <math.h>
 
@@ -48,7 +55,7 @@
 
 namespace fd {
 
-constexpr int TA_D = 128;                 // head size
+constexpr int TA_D = 128;                 // head size of the paged form
 constexpr int TA_BM = 128;                // queries per query tile (the M of the MMAs)
 constexpr int TA_BN = 64;                 // keys per tile
 constexpr int TA_STAGES = 3;              // key/value tiles in flight
@@ -58,12 +65,17 @@ constexpr int TA_PV_WARP = 2 + 4 * TA_NQ;  // warps: 0 TMA, 1 issuer of Q K^T, 2
 constexpr int TA_THREADS = (TA_PV_WARP + 1) * 32;
 constexpr int TA_QSLAB = TA_BM * 128;     // bytes of a [128 queries][64 bf16] slab (Q: two of them; P: one)
 constexpr int TA_KSLAB = TA_BN * 128;     // bytes of a [64 keys][64 bf16] slab (K and V: two each)
-constexpr int TA_QTILE = 2 * TA_QSLAB;    // Q [128][128]
 constexpr int TA_PTILE = TA_QSLAB;        // P [128][64]
-constexpr int TA_KTILE = 2 * TA_KSLAB;    // K or V [64][128]
-// 192 KB + barriers, one CTA per SM: two query tiles (Q 32 KB and P 16 KB each) and three key/value tiles
-// in flight (32 KB each); with one query tile per CTA (see the kernel), one Q and four key/value tiles
-constexpr int TA_SMEM = TA_NQ * (TA_QTILE + TA_PTILE) + TA_STAGES * 2 * TA_KTILE + 256;
+// Key/value tiles in flight for KS key slabs and VS value slabs of 64 dimensions: what fits 227 KB beside the queries (one
+// query tile per CTA with SPLIT, see the kernel, else two) and P, one CTA per SM.
+__host__ __device__ constexpr int ta_stages(int ks, int vs, bool split) {
+    return ks == 3 ? (vs == 2 ? (split ? 3 : 2) : (split ? 4 : 3)) : (vs == 2 ? (split ? TA_STAGES + 1 : TA_STAGES) : (split ? 5 : 4));
+}
+__host__ __device__ constexpr int ta_smem(int ks, int vs, bool split) {
+    return (split ? 1 : TA_NQ) * ks * TA_QSLAB + TA_NQ * TA_PTILE + ta_stages(ks, vs, split) * (ks + vs) * TA_KSLAB + 256;
+}
+static_assert(ta_smem(2, 2, false) <= 232448 && ta_smem(3, 2, false) <= 232448 && ta_smem(3, 1, false) <= 232448 &&
+              ta_smem(3, 2, true) <= 232448 && ta_smem(3, 1, true) <= 232448, "shared memory of a CTA");
 
 __device__ __forceinline__ uint32_t ta_saddr(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
 __device__ __forceinline__ unsigned long long ta_ns() {
@@ -160,21 +172,22 @@ __device__ __forceinline__ uint64_t ta_desc_mn(uint32_t addr, uint32_t slab_byte
 // up.  A query tile's chain of key tiles - what bounds the time of a short prompt, whose few CTAs do not fill
 // the GPU - is half as long this way; every key tile is then used by one group only, which a long prompt pays
 // for in shared-memory and L2 traffic, so the launcher picks this form only while the other leaves SMs idle.
-template <bool SPLIT>
+template <int KS, int VS, bool SPLIT, bool DENSE>
 __global__ void __launch_bounds__(TA_THREADS, 1)
 attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
-                            const __grid_constant__ CUtensorMap map_v, const AttnParams p,
+                            const __grid_constant__ CUtensorMap map_v, const __grid_constant__ CUtensorMap map_r, const AttnParams p,
                             const unsigned long long wait_ns, const int skip_last) {
-    // SPLIT: one copy of the one query tile, and the 32 KB that saves as a fourth key/value tile in flight
-    constexpr int STAGES = SPLIT ? TA_STAGES + 1 : TA_STAGES;
+    // SPLIT: one copy of the one query tile, and what that saves as one more key/value tile in flight
+    constexpr int STAGES = ta_stages(KS, VS, SPLIT);
     constexpr int NQB = SPLIT ? 1 : TA_NQ;
-    static_assert(NQB * TA_QTILE + TA_NQ * TA_PTILE + STAGES * 2 * TA_KTILE + 256 <= TA_SMEM, "shared memory layout");
-    static_assert(STAGES * 2 * TA_KTILE >= (TA_D + 2) * TA_BM * 4, "the ring takes the second group's O, maxima and sums");
+    constexpr int DV = VS * 64, DK = KS * 64;
+    constexpr int QTILE = KS * TA_QSLAB, KTILE = KS * TA_KSLAB, STAGE = (KS + VS) * TA_KSLAB;
+    static_assert(!SPLIT || STAGES * STAGE >= (DV + 2) * TA_BM * 4, "the ring takes the second group's O, maxima and sums");
     extern __shared__ __align__(1024) unsigned char ta_raw[];
     unsigned char* q_s = ta_raw;                             // per query tile: [2 slabs][128 q][64 d]
-    unsigned char* p_s = q_s + NQB * TA_QTILE;             // per query tile: [128 q][64 keys]
+    unsigned char* p_s = q_s + NQB * QTILE;              // per query tile: [128 q][64 keys]
     unsigned char* kv_s = p_s + TA_NQ * TA_PTILE;            // per stage: K [2 slabs][64 keys][64 d], V the same
-    uint64_t* bars = reinterpret_cast<uint64_t*>(kv_s + STAGES * 2 * TA_KTILE);
+    uint64_t* bars = reinterpret_cast<uint64_t*>(kv_s + STAGES * STAGE);
     // bars: [0] q_full, kv_full[S], kv_empty[S]; per query tile: s_full[2], s_free[2], p_ready, o_done
     uint64_t* kv_full = bars + 1;
     uint64_t* kv_empty = kv_full + STAGES;
@@ -263,23 +276,24 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         // next 32 copies together, one chunk ahead, so that no copy waits for a table entry ----
         if (lane == 0) {
             // rows beyond the last token of the step are zero-filled; rows of a following sequence are computed and dropped
-            ta_expect(ta_saddr(&bars[0]), NQB * TA_QTILE);
+            ta_expect(ta_saddr(&bars[0]), NQB * QTILE);
 #pragma unroll
             for (int qt = 0; qt < NQB; ++qt) {
                 const int row = tok0 + qt * TA_BM;
-                ta_tma(ta_saddr(q_s + qt * TA_QTILE), &map_q, ta_saddr(&bars[0]), h * TA_D, row);
-                ta_tma(ta_saddr(q_s + qt * TA_QTILE + TA_QSLAB), &map_q, ta_saddr(&bars[0]), h * TA_D + 64, row);
+#pragma unroll
+                for (int sl = 0; sl < KS; ++sl)
+                    ta_tma(ta_saddr(q_s + qt * QTILE + sl * TA_QSLAB), &map_q, ta_saddr(&bars[0]), h * DK + sl * 64, row);
             }
         }
-        const int first_col = lo / bs;                        // blocks behind a window may have been given back
-        const int last_col = (hi - 1) / bs;                   // last block column that holds a key of this CTA
-        const int box = min(bs, TA_BN);                       // keys of one copy
+        const int first_col = DENSE ? 0 : lo / bs;                        // blocks behind a window may have been given back
+        const int last_col = DENSE ? 0 : (hi - 1) / bs;                   // last block column that holds a key of this CTA
+        const int box = DENSE ? TA_BN : min(bs, TA_BN);                       // keys of one copy
         const int per_tile = TA_BN / box;                     // 1, 2, 4 or 8 copies: chunks of 32 end with a tile
         const int n_boxes = n_tiles * per_tile;
         // block of the g-th copy of this CTA; one outside [first key, last key] is replaced by a valid one:
         // its data is masked, and the softmax warps zero its rows of V
         auto fetch = [&](int g) -> int {
-            if (g >= n_boxes) return 0;
+            if (DENSE || g >= n_boxes) return 0;
             const int col = max(first_col, min((t_begin + g * box) / bs, last_col));
             int blk = p.block_table[(size_t)slot * p.max_blocks + col];
             if (blk < 0 || blk >= p.num_blocks) { set_status(p.status, STATUS_BAD_BLOCK); blk = 0; }
@@ -293,15 +307,28 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             if (it >= STAGES) ok = ta_wait(ta_saddr(&kv_empty[s]), ((it / STAGES) - 1) & 1, abort_flag, p.status, wait_ns);
             if (!__all_sync(0xffffffffu, ok && *abort_flag == 0)) break;
             const uint32_t full = ta_saddr(&kv_full[s]);
-            if (lane == 0) ta_expect(full, 2 * TA_KTILE);
-            unsigned char* ks = kv_s + s * 2 * TA_KTILE;
-            unsigned char* vs = ks + TA_KTILE;
+            if (lane == 0) ta_expect(full, STAGE);
+            unsigned char* ks = kv_s + s * STAGE;
+            unsigned char* vs = ks + KTILE;
             const int t0 = t_begin + it * TA_BN;
             // The tile's copies (4 per cache block: K and V, each in two halves of the head) are issued by as
             // many lanes at once: one lane issuing them one after another took longer than the tile's tensor work.
             const int g0 = it * per_tile;                      // the tile's first copy group; chunks of 32 start on a tile
             if ((g0 & 31) == 0) { blk_cur = blk_next; blk_next = fetch(g0 + 32 + lane); }
             __syncwarp();                                      // the expectation is set before any copy can complete
+            if (DENSE) {
+                // one copy per slab: this head's key dimensions, the shared key part, this head's value
+                __syncwarp();                                  // the expectation is set before any copy can complete
+                if (lane < KS + VS && !(skip_last && it == n_tiles - 1 && lane == 0)) {
+                    const int row = p.row_q_start[b] + t0;
+                    const int kn = p.dense_kn;
+                    const bool shared_part = lane >= kn && lane < KS;
+                    const int col = shared_part ? (lane - kn) * 64 : (h * (kn + VS) + (lane < kn ? lane : lane - KS + kn)) * 64;
+                    ta_tma(ta_saddr(ks + lane * TA_KSLAB), shared_part ? &map_r : &map_k, full, col, row);
+                }
+                issued = it + 1;
+                continue;
+            }
             const int j = lane >> 2, part = lane & 3;
             const int blk = __shfl_sync(0xffffffffu, blk_cur, (g0 + j) & 31);
             if (j < per_tile && !(skip_last && it == n_tiles - 1 && lane == 0)) {      // tests: one copy of the last tile never leaves
@@ -328,7 +355,7 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         for (int it = 0; ok && it < n_tiles; ++it) {
             const int s = it % STAGES;
             ok = ta_wait(ta_saddr(&kv_full[s]), (it / STAGES) & 1, abort_flag, p.status, wait_ns);
-            const uint32_t ks = ta_saddr(kv_s + s * 2 * TA_KTILE);
+            const uint32_t ks = ta_saddr(kv_s + s * STAGE);
 #pragma unroll
             for (int qt = 0; qt < TA_NQ; ++qt) {
                 int j;
@@ -336,9 +363,9 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 if (j >= 2) ok = ta_wait(ta_saddr(&s_free[qt * 2 + (j & 1)]), ((j >> 1) - 1) & 1, abort_flag, p.status, wait_ns);
                 if (!ok) break;
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-                const uint32_t qa = ta_saddr(q_s + (SPLIT ? 0 : qt) * TA_QTILE);
+                const uint32_t qa = ta_saddr(q_s + (SPLIT ? 0 : qt) * QTILE);
 #pragma unroll
-                for (int kk = 0; kk < TA_D / 16; ++kk) {       // 8 steps over the head dimension
+                for (int kk = 0; kk < DK / 16; ++kk) {         // steps over the key's dimensions
                     const uint32_t inner = (kk & 3) * 32;
                     ta_mma(tmem_s + qt * 128 + (j & 1) * TA_BN, ta_desc_k(qa + (kk >> 2) * TA_QSLAB + inner),
                            ta_desc_k(ks + (kk >> 2) * TA_KSLAB + inner), idesc_qk, kk != 0);
@@ -349,14 +376,14 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         if (!ok) for (int i = 0; i < 2 * TA_NQ; ++i) ta_commit(ta_saddr(&s_full[i]));
     } else if (warp == TA_PV_WARP) {
         if (lane == 0) {
-            // ---- issuer of O += P V: N = 128 dims, B (= V) MN-major ----
-            const uint32_t idesc_pv = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 16) | ((uint32_t)(TA_D >> 3) << 17) | ((uint32_t)(128 >> 4) << 24);
+            // ---- issuer of O += P V: N = the value's dimensions, B (= V) MN-major ----
+            const uint32_t idesc_pv = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 16) | ((uint32_t)(DV >> 3) << 17) | ((uint32_t)(128 >> 4) << 24);
             bool ok = true;
             for (int it = 0; ok && it < n_tiles; ++it) {
                 const int s = it % STAGES;
                 // the tile's copies have landed (the other issuer saw it long ago; this thread must see it too)
                 ok = ta_wait(ta_saddr(&kv_full[s]), (it / STAGES) & 1, abort_flag, p.status, wait_ns);
-                const uint32_t vs = ta_saddr(kv_s + s * 2 * TA_KTILE + TA_KTILE);
+                const uint32_t vs = ta_saddr(kv_s + s * STAGE + KTILE);
 #pragma unroll
                 for (int qt = 0; qt < TA_NQ; ++qt) {
                     int j;
@@ -449,7 +476,7 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
                 if (__any_sync(0xffffffffu, alpha != 1.f)) {
 #pragma unroll 1
-                    for (int c0 = 0; c0 < TA_D; c0 += 32) {
+                    for (int c0 = 0; c0 < DV; c0 += 32) {
                         uint32_t v[32];
                         ta_ld32(my_o + lane_base + c0, v);
                         asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
@@ -471,12 +498,11 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             // zero them.  The tile has landed (S was computed from it).  Both query tiles do it (the same zeros),
             // each before its own P V is allowed to start.
             if (r < TA_BN && (t0 + r < lo || t0 + r >= hi)) {
-                unsigned char* vrow = kv_s + (it % STAGES) * 2 * TA_KTILE + TA_KTILE + r * 128;
+                unsigned char* vrow = kv_s + (it % STAGES) * STAGE + KTILE + r * 128;
 #pragma unroll
-                for (int c = 0; c < 8; ++c) {
-                    *reinterpret_cast<uint4*>(vrow + c * 16) = make_uint4(0, 0, 0, 0);
-                    *reinterpret_cast<uint4*>(vrow + TA_KSLAB + c * 16) = make_uint4(0, 0, 0, 0);
-                }
+                for (int sl = 0; sl < VS; ++sl)
+#pragma unroll
+                    for (int c = 0; c < 8; ++c) *reinterpret_cast<uint4*>(vrow + sl * TA_KSLAB + c * 16) = make_uint4(0, 0, 0, 0);
             }
             // P and V (generic-proxy stores) must be visible to the tensor core's reads of shared memory
             asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
@@ -497,7 +523,7 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             // threads have met: the ring is free, and takes the second group's O (float, [dim][row], so that
             // a warp's rows are neighbours) with its maxima and sums behind it.
             float* o_x = reinterpret_cast<float*>(kv_s);
-            float* m_x = o_x + TA_D * TA_BM;
+            float* m_x = o_x + DV * TA_BM;
             float* l_x = m_x + TA_BM;
             const bool has_other = (n_both >> 1) > 0;           // the second group had a key tile at all
             asm volatile("bar.sync 1, 256;" ::: "memory");
@@ -506,7 +532,7 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 m_x[r] = m_run == -INFINITY ? -INFINITY : m_run * scale_log2;
                 l_x[r] = l_run;
 #pragma unroll 1
-                for (int c0 = 0; c0 < TA_D; c0 += 32) {
+                for (int c0 = 0; c0 < DV; c0 += 32) {
                     uint32_t v[32];
                     ta_ld32(my_o + lane_base + c0, v);
                     asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
@@ -532,9 +558,11 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             }
         }
         if (writes) {
-            __nv_bfloat16* orow = static_cast<__nv_bfloat16*>(p.out) + ((size_t)(tok0 + (SPLIT ? 0 : qt * TA_BM) + r) * p.n_q + h) * TA_D;
+            const size_t tok = tok0 + (SPLIT ? 0 : qt * TA_BM) + r;
+            __nv_bfloat16* orow = static_cast<__nv_bfloat16*>(p.out) + (tok * p.n_q + h) * DV;
+            const __nv_bfloat16* grow = DENSE && p.gate != nullptr && r < nq[qt] ? p.gate + tok * p.gate_ld + h * DV : nullptr;
 #pragma unroll 1
-            for (int c0 = 0; c0 < TA_D; c0 += 32) {
+            for (int c0 = 0; c0 < DV; c0 += 32) {
                 uint32_t v[32];
                 ta_ld32(my_o + lane_base + c0, v);
                 asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
@@ -547,6 +575,19 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                     for (int c = 0; c < 32; ++c) v[c] = __float_as_uint(__uint_as_float(v[c]) * w_own);
                 }
                 if (r < nq[qt]) {
+                    if (DENSE && grow != nullptr) {            // the heads' output gate
+#pragma unroll
+                        for (int c = 0; c < 32; c += 8) {
+                            const uint4 g4 = *reinterpret_cast<const uint4*>(grow + c0 + c);
+                            const __nv_bfloat162* g2 = reinterpret_cast<const __nv_bfloat162*>(&g4);
+#pragma unroll
+                            for (int e = 0; e < 4; ++e) {
+                                const float2 z = __bfloat1622float2(g2[e]);
+                                v[c + 2 * e] = __float_as_uint(__fdividef(__uint_as_float(v[c + 2 * e]), 1.f + __expf(-z.x)));
+                                v[c + 2 * e + 1] = __float_as_uint(__fdividef(__uint_as_float(v[c + 2 * e + 1]), 1.f + __expf(-z.y)));
+                            }
+                        }
+                    }
 #pragma unroll
                     for (int c = 0; c < 32; c += 8) {
                         uint32_t w[4];
@@ -625,6 +666,32 @@ static int ta_sm_count() {
     return n;
 }
 
+template <int KS, int VS, bool DENSE>
+static int ta_launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const CUtensorMap& mr, const AttnParams& p,
+                     int n_rows, int max_q_len, cudaStream_t stream) {
+    constexpr int smem_two = ta_smem(KS, VS, false), smem_split = ta_smem(KS, VS, true);
+    static bool configured = false;
+    if (!configured) {
+        cudaError_t e = cudaFuncSetAttribute(attn_prefill_tcgen05_kernel<KS, VS, false, DENSE>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem_two);
+        if (e == cudaSuccess)
+            e = cudaFuncSetAttribute(attn_prefill_tcgen05_kernel<KS, VS, true, DENSE>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem_split);
+        if (e != cudaSuccess) return fail(-3, "attention: cannot get %d bytes of shared memory: %s", smem_two, cudaGetErrorString(e));
+        configured = true;
+    }
+    // Two query tiles per CTA share every key tile; while that leaves SMs without a CTA, one query tile per
+    // CTA with its key tiles dealt to the two softmax groups finishes sooner.
+    const int shared_ctas = ((max_q_len + TA_ROWS - 1) / TA_ROWS) * p.n_q * n_rows;
+    const bool split = g_ta_form == 2 || (g_ta_form == 0 && shared_ctas < ta_sm_count());
+    if (split) {
+        dim3 grid(p.n_q, (max_q_len + TA_BM - 1) / TA_BM, n_rows);
+        attn_prefill_tcgen05_kernel<KS, VS, true, DENSE><<<grid, TA_THREADS, smem_split, stream>>>(mq, mk, mv, mr, p, g_tc_wait_ns, g_tc_skip_last);
+    } else {
+        dim3 grid(p.n_q, (max_q_len + TA_ROWS - 1) / TA_ROWS, n_rows);
+        attn_prefill_tcgen05_kernel<KS, VS, false, DENSE><<<grid, TA_THREADS, smem_two, stream>>>(mq, mk, mv, mr, p, g_tc_wait_ns, g_tc_skip_last);
+    }
+    return check_launch("attention_prefill_tcgen05");
+}
+
 // Returns 1 when it does not take the sizes (the caller falls back to the mma.sync kernel):
 // head size 128, block size a multiple of 8 that divides 128, no split of the keys.
 int launch_attn_prefill_tcgen05(const AttnParams& p, int n_rows, int T, int max_q_len, cudaStream_t stream) {
@@ -638,29 +705,50 @@ int launch_attn_prefill_tcgen05(const AttnParams& p, int n_rows, int T, int max_
     const int box = bs < TA_BN ? bs : TA_BN;
     if (ta_map(p.k_pool, pool_rows, TA_D, box, &mk) != 0) return 1;
     if (ta_map(p.v_pool, pool_rows, TA_D, box, &mv) != 0) return 1;
-    static bool configured = false;
-    if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(attn_prefill_tcgen05_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, TA_SMEM);
-        if (e == cudaSuccess)
-            e = cudaFuncSetAttribute(attn_prefill_tcgen05_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, TA_SMEM);
-        if (e != cudaSuccess) return fail(-3, "attention: cannot get %d bytes of shared memory: %s", TA_SMEM, cudaGetErrorString(e));
-        configured = true;
-    }
-    // Two query tiles per CTA share every key tile; while that leaves SMs without a CTA, one query tile per
-    // CTA with its key tiles dealt to the two softmax groups finishes sooner.
-    const int shared_ctas = ((max_q_len + TA_ROWS - 1) / TA_ROWS) * p.n_q * n_rows;
-    const bool split = g_ta_form == 2 || (g_ta_form == 0 && shared_ctas < ta_sm_count());
-    if (split) {
-        dim3 grid(p.n_q, (max_q_len + TA_BM - 1) / TA_BM, n_rows);
-        attn_prefill_tcgen05_kernel<true><<<grid, TA_THREADS, TA_SMEM, stream>>>(mq, mk, mv, p, g_tc_wait_ns, g_tc_skip_last);
-    } else {
-        dim3 grid(p.n_q, (max_q_len + TA_ROWS - 1) / TA_ROWS, n_rows);
-        attn_prefill_tcgen05_kernel<false><<<grid, TA_THREADS, TA_SMEM, stream>>>(mq, mk, mv, p, g_tc_wait_ns, g_tc_skip_last);
-    }
-    return check_launch("attention_prefill_tcgen05");
+    return ta_launch<2, 2, false>(mq, mk, mv, mk, p, n_rows, max_q_len, stream);
+}
+
+// Whole prompts with keys and values as plain rows (DENSE above).  kv [T, n_q * (64 kn + dv)], rot [T, d - 64 kn] (null when
+// d = 64 kn), q [T, n_q * d]; d 64, 128 or 192, dv 64 or 128.  Returns 1 when it does not take the sizes.
+int launch_attn_prefill_dense(const AttnParams& p, const void* kv, const void* rot, int n_rows, int T, int max_q_len, cudaStream_t stream) {
+    const int ks = p.d / 64, vs = p.dv / 64, kn = p.dense_kn;
+    if (p.d % 64 || p.dv % 64 || ks < 1 || ks > 3 || vs < 1 || vs > 2 || kn < 1 || kn > ks || (kn < ks && rot == nullptr)) return 1;
+    if (ks == 1 && vs == 2) return 1;
+    if ((max_q_len + TA_BM - 1) / TA_BM > 65535 || n_rows > 65535) return 1;
+    CUtensorMap mq, mk, mr;
+    if (ta_map(p.q, T, p.n_q * p.d, TA_BM, &mq) != 0) return 1;
+    if (ta_map(kv, T, p.n_q * (64 * kn + p.dv), TA_BN, &mk) != 0) return 1;
+    mr = mk;
+    if (kn < ks && ta_map(rot, T, p.d - 64 * kn, TA_BN, &mr) != 0) return 1;
+    if (ks == 1) return ta_launch<1, 1, true>(mq, mk, mk, mr, p, n_rows, max_q_len, stream);
+    if (ks == 2) return vs == 1 ? ta_launch<2, 1, true>(mq, mk, mk, mr, p, n_rows, max_q_len, stream)
+                                : ta_launch<2, 2, true>(mq, mk, mk, mr, p, n_rows, max_q_len, stream);
+    return vs == 1 ? ta_launch<3, 1, true>(mq, mk, mk, mr, p, n_rows, max_q_len, stream)
+                   : ta_launch<3, 2, true>(mq, mk, mk, mr, p, n_rows, max_q_len, stream);
 }
 
 }  // namespace fd
+
+// Causal attention of whole prompts over plain rows of keys and values (no cache): q [T, n_q * (64 kn + dr)], kv
+// [T, n_q * (64 kn + dv)] (a head's key dimensions, then its value), rot [T, dr] a key part shared by the heads (dr 0: none);
+// 64 kn + dr 64, 128 or 192; dv 64 or 128.  sink [n_q] or null; gate (rows of gate_ld elements, n_q * dv of them) or null:
+// the heads are multiplied by sigmoid(gate).  Rows of slot -1 are left out.
+extern "C" int fd_attention_dense(const void* q, const void* kv, const void* rot, void* out, const int* row_slot,
+                                  const int* row_q_start, const int* row_q_len, const int* row_ctx_len, int n_rows, int T,
+                                  int max_q_len, int n_q, int kn, int dr, int dv, float scale, int window, const float* sink,
+                                  const void* gate, int gate_ld, int* status, cudaStream_t stream) {
+    if (n_rows == 0 || T == 0) return 0;
+    auto al = [](const void* x) { return (uintptr_t)x % 16 == 0; };
+    FD_REQUIRE(al(q) && al(kv) && al(rot) && al(out) && al(gate) && gate_ld % 8 == 0, -2, "attention_dense: 16-byte alignment");
+    fd::AttnParams p = {};
+    p.q = q; p.out = out; p.row_slot = row_slot; p.row_q_start = row_q_start; p.row_q_len = row_q_len; p.row_ctx_len = row_ctx_len;
+    p.status = status; p.n_q = n_q; p.n_kv = n_q; p.G = 1; p.d = 64 * kn + dr; p.dv = dv; p.v_ld = dv; p.block_size = 64;
+    p.n_kv_pool = n_q; p.kv_div = 1; p.n_splits = 1; p.window = window; p.scale = scale; p.sink = sink; p.v_rep = 1;
+    p.dense_kn = kn; p.gate = static_cast<const __nv_bfloat16*>(gate); p.gate_ld = gate_ld;
+    const int rc = fd::launch_attn_prefill_dense(p, kv, rot, n_rows, T, max_q_len, stream);
+    FD_REQUIRE(rc != 1, -2, "attention_dense: key parts of %d x 64 and %d, values of %d are not taken", kn, dr, dv);
+    return rc;
+}
 
 // 0: the launcher chooses; 1: two query tiles per CTA; 2: one query tile, its key tiles dealt to the two groups
 extern "C" void fd_attn_prefill_set_form(int form) { fd::g_ta_form = form; }

@@ -404,13 +404,14 @@ __global__ void attn_combine_kernel(const float* __restrict__ part_m, const floa
     for (int j = threadIdx.x; j < d; j += blockDim.x) {
         float a = 0.f;
         int s = 0;
+        // (a split that saw no key has weight 0 and may have left its accumulators unwritten)
+        auto part = [&](int i) { return w_s[i] != 0.f ? pa[(size_t)i * d + j] : 0.f; };
         for (; s + 4 <= n_splits; s += 4) {
-            const float a0 = pa[(size_t)(s + 0) * d + j], a1 = pa[(size_t)(s + 1) * d + j];
-            const float a2 = pa[(size_t)(s + 2) * d + j], a3 = pa[(size_t)(s + 3) * d + j];
+            const float a0 = part(s), a1 = part(s + 1), a2 = part(s + 2), a3 = part(s + 3);
             a = fmaf(a0, w_s[s], a); a = fmaf(a1, w_s[s + 1], a);
             a = fmaf(a2, w_s[s + 2], a); a = fmaf(a3, w_s[s + 3], a);
         }
-        for (; s < n_splits; ++s) a = fmaf(pa[(size_t)s * d + j], w_s[s], a);
+        for (; s < n_splits; ++s) a = fmaf(part(s), w_s[s], a);
         if (out_f32) of[j] = a * inv; else o[j] = from_float<T>(a * inv);
     }
 }
@@ -505,8 +506,11 @@ static int attention_impl(const void* q, const void* k_pool, const void* v_pool,
     if (v_ld <= 0) v_ld = dv;
     FD_REQUIRE(v_ld == dv || (v_ld == d && dv <= d && k_pool == v_pool && v_rep == 1), -2,
                "attention: value rows of %d in rows of %d", dv, v_ld);
-    if (v_ld != dv) { use_mma = 0; ext_mma = 0; }     // values inside the keys' rows: the CUDA-core kernel here
-    const bool decode_mma = (use_mma != 0 || (sink_only && ext_mma != 0)) && dtype == 1 && max_q_len == 1 && dv == d;
+    // one cached row per position for all heads, its leading dimensions the values: a tensor-core kernel of its own
+    const bool latent = k_pool == v_pool && n_kv == 1 && dtype == 1 && ext_mma != 0 && v_rep == 1 && !out_f32 && chunk == 0 &&
+                        !(softcap > 0.f) && !(keep_first > 0 && window > 0) && (v_ld != dv || (d != 64 && d != 128));
+    if (v_ld != dv) { use_mma = 0; if (!latent) ext_mma = 0; }
+    const bool decode_mma = !latent && (use_mma != 0 || (sink_only && ext_mma != 0)) && dtype == 1 && max_q_len == 1 && dv == d;
     FD_REQUIRE(n_kv > 0 && n_q % n_kv == 0, -2, "attention: %d query heads are not a multiple of %d KV heads", n_q, n_kv);
     const int G = n_q / n_kv;
     FD_REQUIRE(d % 8 == 0 && d >= 8 && d <= D_MAX, -2, "attention: head size %d must be a multiple of 8 in [8, %d]", d, D_MAX);
@@ -558,7 +562,8 @@ static int attention_impl(const void* q, const void* k_pool, const void* v_pool,
         rc = use_mma == 2 ? 1 : launch_attn_prefill_tcgen05(p, n_rows, T, max_q_len, stream);
         if (rc == 1) rc = launch_attn_prefill_mma(p, n_rows, max_q_len, stream);
     }
-    if (ext && ext_mma && dtype == 1 && max_q_len > 1) {
+    if (latent) rc = launch_attn_latent_mma(p, tok_row, T, stream);
+    else if (ext && ext_mma && dtype == 1 && max_q_len > 1) {
         // of the options the tcgen05 prompt kernel has the keyless term too (head size 128)
         if (sink_only && dv == d) rc = launch_attn_prefill_tcgen05(p, n_rows, T, max_q_len, stream);
         if (rc == 1) rc = launch_attn_prefill_mma_ext(p, n_rows, max_q_len, stream);

@@ -96,6 +96,7 @@ def _declare(L: ctypes.CDLL) -> None:
         "fd_attention_simt": [P, P, P, P, I, P, I, I, I, P, P, P, P, P, I, I, I, I, I, I, F, I, I, I, I, I, P, P, P],
         "fd_attention": [P, P, P, P, I, P, I, I, I, P, P, P, P, P, I, I, I, I, I, I, F, I, I, I, I, I, P, P, P, P, c_ulonglong, P],
         "fd_attention_mma_sync": [P, P, P, P, I, P, I, I, I, P, P, P, P, P, I, I, I, I, I, I, F, I, I, I, I, I, P, P, P, P],
+        "fd_attention_dense": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, F, I, P, P, I, P, P],
         "fd_conv_rope_append": [P, I, I, P, P, P, P, P, I, I, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, P, I, P, P, F, I, I, P],
         "fd_attention_ext": [P, P, P, P, I, P, I, I, I, P, P, P, P, P, I, I, I, I, I, I, F, I, I, I, I, I, P, P, F, I, P, I, I, I, P, I, P],
         "fd_attn_head_mix": [P, P, P, I, I, I, I, I, I, F, P],
@@ -824,6 +825,38 @@ def attention_ext(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, o
         split_len, _ptr(scratch), _ptr(status), float(softcap), int(keep_first), _ptr(sink), v_rep,
         int(out.dtype == torch.float32 and q.dtype != torch.float32 or all_value_heads), int(tensor_cores),
         _ptr(_counters(q.device, n_rows * n_q)) if fused else None, k_pool.shape[-1] if value_dim else 0, _stream()))
+
+
+def attention_dense_takes(key_size: int, rot_size: int, v_size: int) -> bool:
+    """Whether ``attention_dense`` takes heads with so many key dimensions of their own, shared ones, and value dimensions."""
+    k = key_size + rot_size
+    return (key_size % 64 == 0 and rot_size % 64 == 0 and key_size > 0 and k in (64, 128, 192) and v_size in (64, 128)
+            and not (k == 64 and v_size == 128))
+
+
+def attention_dense(q: torch.Tensor, kv: torch.Tensor, rot: Optional[torch.Tensor], out: torch.Tensor, row_slot: torch.Tensor,
+                    row_q_start: torch.Tensor, row_q_len: torch.Tensor, row_ctx_len: torch.Tensor, n_rows: int, max_q_len: int,
+                    n_q: int, key_size: int, v_size: int, scale: float, window: int = 0, sink: Optional[torch.Tensor] = None,
+                    gate: Optional[torch.Tensor] = None, gate_col: int = 0, status: Optional[torch.Tensor] = None) -> None:
+    """Causal attention of whole prompts (every row of the step starts at position 0) over plain rows of keys and values, on
+    the tcgen05 tensor cores (bfloat16).  ``kv`` [T, n_q * (key_size + v_size)]: every head's own key dimensions, then its
+    value; ``rot`` [T, dr]: a key part shared by the heads, or None; ``q`` [T, n_q * (key_size + dr)]; ``out``
+    [T, n_q * v_size].  ``sink`` [n_q] float32: a keyless term per head; ``gate``: the heads are multiplied by sigmoid of its
+    columns from ``gate_col`` on."""
+    T = q.shape[0]
+    dr = 0 if rot is None else rot.shape[1]
+    assert attention_dense_takes(key_size, dr, v_size)
+    assert q.dtype == kv.dtype == out.dtype == torch.bfloat16 and (rot is None or (rot.dtype == q.dtype and rot.shape[0] == T))
+    assert q.shape == (T, n_q * (key_size + dr)) and kv.shape == (T, n_q * (key_size + v_size)) and out.shape == (T, n_q * v_size)
+    assert sink is None or (sink.dtype == torch.float32 and sink.numel() == n_q)
+    assert gate is None or (gate.dtype == q.dtype and gate.shape[0] == T and gate_col + n_q * v_size <= gate.shape[1])
+    _check(lib().fd_attention_dense(_ptr(q), _ptr(kv), _ptr(rot), _ptr(out), _ptr(row_slot), _ptr(row_q_start), _ptr(row_q_len),
+                                    _ptr(row_ctx_len), n_rows, T, max_q_len, n_q, key_size // 64, dr, v_size, float(scale),
+                                    int(window), _ptr(sink), _col_ptr(gate, gate_col) if gate is not None else None,
+                                    gate.shape[1] if gate is not None else 0, _ptr(status), _stream()))
+
+
+LATENT_HEADS = (16, 32)         # query heads a CTA of the latent attention kernel takes: up to 16, else 32
 
 
 def _col_ptr(t: torch.Tensor, first_col: int) -> int:

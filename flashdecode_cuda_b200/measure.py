@@ -22,7 +22,7 @@ LAUNCHERS = ["embed", "add_rmsnorm", "silu_mul", "rope_append", "gemv_qkv_rope",
              "conv_state_update", "gate_mul", "add_concat", "relu2", "moe_route", "moe_align", "moe_gemm", "moe_combine",
              "moe_gather", "gemm_tc_grouped", "glu_mul", "softcap", "lanes_norm", "lanes_fill", "norm_append", "head_gemm",
              "attention_ext", "attn_head_mix", "add_dyn_tanh", "quad_exp_act", "scale_", "axpy_f32", "linear_scan",
-             "head_norm_gate", "add_cast", "side_gate_mul", "token_side_row", "add_row_vector", "low_rank_expand"]
+             "head_norm_gate", "row_norm_gate", "rope_heads", "post_norm", "stream_conv", "attention_dense", "add_cast", "side_gate_mul", "token_side_row", "add_row_vector", "low_rank_expand"]
 
 
 class PartTimer:
@@ -70,6 +70,8 @@ class PartTimer:
         for op in m.stream_ops.values():
             self._wrap_part(op, "stream_op")
         for b in m.blocks:
+            if getattr(b, "completes_stream", False):       # a block that brings its sub-layers' outputs into the stream itself
+                self._wrap_part(b, "norm")
             for name in ("norm1", "norm2"):
                 if getattr(b, name, None) is not None:
                     self._wrap_part(getattr(b, name), "norm")
@@ -154,7 +156,7 @@ def part_work(part, ctx_lens: Sequence[int], q_lens: Sequence[int], real_choice_
         flops, byt = _conv_attention_inner(part, ctx_lens, q_lens, el)
         n_q, dv = part.n_q, part.dv
         return float(flops + 2 * T * H * part.w_in.shape[0] + 2 * T * n_q * dv * H), float(part.weight_bytes() + byt + act)
-    if name in ("Retention", "GatedLinearRecurrence"):
+    if name in ("Retention", "GatedLinearRecurrence", "LightningAttention"):
         flops, byt = _recurrence_inner(part, q_lens)
         nv = part.n_heads * part.dv
         return float(flops + 2 * T * H * part.w_in.shape[0] + 2 * T * nv * H), float(part.weight_bytes() + byt + act)
@@ -197,13 +199,15 @@ def part_work(part, ctx_lens: Sequence[int], q_lens: Sequence[int], real_choice_
     if name == "LatentAttention":
         # the cheaper of attending in the latent's basis (what the part does) and expanding every visible position's
         # keys and values first (what a prompt without a cache could do)
-        n_q, d, dv, r = part.n_q, part.d, part.dv, part.r
+        n_q, d, dv, r, rot, qr = part.n_q, part.d, part.dv, part.r_true, part.rot, part.q_rank
         pairs = visible_pairs(ctx_lens, q_lens, part.window, None)
         n_keys = keys_read(ctx_lens, q_lens, part.window, None)
-        common = 2 * T * H * (n_q * d + r) + 2 * T * n_q * dv * H
-        latent = 2 * T * n_q * r * (d + dv) + 4 * n_q * r * pairs
-        expanded = 2 * n_keys * r * n_q * (d + dv) + 2 * n_q * (d + dv) * pairs
-        return float(common + min(latent, expanded)), float(part.weight_bytes() + n_keys * r * el + act)
+        queries = 2 * T * H * n_q * (d + rot) if qr is None else 2 * T * qr * (H + n_q * (d + rot))
+        gate = 2 * T * H * n_q * dv if part.has_gate else 0
+        common = queries + gate + 2 * T * H * (r + rot) + 2 * T * n_q * dv * H
+        latent = 2 * T * n_q * r * (d + dv) + 2 * n_q * (2 * r + rot) * pairs
+        expanded = 2 * n_keys * r * n_q * (d + dv) + 2 * n_q * (d + rot + dv) * pairs
+        return float(common + min(latent, expanded)), float(part.weight_bytes() + n_keys * (r + rot) * el + act)
     if name in ("SwiGLU", "GatedMLP"):
         return float(2 * T * 3 * H * part.inter), float(part.weight_bytes() + act)
     if name == "RoutedExperts":

@@ -67,6 +67,17 @@ def _pad_cols(w: torch.Tensor, size: int, padded: int) -> torch.Tensor:
     return out
 
 
+def _pad_split_heads(w: torch.Tensor, n_heads: int, *parts) -> torch.Tensor:
+    """w [n_heads * sum of sizes, ...] whose heads have several parts, each (size, padded size): zero rows after each."""
+    out = w.new_zeros((n_heads, sum(p for _, p in parts)) + tuple(w.shape[1:]))
+    rows = w.view((n_heads, sum(s for s, _ in parts)) + tuple(w.shape[1:]))
+    a = b = 0
+    for size, padded in parts:
+        out[:, b:b + size] = rows[:, a:a + size]
+        a, b = a + size, b + padded
+    return out.view((-1,) + tuple(w.shape[1:]))
+
+
 @register_part("mixer", "qk_normed_attention")
 class QKNormedAttention(Mixer):
     """For the mixer's input h [T, hidden]:
@@ -219,11 +230,23 @@ class LatentAttention(Mixer):
         self.rt = rt
         p, n = self.prefix, self.n_q
         pad = lambda w: _pad_heads(w, 1, self.r_true, self.r)            # zero rows up to the padded latent size
-        # Sizes of a head's parts in the activations.
+        # Sizes of a head's parts in the activations: as they are, or, where whole prompts run on the tcgen05 kernel over
+        # plain rows, filled up with zeros to multiples of 64 (zero rows of the projections: no score and no output changes)
         self.dx, self.rx, self.vx = self.d, self.rot, self.dv
+        up64 = lambda size: -(-size // 64) * 64
+        dx, rx, vx = up64(self.d), up64(self.rot), up64(self.dv)
+        if dx + rx == 64 and vx == 128:
+            dx = 128
+        expanded = 3 if K.attention_dense_takes(dx, rx, vx) else 0
+        # which attention kernel the cached row itself reaches (3 tcgen05, 2 mma.sync, 1 mma.sync at wide heads, 0 others)
+        latent = {128: 3, 64: 2, 192: 1, 256: 1}.get(self.r, 0) if not (self.rot or self.has_sink) else 0
+        self.expands = rt.dtype == torch.bfloat16 and (expanded > latent or (expanded == latent > 0 and 2 * self.r > dx + vx))
+        if self.expands:
+            self.dx, self.rx, self.vx = dx, rx, vx
         self.kx = self.dx + self.rx
         w_q = tensors.pop(f"{p}.q" if self.q_rank is None else f"{p}.uq")
         dkv = tensors.pop(f"{p}.dkv")
+        w_q = _pad_split_heads(w_q, n, (self.d, self.dx), (self.rot, self.rx))
         qr = self.qr = 0 if self.q_rank is None else _up8(self.q_rank)
         first = w_q if self.q_rank is None else _pad_heads(tensors.pop(f"{p}.dq"), 1, self.q_rank, qr)
         mats = [first, pad(dkv[:self.r_true]), _pad_heads(dkv[self.r_true:], 1, self.rot, self.rp)]     # [q | latent | k_r | gate]
@@ -241,14 +264,15 @@ class LatentAttention(Mixer):
         uv = _pad_cols(_pad_heads(tensors.pop(f"{p}.uv"), n, self.dv, self.vx), self.r_true, self.r)
         self.w_qc = uk.view(n, self.dx, self.r).transpose(1, 2).contiguous()
         self.w_cv = uv.view(n, self.vx, self.r).contiguous()
-        self.w_o = tensors[f"{p}.o"]
+        w_o = tensors[f"{p}.o"]
+        if self.vx != self.dv:              # zero columns where the filled-up value dimensions arrive
+            w_o = _pad_heads(w_o.t().contiguous(), n, self.dv, self.vx).t().contiguous()
+            tensors[f"{p}.o"] = w_o
+        self.w_o = w_o
         self.sink = tensors[f"{p}.sink"].float().contiguous() if self.has_sink else None
-        # which attention kernel each order reaches (3 tcgen05, 2 mma.sync, 1 mma.sync at wide heads, 0 CUDA cores)
-        rank = lambda size: {128: 3, 64: 2, 192: 1, 256: 1}.get(size, 0)
-        latent, expanded = rank(self.r), (rank(self.d) if self.d == self.dv else 0)
-        self.expands = rt.dtype == torch.bfloat16 and not (self.rot or self.has_sink or self.has_gate or qr) and \
-            (expanded > latent or (expanded == latent and expanded > 1 and 2 * self.r > self.d + self.dv))
-        self.w_kv = torch.cat([uk, uv], dim=0).contiguous() if self.expands else None      # [heads (d + dv), kv_rank]
+        # [heads (dx + vx), kv_rank]: head by head its key rows, then its value rows
+        self.w_kv = torch.cat([uk.view(n, self.dx, self.r), uv.view(n, self.vx, self.r)], dim=1).reshape(
+            n * (self.dx + self.vx), self.r).contiguous() if self.expands else None
 
     def weight_bytes(self) -> int:
         # (the expansion matrix is a second copy of .uk and .uv in another order: a step reads one of the two)
@@ -278,27 +302,20 @@ class LatentAttention(Mixer):
         first = ws.get("lat_q_in", (T, self.qr or n * self.kx), x.dtype)
         out = ws.get("mixer_out", (T, self.hidden_size), x.dtype)
         if self.expands and ctx.max_q_len > 1 and not any(ctx.h_ctx_len):
-            # whole prompts: expand the step's own keys and values and attend over them
+            # whole prompts: expand the step's own keys and values and attend over them as they lie
             c = ws.get("lat_c", (T, self.r), x.dtype)
-            self._append(ctx, proj, first, lc, k_rows=c)
+            kr = ws.get("lat_kr", (T, self.rx), x.dtype) if self.rot else None
+            self._append(ctx, proj, first, lc, k_rows=c, r_rows=kr)
             q = self._queries(ctx, first)
+            if self.rot:
+                K.rope_heads(q, self.kx, self.dx, q, self.kx, self.dx, self.position.cos, self.position.sin, ctx.tok_pos, n,
+                             self.rot, self.rot, rt.status)
             kv = ws.get("lat_kv", (T, self.w_kv.shape[0]), x.dtype)
             matmul(c, self.w_kv, None, kv, status=rt.status)
-            bs = lc.group.block_size
-            per_row = -(-ctx.max_q_len // bs)
-            n_blocks = ctx.n_rows * per_row
-            k_tmp = ws.get("lat_k_pages", (n_blocks, self.n_q, bs, self.d), x.dtype)
-            v_tmp = ws.get("lat_v_pages", (n_blocks, self.n_q, bs, self.dv), x.dtype)
-            table = ws.get("lat_page_table", (ctx.n_rows, per_row), torch.int32)       # row i owns pages i * per_row ...
-            torch.arange(n_blocks, out=table.view(-1))
-            rows = ws.get("lat_page_rows", (ctx.n_rows,), torch.int32)
-            torch.arange(ctx.n_rows, out=rows)
-            K.norm_append(kv, None, None, None, self.eps, ctx.tok_row, ctx.tok_pos, rows, k_tmp, v_tmp, table, self.n_q,
-                          True, rt.status)
-            av = ws.get("lat_v", (T, self.n_q * self.dv), x.dtype)
-            K.attention(q, k_tmp, v_tmp, av, table, ctx.tok_row, rows, ctx.row_q_start, ctx.row_q_len, ctx.row_ctx_len,
-                        ctx.n_rows, ctx.max_q_len, self.n_q, self.n_q, self.d, self.scale, self.window or 0, 1, 0, None,
-                        rt.status)
+            av = ws.get("lat_v", (T, n * self.vx), x.dtype)
+            K.attention_dense(q, kv, kr, av, ctx.row_slot, ctx.row_q_start, ctx.row_q_len, ctx.row_ctx_len, ctx.n_rows,
+                              ctx.max_q_len, n, self.dx, self.vx, self.scale, self.window or 0, self.sink,
+                              proj if self.has_gate else None, self.gate_col if self.has_gate else 0, rt.status)
             return matmul(av, self.w_o, None, out, target_ctas=4 * rt.sm_count, status=rt.status)
         self._append(ctx, proj, first, lc)
         q = self._queries(ctx, first)
@@ -309,11 +326,18 @@ class LatentAttention(Mixer):
             K.rope_heads(q, self.kx, self.dx, qc, size, self.r, self.position.cos, self.position.sin, ctx.tok_pos, n, self.rot,
                          self.rp, rt.status)
         ac = ws.get("lat_ac", (T, n * self.r), x.dtype)
-        n_splits, split_len, scratch = decode_splits(ctx, n, 1, self.r, x.dtype, rt, size if not self.rot else 0)
+        # the latent kernel: bfloat16 steps except those whose row size a faster kernel takes without these options
+        plain = not self.rot and not self.has_sink
+        tensor_rows = x.dtype == torch.bfloat16 and not (plain and (self.r in (64, 128) or ctx.max_q_len > 1))
+        if tensor_rows:
+            per_cta = K.LATENT_HEADS[n > K.LATENT_HEADS[0]]
+            n_splits, split_len, scratch = decode_splits(ctx, n, -(-n // per_cta), self.r, x.dtype, rt)
+        else:
+            n_splits, split_len, scratch = decode_splits(ctx, n, 1, self.r, x.dtype, rt, size if plain else 0)
         args = (qc, lc.k_pool, lc.k_pool, ac, lc.group.table, ctx.tok_row, ctx.row_slot, ctx.row_q_start, ctx.row_q_len,
                 ctx.row_ctx_len, ctx.n_rows, ctx.max_q_len, n, 1, size, self.scale, self.window or 0, n_splits, split_len,
                 scratch, rt.status)
-        if self.rot or self.has_sink:
+        if tensor_rows or not plain:
             K.attention_ext(*args, sink=self.sink, value_dim=self.r if self.rot else 0)
         else:
             K.attention(*args)

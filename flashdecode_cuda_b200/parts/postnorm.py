@@ -137,6 +137,8 @@ class PostNormBlock(Block):
     feed-forward; a ``norm2`` given all the same declares its tensor and never runs);  then x <- the learned average of
     the embedding output and all layers' results so far (``depth``, optional).  Takes and returns a ``PendingPost``."""
 
+    completes_stream = True
+
     def __init__(self, norm1, mixer, norm2=None, feed_forward=None, input_conv=None, depth=None):
         self.norm1, self.mixer, self.norm2, self.feed_forward = norm1, mixer, norm2, feed_forward
         self.input_conv, self.depth = input_conv, depth
