@@ -75,12 +75,58 @@ head_gemm_kernel(const T* __restrict__ a, const T* __restrict__ w, T* __restrict
     }
 }
 
+// A rotated part of every head: dst[t, h, 0 .. places) = rot(src[t, h, 0 .. nr)), zeros after it; src and dst may be the
+// same memory (places == nr then).  Pointers at the first rotated dimension of the first head.
+template <typename T>
+struct RopePart {
+    const T* src; int s_ld, s_hs;
+    T* dst; int d_ld, d_hs;
+    const float* cos_t; const float* sin_t; int table_len;
+    const int* tok_pos;
+    int heads, nr, places;
+    int* status;
+};
+
+template <typename T>
+__device__ __forceinline__ void rope_token(const RopePart<T>& r, int t) {
+    const int pos = r.tok_pos[t];
+    if (pos < 0 || pos >= r.table_len) {
+        if (threadIdx.x == 0) set_status(r.status, STATUS_BAD_POSITION);
+        return;
+    }
+    const int half = r.nr >> 1, pp = r.places >> 1;
+    const float* c = r.cos_t + (size_t)pos * half;
+    const float* s = r.sin_t + (size_t)pos * half;
+    for (int e = threadIdx.x; e < r.heads * pp; e += blockDim.x) {
+        const int h = e / pp, i = e - h * pp;
+        T a = from_float<T>(0.f), b = a;
+        if (i < half) {
+            const T* x = r.src + (size_t)t * r.s_ld + (size_t)h * r.s_hs + 2 * i;
+            const float u = to_float(x[0]), v = to_float(x[1]);
+            a = from_float<T>(u * c[i] - v * s[i]);
+            b = from_float<T>(v * c[i] + u * s[i]);
+        }
+        T* o = r.dst + (size_t)t * r.d_ld + (size_t)h * r.d_hs + 2 * i;
+        o[0] = a;
+        o[1] = b;
+    }
+}
+
+template <typename T>
+__global__ void rope_heads_kernel(const RopePart<T> r) { rope_token<T>(r, blockIdx.x); }
+
 // Steps of few rows in bfloat16 (K a multiple of 8): a warp per output column (head, n) reads that row of w once in
-// 16-byte pieces and takes it against every row of a; eight warps per CTA.
+// 16-byte pieces and takes it against every row of a; eight warps per CTA.  The CTAs behind those (rope.heads > 0: one per row)
+// turn the heads' rotated parts.
 template <int MAXT>
 __global__ void __launch_bounds__(256)
 head_gemv_kernel(const __nv_bfloat16* __restrict__ a, const __nv_bfloat16* __restrict__ w, __nv_bfloat16* __restrict__ out,
-                 const __nv_bfloat16* __restrict__ gate, const HeadStrides st, int T_rows, int heads, int N, int K) {
+                 const __nv_bfloat16* __restrict__ gate, const HeadStrides st, const RopePart<__nv_bfloat16> rope, int n_product_ctas,
+                 int T_rows, int heads, int N, int K) {
+    if ((int)blockIdx.x >= n_product_ctas) {
+        rope_token<__nv_bfloat16>(rope, blockIdx.x - n_product_ctas);
+        return;
+    }
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int col = blockIdx.x * 8 + warp;
     if (col >= heads * N) return;
@@ -120,61 +166,68 @@ head_gemv_kernel(const __nv_bfloat16* __restrict__ a, const __nv_bfloat16* __res
     }
 }
 
-// dst[t, h, 0 .. places) = rot(src[t, h, 0 .. nr)), zeros after it; src and dst may be the same memory (places == nr then).
-template <typename T>
-__global__ void rope_heads_kernel(const T* src, int s_ld, int s_hs, T* dst, int d_ld, int d_hs,
-                                  const float* __restrict__ cos_t, const float* __restrict__ sin_t, int table_len,
-                                  const int* __restrict__ tok_pos, int heads, int nr, int places, int* status) {
-    const int t = blockIdx.x;
-    const int pos = tok_pos[t];
-    if (pos < 0 || pos >= table_len) {
-        if (threadIdx.x == 0) set_status(status, STATUS_BAD_POSITION);
-        return;
-    }
-    const int half = nr >> 1, pp = places >> 1;
-    const float* c = cos_t + (size_t)pos * half;
-    const float* s = sin_t + (size_t)pos * half;
-    for (int e = threadIdx.x; e < heads * pp; e += blockDim.x) {
-        const int h = e / pp, i = e - h * pp;
-        T a = from_float<T>(0.f), b = a;
-        if (i < half) {
-            const T* x = src + (size_t)t * s_ld + (size_t)h * s_hs + 2 * i;
-            const float u = to_float(x[0]), v = to_float(x[1]);
-            a = from_float<T>(u * c[i] - v * s[i]);
-            b = from_float<T>(v * c[i] + u * s[i]);
-        }
-        T* o = dst + (size_t)t * d_ld + (size_t)h * d_hs + 2 * i;
-        o[0] = a;
-        o[1] = b;
-    }
-}
-
 }  // namespace fd
 
 using namespace fd;
 
+template <typename T>
+static int launch_rope(const RopePart<T>& r, int n_tok, cudaStream_t stream) {
+    const int work = r.heads * r.places / 2;
+    const dim3 block(work >= 256 ? 256 : (work + 31) / 32 * 32);
+    return launch("rope_heads", rope_heads_kernel<T>, dim3(n_tok), block, 0, stream, dim3(1, 1, 1), r);
+}
+
+template <typename T>
+static RopePart<T> rope_part(const void* src, int s_ld, int s_hs, void* dst, int d_ld, int d_hs, const float* cos_t,
+                             const float* sin_t, int table_len, const int* tok_pos, int heads, int nr, int places, int* status) {
+    RopePart<T> r;
+    r.src = static_cast<const T*>(src); r.s_ld = s_ld; r.s_hs = s_hs;
+    r.dst = static_cast<T*>(dst); r.d_ld = d_ld; r.d_hs = d_hs;
+    r.cos_t = cos_t; r.sin_t = sin_t; r.table_len = table_len; r.tok_pos = tok_pos;
+    r.heads = heads; r.nr = nr; r.places = places; r.status = status;
+    return r;
+}
+
 // a: [T, heads, K] with row stride a_ld and head stride a_hs (elements); out likewise; gate (or null): sigmoid(gate) times out.
+// nr > 0: the nr dimensions at a + r_src of every head are turned (cos_t / sin_t [table_len, nr / 2]) into the r_places at
+// out + r_dst, in the same launch where the product is the one for few rows.
 extern "C" int fd_head_gemm(const void* a, int a_ld, int a_hs, const void* w, void* out, int o_ld, int o_hs, const void* gate,
-                            int g_ld, int g_hs, int dtype, int T, int heads, int N, int K, cudaStream_t stream) {
+                            int g_ld, int g_hs, int dtype, int T, int heads, int N, int K, int r_src, int r_dst, int nr,
+                            int r_places, const float* cos_t, const float* sin_t, int table_len, const int* tok_pos, int* status,
+                            cudaStream_t stream) {
     if (T == 0) return 0;
     FD_REQUIRE(heads > 0 && heads <= 65535 && N > 0 && K > 0, -2, "head_gemm: %d heads, N %d, K %d", heads, N, K);
+    FD_REQUIRE(nr >= 0 && nr % 2 == 0 && (nr == 0 || (r_places >= nr && r_places % 2 == 0 && cos_t && sin_t && tok_pos)), -2,
+               "head_gemm: a rotated part of %d dimensions in %d places", nr, r_places);
+    typedef __nv_bfloat16 bf16;
     const HeadStrides st = {a_ld, a_hs, o_ld, o_hs, g_ld, g_hs};
+    const dim3 one(1, 1, 1);
     if (dtype == 1 && T <= 16 && K % 8 == 0 && a_ld % 8 == 0 && a_hs % 8 == 0 && (uintptr_t)a % 16 == 0 && (uintptr_t)w % 16 == 0) {
-        const dim3 g((unsigned)((heads * (long long)N + 7) / 8));
+        const int ctas = (int)((heads * (long long)N + 7) / 8);
+        const RopePart<bf16> rp = rope_part<bf16>((const bf16*)a + r_src, a_ld, a_hs, (bf16*)out + r_dst, o_ld, o_hs, cos_t, sin_t,
+                                                  table_len, tok_pos, heads, nr, r_places, status);
+        const dim3 g((unsigned)(ctas + (nr > 0 ? T : 0)));
         if (T <= 8)
-            return launch("head_gemm", head_gemv_kernel<8>, g, dim3(256), 0, stream, dim3(1, 1, 1), (const __nv_bfloat16*)a,
-                          (const __nv_bfloat16*)w, (__nv_bfloat16*)out, (const __nv_bfloat16*)gate, st, T, heads, N, K);
-        return launch("head_gemm", head_gemv_kernel<16>, g, dim3(256), 0, stream, dim3(1, 1, 1), (const __nv_bfloat16*)a,
-                      (const __nv_bfloat16*)w, (__nv_bfloat16*)out, (const __nv_bfloat16*)gate, st, T, heads, N, K);
+            return launch("head_gemm", head_gemv_kernel<8>, g, dim3(256), 0, stream, one, (const bf16*)a, (const bf16*)w, (bf16*)out,
+                          (const bf16*)gate, st, rp, ctas, T, heads, N, K);
+        return launch("head_gemm", head_gemv_kernel<16>, g, dim3(256), 0, stream, one, (const bf16*)a, (const bf16*)w, (bf16*)out,
+                      (const bf16*)gate, st, rp, ctas, T, heads, N, K);
     }
     dim3 grid((N + HG_NT - 1) / HG_NT, (T + HG_MT - 1) / HG_MT, heads);
     FD_REQUIRE(grid.y <= 65535, -2, "head_gemm: %d rows are too many", T);
+    int rc;
     if (dtype == 0)
-        return launch("head_gemm", head_gemm_kernel<float>, grid, dim3(HG_THREADS), 0, stream, dim3(1, 1, 1), (const float*)a,
-                      (const float*)w, (float*)out, (const float*)gate, st, T, heads, N, K);
-    return launch("head_gemm", head_gemm_kernel<__nv_bfloat16>, grid, dim3(HG_THREADS), 0, stream, dim3(1, 1, 1),
-                  (const __nv_bfloat16*)a, (const __nv_bfloat16*)w, (__nv_bfloat16*)out, (const __nv_bfloat16*)gate, st, T, heads,
-                  N, K);
+        rc = launch("head_gemm", head_gemm_kernel<float>, grid, dim3(HG_THREADS), 0, stream, one, (const float*)a, (const float*)w,
+                    (float*)out, (const float*)gate, st, T, heads, N, K);
+    else
+        rc = launch("head_gemm", head_gemm_kernel<bf16>, grid, dim3(HG_THREADS), 0, stream, one, (const bf16*)a, (const bf16*)w,
+                    (bf16*)out, (const bf16*)gate, st, T, heads, N, K);
+    if (rc || nr == 0) return rc;
+    if (dtype == 0)
+        return launch_rope(rope_part<float>((const float*)a + r_src, a_ld, a_hs, (float*)out + r_dst, o_ld, o_hs, cos_t, sin_t,
+                                            table_len, tok_pos, heads, nr, r_places, status), T, stream);
+    return launch_rope(rope_part<bf16>((const bf16*)a + r_src, a_ld, a_hs, (bf16*)out + r_dst, o_ld, o_hs, cos_t, sin_t, table_len,
+                                       tok_pos, heads, nr, r_places, status), T, stream);
 }
 
 // src / dst: pointers to the first rotated dimension of the first head; cos_t / sin_t [table_len, nr / 2].
@@ -184,12 +237,9 @@ extern "C" int fd_rope_heads(const void* src, int s_ld, int s_hs, void* dst, int
     if (T == 0 || nr == 0) return 0;
     FD_REQUIRE(heads > 0 && nr > 0 && nr % 2 == 0 && places >= nr && places % 2 == 0, -2, "rope_heads: %d of %d dimensions", nr, places);
     FD_REQUIRE(src != dst || places == nr, -2, "rope_heads: in place there is nothing to fill up");
-    const int work = heads * places / 2;
-    const dim3 block(work >= 256 ? 256 : (work + 31) / 32 * 32);
     if (dtype == 0)
-        return launch("rope_heads", rope_heads_kernel<float>, dim3(T), block, 0, stream, dim3(1, 1, 1), (const float*)src, s_ld,
-                      s_hs, (float*)dst, d_ld, d_hs, cos_t, sin_t, table_len, tok_pos, heads, nr, places, status);
-    return launch("rope_heads", rope_heads_kernel<__nv_bfloat16>, dim3(T), block, 0, stream, dim3(1, 1, 1),
-                  (const __nv_bfloat16*)src, s_ld, s_hs, (__nv_bfloat16*)dst, d_ld, d_hs, cos_t, sin_t, table_len, tok_pos,
-                  heads, nr, places, status);
+        return launch_rope(rope_part<float>(src, s_ld, s_hs, dst, d_ld, d_hs, cos_t, sin_t, table_len, tok_pos, heads, nr, places,
+                                            status), T, stream);
+    return launch_rope(rope_part<__nv_bfloat16>(src, s_ld, s_hs, dst, d_ld, d_hs, cos_t, sin_t, table_len, tok_pos, heads, nr,
+                                                places, status), T, stream);
 }

@@ -120,7 +120,7 @@ def _declare(L: ctypes.CDLL) -> None:
         "fd_lanes_fill": [P, P, I, I, I, P],
         "fd_lanes_sum": [P, I, P, P, P, P, P, I, I, I, P],
         "fd_norm_append": [P, I, P, I, P, P, F, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, P, I, I, P, P, I, I, I, P, I, P, P],
-        "fd_head_gemm": [P, I, I, P, P, I, I, P, I, I, I, I, I, I, I, P],
+        "fd_head_gemm": [P, I, I, P, P, I, I, P, I, I, I, I, I, I, I, I, I, I, I, P, P, I, P, P, P],
         "fd_rope_heads": [P, I, I, P, I, I, I, P, P, I, P, I, I, I, I, P, P],
         "fd_post_norm": [P, I, P, P, I, P, I, F, P, I, P, LL, I, I, P, P, I, P, I, F, P, P, I, P, P, P, I, I, P],
         "fd_stream_conv": [P, P, P, P, I, P, P, P, I, I, I, P],
@@ -368,10 +368,12 @@ HEAD_GEMM_LIBRARY_ROWS = 64      # from this many rows on, the per-head products
 
 
 def head_gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, a_size: int = 0, out_size: int = 0,
-              gate: Optional[torch.Tensor] = None, gate_col: int = 0) -> None:
+              gate: Optional[torch.Tensor] = None, gate_col: int = 0, rope=None) -> None:
     """out[t, h, :N] = w[h] a[t, h, :K]: a [T, heads * a_size], w [heads, N, K], out [T, heads * out_size]; ``a_size`` /
     ``out_size``: the places a head has there (0: K and N; the places behind are neither read nor written).  ``gate``: out is
-    multiplied by sigmoid of its columns ``gate_col + h * N + n``.  Float accumulation.  float32: the library's own CUDA-core
+    multiplied by sigmoid of its columns ``gate_col + h * N + n``.  ``rope`` = (src_off, dst_off, rot, places, cos, sin, tok_pos,
+    status): the ``rot`` dimensions of every head of a behind ``src_off`` go, turned, to out (see ``rope_heads``), in the same
+    launch for steps of up to 16 rows.  Float accumulation.  float32: the library's own CUDA-core
     kernel with k ascending (no bit of a row depends on the step's other rows); bfloat16: a warp per output column for
     steps of up to 16 rows, cuBLAS's strided batched product for prompts (without a gate)."""
     heads, N, Kd = w.shape
@@ -384,10 +386,16 @@ def head_gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, a_size: int =
     if a.dtype == torch.bfloat16 and T >= HEAD_GEMM_LIBRARY_ROWS and gate is None:
         torch.bmm(a.view(T, heads, a_size)[:, :, :Kd].transpose(0, 1), w.transpose(1, 2),
                   out=out.view(T, heads, out_size)[:, :, :N].transpose(0, 1))
+        if rope is not None:
+            src_off, dst_off, rot, places, cos, sin, tok_pos, status = rope
+            rope_heads(a, a_size, src_off, out, out_size, dst_off, cos, sin, tok_pos, heads, rot, places, status)
         return
+    src_off, dst_off, rot, places, cos, sin, tok_pos, status = rope or (0, 0, 0, 0, None, None, None, None)
+    assert src_off + rot <= a_size and dst_off + places <= out_size and (not rot or cos.shape[1] == rot // 2)
     _check(lib().fd_head_gemm(_ptr(a), heads * a_size, a_size, _ptr(w), _ptr(out), heads * out_size, out_size,
                               _col_ptr(gate, gate_col) if gate is not None else None, gate.shape[1] if gate is not None else 0,
-                              N, _dt(a.dtype), T, heads, N, Kd, _stream()))
+                              N, _dt(a.dtype), T, heads, N, Kd, src_off, dst_off, rot, places, _ptr(cos), _ptr(sin),
+                              cos.shape[0] if rot else 0, _ptr(tok_pos), _ptr(status), _stream()))
 
 
 def rope_heads(src: torch.Tensor, src_size: int, src_off: int, dst: torch.Tensor, dst_size: int, dst_off: int,

@@ -321,10 +321,8 @@ class LatentAttention(Mixer):
         q = self._queries(ctx, first)
         size = self.r + self.rp
         qc = ws.get("lat_qc", (T, n * size), x.dtype)
-        K.head_gemm(q, self.w_qc, qc, a_size=self.kx, out_size=size)
-        if self.rot:
-            K.rope_heads(q, self.kx, self.dx, qc, size, self.r, self.position.cos, self.position.sin, ctx.tok_pos, n, self.rot,
-                         self.rp, rt.status)
+        rope = (self.dx, self.r, self.rot, self.rp, self.position.cos, self.position.sin, ctx.tok_pos, rt.status) if self.rot else None
+        K.head_gemm(q, self.w_qc, qc, a_size=self.kx, out_size=size, rope=rope)
         ac = ws.get("lat_ac", (T, n * self.r), x.dtype)
         # the latent kernel: bfloat16 steps except those whose row size a faster kernel takes without these options
         plain = not self.rot and not self.has_sink

@@ -202,12 +202,12 @@ def test_queries_into_the_latents_basis_and_back_behind_the_gate(dtype, T, heads
     q, w = torch.randn(T, heads, d + rot).to(dt), (torch.randn(heads, r, d) / d ** 0.5).to(dt)
     out = torch.full((T, heads * (r + tp)), 7.0, dtype=dt, device=DEV)
     qd = q.reshape(T, -1).to(DEV)
-    K.head_gemm(qd, w.to(DEV), out, a_size=d + rot, out_size=r + tp)
     pos = RotaryScaled(rot, 1000.0, None)
     pos.prepare(512, _Rt)
     tok_pos = torch.randint(0, 400, (T,))
     status = new_status()
-    K.rope_heads(qd, d + rot, d, out, r + tp, r, pos.cos, pos.sin, tok_pos.to(torch.int32).to(DEV), heads, rot, tp, status)
+    K.head_gemm(qd, w.to(DEV), out, a_size=d + rot, out_size=r + tp,
+                rope=(d, r, rot, tp, pos.cos, pos.sin, tok_pos.to(torch.int32).to(DEV), status))
     got = out.view(T, heads, r + tp).double().cpu()
     f, _ = P.rot_frequencies(rot, 1000.0)
     turned = P.rotate_pairs(q[:, :, d:].double(), tok_pos, f, 1.0)
