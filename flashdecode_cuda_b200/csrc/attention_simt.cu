@@ -401,10 +401,26 @@ __global__ void attn_combine_kernel(const float* __restrict__ part_m, const floa
     if (sink != nullptr) l += expf(sk - m);
     const float inv = l > 0.f ? 1.f / l : 0.f;
     const float* pa = part_acc + row * n_splits * d;
+    if ((d & 3) == 0) {
+        // four dims a thread, eight splits' loads in flight; per dim the sums are those of the loop below, in its order
+        for (int j = threadIdx.x * 4; j < d; j += blockDim.x * 4) {
+            float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+            for (int s = 0; s < n_splits; ++s) {
+                const float w = w_s[s];
+                // (a split that saw no key has weight 0 and may have left its accumulators unwritten)
+                const float4 v = w != 0.f ? *reinterpret_cast<const float4*>(pa + (size_t)s * d + j) : make_float4(0.f, 0.f, 0.f, 0.f);
+                a.x = fmaf(v.x, w, a.x); a.y = fmaf(v.y, w, a.y); a.z = fmaf(v.z, w, a.z); a.w = fmaf(v.w, w, a.w);
+            }
+            const float r[4] = {a.x * inv, a.y * inv, a.z * inv, a.w * inv};
+#pragma unroll
+            for (int e = 0; e < 4; ++e) { if (out_f32) of[j + e] = r[e]; else o[j + e] = from_float<T>(r[e]); }
+        }
+        return;
+    }
     for (int j = threadIdx.x; j < d; j += blockDim.x) {
         float a = 0.f;
         int s = 0;
-        // (a split that saw no key has weight 0 and may have left its accumulators unwritten)
         auto part = [&](int i) { return w_s[i] != 0.f ? pa[(size_t)i * d + j] : 0.f; };
         for (; s + 4 <= n_splits; s += 4) {
             const float a0 = part(s), a1 = part(s + 1), a2 = part(s + 2), a3 = part(s + 3);

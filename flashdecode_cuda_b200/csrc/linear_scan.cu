@@ -400,6 +400,7 @@ __global__ void head_norm_gate_kernel(const float* __restrict__ o, const float* 
 
 // A CTA per token: y = o / sqrt(mean(o^2) + eps) * w over ALL n values of the row, times sigmoid(gate).
 constexpr int ROW_GATE_THREADS = 256;
+constexpr int ROW_GATE_CACHED = 16;       // values of a row a thread holds in registers
 template <typename T>
 __global__ void __launch_bounds__(ROW_GATE_THREADS)
 row_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ w, const T* __restrict__ gate, int ldg,
@@ -408,6 +409,33 @@ row_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ w, c
     const size_t t = blockIdx.x;
     const float* x = o + t * n;
     float ss = 0.f;
+    if (n <= ROW_GATE_CACHED * (int)blockDim.x && n % 4 == 0 && ldg % 4 == 0 && ((uintptr_t)gate | (uintptr_t)out | (uintptr_t)x) % 16 == 0) {
+        // the row in registers, four values a piece, gate and weight asked for before the reduction
+        float4 xv[ROW_GATE_CACHED / 4], wv[ROW_GATE_CACHED / 4];
+        float gv[ROW_GATE_CACHED / 4][4];
+#pragma unroll
+        for (int k = 0; k < ROW_GATE_CACHED / 4; ++k) {
+            const int j = (k * blockDim.x + threadIdx.x) * 4;
+            if (j >= n) continue;
+            xv[k] = *reinterpret_cast<const float4*>(x + j);
+            wv[k] = make_float4(w[j], w[j + 1], w[j + 2], w[j + 3]);
+            const T* g = gate + t * ldg + j;
+#pragma unroll
+            for (int e = 0; e < 4; ++e) gv[k][e] = to_float(g[e]);
+            ss = fmaf(xv[k].x, xv[k].x, ss); ss = fmaf(xv[k].y, xv[k].y, ss);
+            ss = fmaf(xv[k].z, xv[k].z, ss); ss = fmaf(xv[k].w, xv[k].w, ss);
+        }
+        const float rs = 1.f / sqrtf(block_sum(ss, red) / (float)n + eps);
+#pragma unroll
+        for (int k = 0; k < ROW_GATE_CACHED / 4; ++k) {
+            const int j = (k * blockDim.x + threadIdx.x) * 4;
+            if (j >= n) continue;
+            const float y[4] = {xv[k].x * rs * wv[k].x, xv[k].y * rs * wv[k].y, xv[k].z * rs * wv[k].z, xv[k].w * rs * wv[k].w};
+#pragma unroll
+            for (int e = 0; e < 4; ++e) out[t * n + j + e] = from_float<T>(y[e] / (1.f + expf(-gv[k][e])));
+        }
+        return;
+    }
     for (int j = threadIdx.x; j < n; j += blockDim.x) ss = fmaf(x[j], x[j], ss);
     const float rs = 1.f / sqrtf(block_sum(ss, red) / (float)n + eps);
     for (int j = threadIdx.x; j < n; j += blockDim.x) {
