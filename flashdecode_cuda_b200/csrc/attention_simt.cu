@@ -1,6 +1,7 @@
 // Causal grouped-query attention over the paged KV cache on the CUDA cores,
-// for any head size that is a multiple of 8 (up to 256; values may have a
-// size of their own), any group size up to 64, any block size, an optional
+// for any head size that is a multiple of 8 (keys up to 640, values up to 512 and
+// of a size of their own, or the leading columns of the keys' rows), any group
+// size, any block size, an optional
 // sliding window or chunked visibility (keys of the query's own chunk of
 // `chunk` positions only, chunks counted from the start of the sequence),
 // float or bfloat16 storage.  Options that only this kernel has: scores capped by a

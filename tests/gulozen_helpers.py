@@ -51,7 +51,7 @@ GULOZEN: Dict[str, dict] = {
     "A": model(211, 96, 1e-6, [
         latent(6, 24, 8, 40, 40, 48, 0.25, 500.0, (8.0, 64, 4.0, 1.0), moe(6, 2, 40)),
         lightning(3, 24, 40, mlp=moe(5, 3, 24)),
-        latent(2, 64, 16, 64, 56, 72, 0.12, 20000.0, (4.0, 512, 32.0, 1.0), moe(7, 4, 16)),
+        latent(2, 64, 16, 64, 56, 72, 0.12, 30000.0, (5.0, 512, 16.0, 1.0), moe(7, 4, 16)),
     ], groups=3, taps=3, emb_scale=30.0),
     # one norm group, one tap (no convolution state), scale left out, plain frequencies, one head, rotated part of two
     # dimensions, every expert chosen, one choice; layers without a feed-forward; lightning heads of one size and one head

@@ -118,7 +118,7 @@ def test_head_parts_are_filled_up_apart():
 
 
 @pytest.mark.parametrize("dims,base,scaling", [(16, 10000.0, None), (48, 1e6, (8.0, 1024, 32.0, 1.0)), (8, 100.0, (4.0, 64, 8.0, 2.0)),
-                                               (64, 20000.0, (4.0, 2048, 32.0, 1.0)), (2, 50.0, (2.0, 64, 1.0, 1.0))])
+                                               (64, 30000.0, (6.0, 4096, 24.0, 1.5)), (2, 50.0, (2.0, 64, 1.0, 1.0))])
 def test_rotation_tables_follow_the_stretched_frequencies(dims, base, scaling):
     sc = None if scaling is None else dict(zip(("factor", "original", "fast", "slow"), scaling))
     f, mag = P.rot_frequencies(dims, base, sc)

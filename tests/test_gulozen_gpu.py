@@ -714,7 +714,7 @@ def test_long_prompts_at_sizes_of_the_tensor_core_kernels(tmp_path, dtype):
     prompts of several hundred tokens: many segments of the recurrence, many key tiles; each prompt alone, then the two
     together and decoded on."""
     cfg = GH.model(333, 256, 1e-5, [
-        GH.latent(2, 128, 64, 128, 96, 128, 0.06, 20000.0, (4.0, 256, 32.0, 1.0), GH.moe(8, 2, 128)),
+        GH.latent(2, 128, 64, 128, 96, 128, 0.06, 40000.0, (4.0, 256, 32.0, 1.0), GH.moe(8, 2, 128)),
         GH.lightning(2, 64, 64, [0.9, 0.995]),
         GH.latent(18, 64, 64, 64, 64, 192, 0.09, 10000.0, None, GH.moe(4, 3, 128)),
         GH.lightning(1, 128, 128, [0.98], GH.moe(6, 2, 256))], groups=4, taps=4, emb_scale=20.0)
