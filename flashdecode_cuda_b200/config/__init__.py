@@ -12,6 +12,7 @@ from pathlib import Path
 from typing import Any, Dict, List, Union
 
 from ..registry import architecture
+from .bifatar import BifatarConfig
 from .botusun import BotusunConfig
 from .gulozen import GulozenConfig
 from .lonasun import LonasunConfig
@@ -64,4 +65,4 @@ def load_config(source: Union[str, Path, Dict[str, Any]]):
     raise ConfigError(f"no config.json at {source!r} and no preset of that name; presets: {preset_names()}")
 
 
-__all__ = ["ConfigError", "Qwen2Config", "BotusunConfig", "GulozenConfig", "LonasunConfig", "NizazenConfig", "RevelixConfig", "load_config", "config_from_dict", "preset_dict", "preset_names"]
+__all__ = ["ConfigError", "Qwen2Config", "BifatarConfig", "BotusunConfig", "GulozenConfig", "LonasunConfig", "NizazenConfig", "RevelixConfig", "load_config", "config_from_dict", "preset_dict", "preset_names"]

@@ -9,7 +9,9 @@ struct AttnParams {
     const void* q;             // [T, n_q * d]
     const void* k_pool;        // [num_blocks, n_kv, block_size, d]
     const void* v_pool;        // [num_blocks, n_kv, block_size, dv]
-    void* out;                 // [T, n_q * dv]
+    void* out;                 // [T, n_q * dv], rows of out_ld elements, every value times out_scale (in float)
+    int out_ld;
+    float out_scale;
     float* part_m;             // [T, n_q, n_splits]
     float* part_l;
     float* part_acc;           // [T, n_q, n_splits, dv]

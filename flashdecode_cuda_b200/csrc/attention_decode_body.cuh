@@ -30,6 +30,12 @@ __device__ __forceinline__ float dm_ex2(float x) {
     return y;
 }
 
+// cap * tanh(x) in units of log2(e), x = score * scale / cap, from the raw score: cap (1 - 2 / (e^(2x) + 1)), whose error
+// stays below 1e-6 of the cap
+__device__ __forceinline__ float dm_cap(float s, float cap_in, float cap_out) {
+    return fmaf(-2.f * cap_out, __fdividef(1.f, exp2f(fminf(s * cap_in, 120.f)) + 1.f), cap_out);
+}
+
 // transpose of an 8 x 8 tile of 16-bit values held across the warp in the fragment layout of mma
 __device__ __forceinline__ uint32_t movmatrix_trans(uint32_t a) {
     uint32_t d;
@@ -60,7 +66,7 @@ __device__ __forceinline__ void attn_decode_item(const AttnParams& p, const int 
         // padding row: zeros, written here when no merge kernel follows
         if (p.counters != nullptr && split == 0)
             for (int e = tid; e < G * D; e += DM_THREADS)
-                static_cast<__nv_bfloat16*>(p.out)[((size_t)tok * p.n_q + kvh * G) * D + e] = __float2bfloat16_rn(0.f);
+                static_cast<__nv_bfloat16*>(p.out)[(size_t)tok * p.out_ld + kvh * G * D + e] = __float2bfloat16_rn(0.f);
         return;
     }
     const int ctx = p.row_ctx_len[b];
@@ -104,7 +110,10 @@ __device__ __forceinline__ void attn_decode_item(const AttnParams& p, const int 
     for (int i = 0; i < NO; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
     float m_run[2] = {-INFINITY, -INFINITY};   // heads lane/4 and lane/4 + 8; TR: heads 2 (lane%4) and + 1
     float l_run[2] = {0.f, 0.f};               // per-thread partial sums (its share of each tile's keys)
-    const float scale_log2 = p.scale * 1.4426950408889634f;
+    // capped scores: the maxima are then kept of score * log2(e) after the cap instead of raw scores (a factor of 1 from there on)
+    const bool capped = p.softcap > 0.f;
+    const float scale_log2 = capped ? 1.f : p.scale * 1.4426950408889634f;
+    const float cap_in = capped ? 2.f * 1.4426950408889634f * p.scale / p.softcap : 0.f, cap_out = p.softcap * 1.4426950408889634f;
 
     unsigned char* my = kv_s + warp * WARP_BYTES;
     const int bs = p.block_size;
@@ -258,6 +267,10 @@ __device__ __forceinline__ void attn_decode_item(const AttnParams& p, const int 
             }
 #pragma unroll
             for (int e = 0; e < 4; ++e) s[e] += s2[e];
+            if (capped) {
+#pragma unroll
+                for (int e = 0; e < 4; ++e) s[e] = dm_cap(s[e], cap_in, cap_out);
+            }
             // mask (only a split's first and last tile can hold keys outside [lo, hi)) and online softmax, base 2,
             // the maximum kept in units of the raw scores (scale > 0)
             if (t0 < lo || t0 + DM_TILE > hi) {
@@ -303,6 +316,12 @@ __device__ __forceinline__ void attn_decode_item(const AttnParams& p, const int 
                 ldmatrix_x4(ks32 + k_off[kk], b0, b1, b2, b3);
                 mma_bf16(s[0], qf[kk][0], qf[kk][1], qf[kk][2], qf[kk][3], b0, b1);
                 mma_bf16(s[1], qf[kk][0], qf[kk][1], qf[kk][2], qf[kk][3], b2, b3);
+            }
+            if (capped) {
+    #pragma unroll
+                for (int nt = 0; nt < 2; ++nt)
+    #pragma unroll
+                    for (int e = 0; e < 4; ++e) s[nt][e] = dm_cap(s[nt][e], cap_in, cap_out);
             }
             // mask and online softmax (base 2, the maximum kept in units of the raw scores: scale > 0);
             // this thread's keys: t0 + (lane%4)*2 + {0,1} (+8).  Only a split's first and last tile can hold
@@ -426,7 +445,8 @@ __device__ __forceinline__ void attn_decode_item(const AttnParams& p, const int 
         } else {
             // a keyless term exp(sink[h]) joins the denominator (the maxima are raw scores: both in units of log2)
             if (p.sink != nullptr && l > 0.f) l += exp2f(p.sink[kvh * G + r] * 1.4426950408889634f - m * scale_log2);
-            static_cast<__nv_bfloat16*>(p.out)[row * D + j] = __float2bfloat16_rn(l > 0.f ? a / l : 0.f);
+            static_cast<__nv_bfloat16*>(p.out)[(size_t)tok * p.out_ld + (kvh * G + r) * D + j] =
+                __float2bfloat16_rn(l > 0.f ? a / l * p.out_scale : 0.f);
         }
     }
     if (p.n_splits == 1 || p.counters == nullptr) return;
@@ -486,7 +506,7 @@ __device__ __forceinline__ void attn_decode_item(const AttnParams& p, const int 
         }
         lsum = warp_sum(lsum);
         if (p.sink != nullptr && lsum > 0.f) lsum += expf(p.sink[kvh * G + r] - m);       // the keyless term, once per head
-        const float inv = lsum > 0.f ? 1.f / lsum : 0.f;
+        const float inv = lsum > 0.f ? p.out_scale / lsum : 0.f;
         for (int s = lane; s < ns; s += 32) wgt[r * ns + s] *= inv;
     }
     sync();
@@ -517,7 +537,7 @@ __device__ __forceinline__ void attn_decode_item(const AttnParams& p, const int 
         uint2 o2;
         *reinterpret_cast<__nv_bfloat162*>(&o2.x) = __floats2bfloat162_rn(a.x, a.y);
         *reinterpret_cast<__nv_bfloat162*>(&o2.y) = __floats2bfloat162_rn(a.z, a.w);
-        *reinterpret_cast<uint2*>(static_cast<__nv_bfloat16*>(p.out) + row * D + j4 * 4) = o2;
+        *reinterpret_cast<uint2*>(static_cast<__nv_bfloat16*>(p.out) + (size_t)tok * p.out_ld + (kvh * G + r) * D + j4 * 4) = o2;
     }
 }
 

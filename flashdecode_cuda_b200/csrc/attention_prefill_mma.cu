@@ -283,18 +283,18 @@ attn_prefill_mma_kernel(const AttnParams p) {
             f = m == -INFINITY ? 0.f : exp2f(m - m2);
             l = l * f + exp2f(sk - m2);
         }
-        const float inv = l > 0.f ? f / l : 0.f;
+        const float inv = l > 0.f ? f / l * p.out_scale : 0.f;
 #pragma unroll
         for (int j = 0; j < VR; ++j) {
-            const size_t orow_i = EXT ? ((size_t)(tok0 + r) * p.n_q + h) * p.v_rep + vhi + j : (size_t)(tok0 + r) * p.n_q + h;
+            const size_t orow_i = (size_t)(tok0 + r) * p.out_ld + (EXT ? h * p.v_rep + vhi + j : h) * D;
             if (EXT && p.out_f32) {
-                float* orow = static_cast<float*>(p.out) + orow_i * D + (lane & 3) * 2;
+                float* orow = static_cast<float*>(p.out) + orow_i + (lane & 3) * 2;
 #pragma unroll
                 for (int nt = 0; nt < D / 8; ++nt)
                     *reinterpret_cast<float2*>(orow + nt * 8) = make_float2(o[j][nt][hh * 2] * inv, o[j][nt][hh * 2 + 1] * inv);
                 continue;
             }
-            __nv_bfloat16* orow = og + orow_i * D + (lane & 3) * 2;
+            __nv_bfloat16* orow = og + orow_i + (lane & 3) * 2;
 #pragma unroll
             for (int nt = 0; nt < D / 8; ++nt)
                 *reinterpret_cast<__nv_bfloat162*>(orow + nt * 8) =

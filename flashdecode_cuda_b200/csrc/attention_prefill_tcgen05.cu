@@ -414,7 +414,11 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         // chunked visibility: this row's first visible key, and that of the tile's last row
         const int cs_pos = p.chunk > 0 ? (pos / p.chunk) * p.chunk : 0;
         const int cs_last = p.chunk > 0 ? ((p_first[qt] + TA_BM - 1) / p.chunk) * p.chunk : 0;
-        const float scale_log2 = p.scale * 1.4426950408889634f;   // > 0: the maximum is taken over raw scores
+        // > 0: the maximum is taken over raw scores, or, capped, over score * log2(e) after the cap (a factor of 1 from there on)
+        const bool capped = p.softcap > 0.f;
+        const float scale_log2 = capped ? 1.f : p.scale * 1.4426950408889634f;
+        const float cap_in = capped ? 2.f * 1.4426950408889634f * p.scale / p.softcap : 0.f;
+        const float cap_out = p.softcap * 1.4426950408889634f;
         float m_run = -INFINITY, l_run = 0.f;                      // running maximum (raw score) and sum
         bool ok = true;
         const int n_both = it_hi[qt] - it_lo[qt];
@@ -437,6 +441,11 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             // the scores are in registers: the S buffer may take the key tile after next
             asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
             ta_arrive(ta_saddr(&s_free[qt * 2 + (j & 1)]));
+            if (capped) {            // cap tanh(x) as cap (1 - 2 / (e^(2x) + 1)), in float: its error stays below 1e-6 of the cap
+#pragma unroll
+                for (int c = 0; c < TA_BN; ++c)
+                    x[c] = fmaf(-2.f * cap_out, __fdividef(1.f, ta_ex2(fminf(x[c] * cap_in, 120.f)) + 1.f), cap_out);
+            }
             const bool need_mask = t0 + TA_BN - 1 > p_first[qt] || t0 < my_lo || t0 + TA_BN > my_hi ||
                                    (p.window > 0 && t0 < p_first[qt] + TA_BM - p.window) || t0 < cs_last;
             if (need_mask) {
@@ -514,7 +523,7 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         // a keyless term exp(sink[h]) joins the denominator: relative to the running maximum, like every other term
         const float sink_log2 = p.sink != nullptr ? p.sink[h] * 1.4426950408889634f : 0.f;
         if (!SPLIT && p.sink != nullptr && l_run > 0.f) l_run += ta_ex2(sink_log2 - m_run * scale_log2);
-        float w_own = l_run > 0.f ? 1.f / l_run : 0.f;          // what this thread's O is multiplied by
+        float w_own = l_run > 0.f ? p.out_scale / l_run : 0.f;          // what this thread's O is multiplied by
         float w_other = 0.f;                                    // SPLIT: and the other group's
         const float* o_other = nullptr;
         bool writes = ok && n_mine > 0;
@@ -551,7 +560,7 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 const float a1 = m1 == -INFINITY ? 0.f : ta_ex2(m1 - m);
                 float l = l_run * a0 + l1 * a1;
                 if (p.sink != nullptr && l > 0.f) l += ta_ex2(sink_log2 - m);
-                const float inv = l > 0.f ? 1.f / l : 0.f;
+                const float inv = l > 0.f ? p.out_scale / l : 0.f;
                 w_own = a0 * inv;
                 w_other = a1 * inv;
                 if (has_other) o_other = o_x + r;
@@ -559,7 +568,7 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         }
         if (writes) {
             const size_t tok = tok0 + (SPLIT ? 0 : qt * TA_BM) + r;
-            __nv_bfloat16* orow = static_cast<__nv_bfloat16*>(p.out) + (tok * p.n_q + h) * DV;
+            __nv_bfloat16* orow = static_cast<__nv_bfloat16*>(p.out) + tok * p.out_ld + h * DV;
             const __nv_bfloat16* grow = DENSE && p.gate != nullptr && r < nq[qt] ? p.gate + tok * p.gate_ld + h * DV : nullptr;
 #pragma unroll 1
             for (int c0 = 0; c0 < DV; c0 += 32) {
@@ -744,6 +753,7 @@ extern "C" int fd_attention_dense(const void* q, const void* kv, const void* rot
     p.q = q; p.out = out; p.row_slot = row_slot; p.row_q_start = row_q_start; p.row_q_len = row_q_len; p.row_ctx_len = row_ctx_len;
     p.status = status; p.n_q = n_q; p.n_kv = n_q; p.G = 1; p.d = 64 * kn + dr; p.dv = dv; p.v_ld = dv; p.block_size = 64;
     p.n_kv_pool = n_q; p.kv_div = 1; p.n_splits = 1; p.window = window; p.scale = scale; p.sink = sink; p.v_rep = 1;
+    p.out_ld = n_q * dv; p.out_scale = 1.f;
     p.dense_kn = kn; p.gate = static_cast<const __nv_bfloat16*>(gate); p.gate_ld = gate_ld;
     const int rc = fd::launch_attn_prefill_dense(p, kv, rot, n_rows, T, max_q_len, stream);
     FD_REQUIRE(rc != 1, -2, "attention_dense: key parts of %d x 64 and %d, values of %d are not taken", kn, dr, dv);

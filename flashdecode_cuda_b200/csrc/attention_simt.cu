@@ -337,12 +337,13 @@ attn_tile_kernel(const AttnParams p) {
                 f = m == -INFINITY ? 0.f : expf(m - m2);
                 l = l * f + expf(sk - m2);
             }
-            const float inv = l > 0.f ? f / l : 0.f;
+            const float inv = l > 0.f ? f / l * p.out_scale : 0.f;
+            const size_t orow = (size_t)(tok0 + qi) * p.out_ld + (row - (size_t)(tok0 + qi) * p.n_q * p.v_rep) * dv;
             if (p.out_f32) {
-                *reinterpret_cast<float4*>(static_cast<float*>(p.out) + row * dv + dc * 4) =
+                *reinterpret_cast<float4*>(static_cast<float*>(p.out) + orow + dc * 4) =
                     make_float4(acc[i][0] * inv, acc[i][1] * inv, acc[i][2] * inv, acc[i][3] * inv);
             } else {
-                T* o = og + row * dv + dc * 4;
+                T* o = og + orow + dc * 4;
 #pragma unroll
                 for (int j = 0; j < 4; ++j) o[j] = from_float<T>(acc[i][j] * inv);
             }
@@ -362,15 +363,15 @@ __global__ void attn_combine_kernel(const float* __restrict__ part_m, const floa
                                     const float* __restrict__ part_acc, T* __restrict__ out,
                                     const int* __restrict__ tok_row, const int* __restrict__ row_slot,
                                     int n_q, int d, int n_splits, const float* __restrict__ sink, int v_rep,
-                                    int out_f32) {
+                                    int out_f32, int out_ld, float out_scale) {
     __shared__ float w_s[COMBINE_MAX_SPLITS];
     __shared__ float red[33];
     pdl_launch_dependents();
     pdl_wait();
     const int tok = blockIdx.y, h = blockIdx.x;
     const size_t row = (size_t)tok * n_q + h;
-    T* o = out + row * d;
-    float* of = reinterpret_cast<float*>(out) + row * d;       // the same row when the output is float whatever T is
+    T* o = out + (size_t)tok * out_ld + (size_t)h * d;
+    float* of = reinterpret_cast<float*>(out) + (size_t)tok * out_ld + (size_t)h * d;       // the same row when the output is float whatever T is
     if (row_slot[tok_row[tok]] < 0) {
         for (int j = threadIdx.x; j < d; j += blockDim.x) { if (out_f32) of[j] = 0.f; else o[j] = from_float<T>(0.f); }
         return;
@@ -400,7 +401,7 @@ __global__ void attn_combine_kernel(const float* __restrict__ part_m, const floa
     }
     float l = block_sum(lsum, red);
     if (sink != nullptr) l += expf(sk - m);
-    const float inv = l > 0.f ? 1.f / l : 0.f;
+    const float inv = l > 0.f ? out_scale / l : 0.f;
     const float* pa = part_acc + row * n_splits * d;
     if ((d & 3) == 0) {
         // four dims a thread, eight splits' loads in flight; per dim the sums are those of the loop below, in its order
@@ -511,15 +512,16 @@ static int attention_impl(const void* q, const void* k_pool, const void* v_pool,
                           int n_splits, int split_len, float* scratch, int* counters, int* status, int use_mma,
                           cudaStream_t stream, const void* prefetch = nullptr, unsigned long long prefetch_bytes = 0,
                           float softcap = 0.f, int keep_first = 0, const float* sink = nullptr, int v_rep = 1,
-                          int out_f32 = 0, int ext_mma = 0, int v_ld = 0) {
+                          int out_f32 = 0, int ext_mma = 0, int v_ld = 0, int out_ld = 0, float out_scale = 1.f) {
     if (n_rows == 0 || T == 0) return 0;
     FD_REQUIRE(softcap >= 0.f && keep_first >= 0 && v_rep >= 1 && (v_rep == 1 || v_rep == n_kv), -2,
                "attention: soft cap %g, %d kept first keys, weights applied to %d value heads of %d", softcap, keep_first,
                v_rep, n_kv);
     const bool ext = softcap > 0.f || (keep_first > 0 && window > 0) || sink != nullptr || v_rep > 1 || out_f32;
     if (ext) use_mma = 0;
-    // of the options the tensor-core decode kernel has the keyless term: a decode step that asks for nothing else runs there
-    const bool sink_only = sink != nullptr && !(softcap > 0.f) && !(keep_first > 0 && window > 0) && v_rep == 1 && !out_f32;
+    // of the options the tensor-core decode kernel has the cap and the keyless term: a decode step that asks for nothing else
+    // runs there (and a prompt step on the tcgen05 kernel, which has the same two)
+    const bool tc_options = ext && !(keep_first > 0 && window > 0) && v_rep == 1 && !out_f32;
     if (v_ld <= 0) v_ld = dv;
     FD_REQUIRE(v_ld == dv || (v_ld == d && dv <= d && k_pool == v_pool && v_rep == 1), -2,
                "attention: value rows of %d in rows of %d", dv, v_ld);
@@ -527,7 +529,7 @@ static int attention_impl(const void* q, const void* k_pool, const void* v_pool,
     const bool latent = k_pool == v_pool && n_kv == 1 && dtype == 1 && ext_mma != 0 && v_rep == 1 && !out_f32 && chunk == 0 &&
                         !(softcap > 0.f) && !(keep_first > 0 && window > 0) && (v_ld != dv || (d != 64 && d != 128));
     if (v_ld != dv) { use_mma = 0; if (!latent) ext_mma = 0; }
-    const bool decode_mma = !latent && (use_mma != 0 || (sink_only && ext_mma != 0)) && dtype == 1 && max_q_len == 1 && dv == d;
+    const bool decode_mma = !latent && (use_mma != 0 || (tc_options && ext_mma != 0)) && dtype == 1 && max_q_len == 1 && dv == d;
     FD_REQUIRE(n_kv > 0 && n_q % n_kv == 0, -2, "attention: %d query heads are not a multiple of %d KV heads", n_q, n_kv);
     const int G = n_q / n_kv;
     FD_REQUIRE(d % 8 == 0 && d >= 8 && d <= D_MAX, -2, "attention: head size %d must be a multiple of 8 in [8, %d]", d, D_MAX);
@@ -544,10 +546,13 @@ static int attention_impl(const void* q, const void* k_pool, const void* v_pool,
                "attention: queries, cache pools and scratch memory must be 16-byte aligned");
     FD_REQUIRE(n_splits == 1 || T <= 65535, -2, "attention: the split form takes at most 65535 tokens, got %d", T);
     FD_REQUIRE(n_rows <= 65535 && n_kv <= 65535, -2, "attention: batch of %d rows too large", n_rows);
+    FD_REQUIRE(out_ld == 0 || (out_ld >= n_q * v_rep * dv && out_ld % 8 == 0 && (uintptr_t)out % 16 == 0 && !latent), -2,
+               "attention: output rows of %d elements (a multiple of 8, 16-byte aligned, at least %d)", out_ld, n_q * v_rep * dv);
 
     AttnParams p;
     p.pf_ptr = (const unsigned char*)prefetch; p.pf_bytes = prefetch ? prefetch_bytes : 0;
     p.q = q; p.k_pool = k_pool; p.v_pool = v_pool; p.out = out;
+    p.out_ld = out_ld > 0 ? out_ld : n_q * v_rep * dv; p.out_scale = out_scale;
     const size_t n_part = (size_t)T * n_q * v_rep * n_splits;
     // accumulators first: they are stored as float4 and must stay 16-byte aligned
     p.part_acc = scratch;
@@ -581,8 +586,7 @@ static int attention_impl(const void* q, const void* k_pool, const void* v_pool,
     }
     if (latent) rc = launch_attn_latent_mma(p, tok_row, T, stream);
     else if (ext && ext_mma && dtype == 1 && max_q_len > 1) {
-        // of the options the tcgen05 prompt kernel has the keyless term too (head size 128)
-        if (sink_only && dv == d) rc = launch_attn_prefill_tcgen05(p, n_rows, T, max_q_len, stream);
+        if (tc_options && dv == d) rc = launch_attn_prefill_tcgen05(p, n_rows, T, max_q_len, stream);
         if (rc == 1) rc = launch_attn_prefill_mma_ext(p, n_rows, max_q_len, stream);
     }
     if (rc == 1)
@@ -593,10 +597,10 @@ static int attention_impl(const void* q, const void* k_pool, const void* v_pool,
     if (dtype == 0)
         return launch("attention_combine", attn_combine_kernel<float>, grid, dim3(128), 0, stream, dim3(1, 1, 1),
                       (const float*)p.part_m, (const float*)p.part_l, (const float*)p.part_acc, (float*)out, tok_row,
-                      row_slot, n_q * v_rep, dv, n_splits, sink, v_rep, out_f32);
+                      row_slot, n_q * v_rep, dv, n_splits, sink, v_rep, out_f32, p.out_ld, out_scale);
     return launch("attention_combine", attn_combine_kernel<bf16>, grid, dim3(128), 0, stream, dim3(1, 1, 1),
                   (const float*)p.part_m, (const float*)p.part_l, (const float*)p.part_acc, (bf16*)out, tok_row,
-                  row_slot, n_q * v_rep, dv, n_splits, sink, v_rep, out_f32);
+                  row_slot, n_q * v_rep, dv, n_splits, sink, v_rep, out_f32, p.out_ld, out_scale);
 }
 
 // out[t, h, :] = scale * sum_g mix[h, g] * o[t, g, vh(h), :] with vh(h) = h / (n_q / n_kv): every head takes the other
@@ -666,11 +670,13 @@ extern "C" int fd_attention(const void* q, const void* k_pool, const void* v_poo
                             const int* row_q_len, const int* row_ctx_len, int n_rows, int T,
                             int max_q_len, int n_q, int n_kv, int d, float scale, int window, int dv, int chunk,
                             int n_splits, int split_len, float* scratch, int* counters, int* status,
-                            const void* prefetch, unsigned long long prefetch_bytes, cudaStream_t stream) {
+                            const void* prefetch, unsigned long long prefetch_bytes, int out_ld, float out_scale,
+                            cudaStream_t stream) {
     FD_REQUIRE((uintptr_t)prefetch % 16 == 0, -2, "attention: the memory to prefetch must be 16-byte aligned");
     return attention_impl(q, k_pool, v_pool, out, dtype, block_table, max_blocks, num_blocks, block_size, tok_row,
                           row_slot, row_q_start, row_q_len, row_ctx_len, n_rows, T, max_q_len, n_q, n_kv, d, scale,
-                          window, dv, chunk, n_splits, split_len, scratch, counters, status, 1, stream, prefetch, prefetch_bytes);
+                          window, dv, chunk, n_splits, split_len, scratch, counters, status, 1, stream, prefetch, prefetch_bytes,
+                          0.f, 0, nullptr, 1, 0, 0, 0, out_ld, out_scale);
 }
 
 // The same without the tcgen05 kernel: prompts go to the mma.sync kernel (head sizes other than 128 always
@@ -692,9 +698,10 @@ extern "C" int fd_attention_mma_sync(const void* q, const void* k_pool, const vo
 // first so many positions stay visible; sink [n_q] (or null): a keyless term exp(sink[h]) in head h's denominator;
 // v_rep == n_kv: every query head's weights are applied to all value heads and out is [T, n_q, n_kv, dv] (scratch for
 // the split form: fd_attn_scratch_floats(T, n_q * n_kv, dv, n_splits)); out_f32: out is float.  Decode steps in bfloat16
-// whose only option is the keyless term run on the tensor-core decode kernel when use_mma is set and it takes the sizes
+// whose only options are the cap and the keyless term run on the tensor-core decode kernel when use_mma is set and it takes the sizes
 // (counters: as for fd_attention, the kernel then merges its own splits).  v_ld: 0, or d when v_pool is k_pool and the
-// values are the first dv columns of the keys' rows.
+// values are the first dv columns of the keys' rows.  out_ld (0: rows side by side) and out_scale: elements from one token's
+// output to the next one's, and a constant that every output is multiplied by.
 extern "C" int fd_attention_ext(const void* q, const void* k_pool, const void* v_pool, void* out, int dtype,
                                 const int* block_table, int max_blocks, int num_blocks, int block_size,
                                 const int* tok_row, const int* row_slot, const int* row_q_start,
@@ -702,11 +709,11 @@ extern "C" int fd_attention_ext(const void* q, const void* k_pool, const void* v
                                 int max_q_len, int n_q, int n_kv, int d, float scale, int window, int dv, int chunk,
                                 int n_splits, int split_len, float* scratch, int* status, float softcap, int keep_first,
                                 const float* sink, int v_rep, int out_f32, int use_mma, int* counters, int v_ld,
-                                cudaStream_t stream) {
+                                int out_ld, float out_scale, cudaStream_t stream) {
     return attention_impl(q, k_pool, v_pool, out, dtype, block_table, max_blocks, num_blocks, block_size, tok_row,
                           row_slot, row_q_start, row_q_len, row_ctx_len, n_rows, T, max_q_len, n_q, n_kv, d, scale,
                           window, dv, chunk, n_splits, split_len, scratch, counters, status, 0, stream, nullptr, 0,
-                          softcap, keep_first, sink, v_rep, out_f32, use_mma, v_ld);
+                          softcap, keep_first, sink, v_rep, out_f32, use_mma, v_ld, out_ld, out_scale);
 }
 
 // o [T, n_q, n_kv, dv] float, mix [n_q, n_q] float; out (dtype 0 float32, 1 bfloat16): pointer to the first output

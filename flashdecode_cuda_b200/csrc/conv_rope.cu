@@ -17,7 +17,7 @@
 //    of a packed projection);
 //  * add_concat: [resid + delta | other] as one row, for a product that re-enters
 //    the residual stream;
-//  * relu2: y = max(x, 0)^2.
+//  * relu2: y = max(x, 0)^2; relu2_cols: the same from a column range of one matrix to one of another.
 //
 // The convolution, the angles' use and the sigmoid are float; storage is float
 // or bfloat16.  The state is float in both.  The k-th tap multiplies the value
@@ -283,6 +283,36 @@ __global__ void relu2_kernel(const T* __restrict__ x, T* __restrict__ out, size_
     }
 }
 
+// out[m, c] = max(x[m, c], 0)^2 for C columns of rows of ldx and ldo elements; VEC: eight columns a thread (16-byte pieces of bfloat16)
+template <typename T, int VEC>
+__global__ void relu2_cols_kernel(const T* __restrict__ x, int ldx, T* __restrict__ out, int ldo, int C, size_t total) {
+    size_t e = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    const size_t stride = (size_t)gridDim.x * blockDim.x;
+    const int per = C / VEC;
+    for (; e < total; e += stride) {
+        const size_t m = e / per;
+        const int c = (int)(e - m * per) * VEC;
+        if (VEC == 1) {
+            const float v = fmaxf(to_float(x[m * ldx + c]), 0.f);
+            out[m * ldo + c] = from_float<T>(v * v);
+        } else {
+            alignas(16) T in[VEC];
+            alignas(16) T y[VEC];
+#pragma unroll
+            for (int j = 0; j < VEC * (int)sizeof(T) / 16; ++j)
+                reinterpret_cast<uint4*>(in)[j] = reinterpret_cast<const uint4*>(x + m * ldx + c)[j];
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) {
+                const float v = fmaxf(to_float(in[j]), 0.f);
+                y[j] = from_float<T>(v * v);
+            }
+#pragma unroll
+            for (int j = 0; j < VEC * (int)sizeof(T) / 16; ++j)
+                reinterpret_cast<uint4*>(out + m * ldo + c)[j] = reinterpret_cast<const uint4*>(y)[j];
+        }
+    }
+}
+
 static int grid_for(size_t total, int threads) {
     const size_t b = (total + threads - 1) / threads;
     return (int)(b < 148 * 16 ? b : 148 * 16);
@@ -392,4 +422,19 @@ extern "C" int fd_relu2(const void* x, void* out, int dtype, long long total, cu
                       dim3(1, 1, 1), (const float*)x, (float*)out, (size_t)total);
     return launch("relu2", relu2_kernel<bf16>, dim3(grid_for((size_t)total, 256)), dim3(256), 0, stream, dim3(1, 1, 1),
                   (const bf16*)x, (bf16*)out, (size_t)total);
+}
+
+// x: pointer to the first of C columns of a matrix with rows of ldx elements; out: likewise, rows of ldo elements; M rows.
+extern "C" int fd_relu2_cols(const void* x, int ldx, void* out, int ldo, int dtype, int M, int C, cudaStream_t stream) {
+    if (M == 0 || C == 0) return 0;
+    FD_REQUIRE(ldx >= C && ldo >= C, -2, "relu2_cols: %d columns of rows of %d and %d", C, ldx, ldo);
+    const bool vec = C % 8 == 0 && ldx % 8 == 0 && ldo % 8 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)out % 16 == 0;
+    const size_t total = (size_t)M * (vec ? C / 8 : C);
+    const dim3 grid(grid_for(total, 256)), block(256), one(1, 1, 1);
+    if (dtype == 0) {
+        if (vec) return launch("relu2_cols", relu2_cols_kernel<float, 8>, grid, block, 0, stream, one, (const float*)x, ldx, (float*)out, ldo, C, total);
+        return launch("relu2_cols", relu2_cols_kernel<float, 1>, grid, block, 0, stream, one, (const float*)x, ldx, (float*)out, ldo, C, total);
+    }
+    if (vec) return launch("relu2_cols", relu2_cols_kernel<bf16, 8>, grid, block, 0, stream, one, (const bf16*)x, ldx, (bf16*)out, ldo, C, total);
+    return launch("relu2_cols", relu2_cols_kernel<bf16, 1>, grid, block, 0, stream, one, (const bf16*)x, ldx, (bf16*)out, ldo, C, total);
 }

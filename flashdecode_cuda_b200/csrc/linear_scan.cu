@@ -10,6 +10,8 @@
 //  * mode 2 (decay per key channel): a_t = sigmoid(z_t)^(1/tau) per channel with z a float array of its own (the output
 //    of a product of its own), b_t = k_t, q_t = q_t * q_scale.  The power is taken as exp(log sigmoid(z) / tau) with
 //    log sigmoid(z) = -log(1 + e^-z) worked out on the side where the exponential cannot overflow.
+//  * mode 3 (decay and step size per head that follow the input): a_t = decay_t[h] for every channel and b_t = step_t[h] k_t,
+//    both from a float array [T, H, 2] (step, decay) of its own; `rep` heads share one q and one k.
 //
 // The state lives in float per cache slot and is carried from step to step; a step's tokens of a sequence are walked in
 // order, so the sums of every state element are the same whether a prompt comes whole, in portions or token by token.
@@ -35,7 +37,7 @@
 //    decay that comes through a narrow projection);
 //  * row_norm_gate: one norm over a token's heads side by side, times a weight per channel, times sigmoid(gate).
 //  * head_norm_gate: y = o / sqrt(mean(o^2) + eps) per token and head (over dv), times an optional weight [dv], times
-//    an optional silu(gate) read from a column range of a packed projection, times a constant; written with a row
+//    an optional silu(gate) read from a column range of a packed projection or sigmoid of a float array, times a constant; written with a row
 //    stride and a column offset of its own so that several mixers can fill one buffer.
 #include <math.h>
 
@@ -55,6 +57,7 @@ struct ScanParams {
     const float* lower;                // [H * d] (mode 1)
     const float* gate; int gate_ld;    // [T, gate_ld] from the first of the H * d columns on (mode 2)
     float q_scale, inv_tau;            // (mode 2)
+    const float* step; int rep;        // (mode 3) [T, H, 2]; heads per q / k head (1 in the other modes)
     const float* cos_t; const float* sin_t; int table_len, rot;
     float k_scale;
     int silu;                          // (mode 0) q, k and v pass silu
@@ -99,8 +102,9 @@ __device__ __forceinline__ void stage_tokens(const ScanParams& p, int h, int tok
             const int tt = idx / DP, i = idx - tt * DP;
             if (i >= d) continue;
             const size_t row = (size_t)(tok0 + tt) * p.ld;
-            xq[u] = to_float(proj[row + p.q_col + h * d + i]);
-            xk[u] = to_float(proj[row + p.k_col + h * d + i]);
+            const int qk = (h / p.rep) * d + i;
+            xq[u] = to_float(proj[row + p.q_col + qk]);
+            xk[u] = to_float(proj[row + p.k_col + qk]);
             if (p.mode == 0 && i < p.rot) {
                 const int pos = pos0 + tt;
                 if (pos < p.table_len) {
@@ -118,6 +122,10 @@ __device__ __forceinline__ void stage_tokens(const ScanParams& p, int h, int tok
                 cc[u] = p.lower[h * d + i];
             } else if (p.mode == 2) {
                 cc[u] = p.gate[(size_t)(tok0 + tt) * p.gate_ld + h * d + i];
+            } else if (p.mode == 3) {
+                const float2 sd = *reinterpret_cast<const float2*>(p.step + ((size_t)(tok0 + tt) * p.H + h) * 2);
+                cc[u] = sd.x;
+                ss[u] = sd.y;
             }
         }
 #pragma unroll
@@ -141,6 +149,10 @@ __device__ __forceinline__ void stage_tokens(const ScanParams& p, int h, int tok
                 at[0] = xq[u] * p.q_scale;
                 at[CS] = xk[u];
                 at[2 * CS] = expf(log_sig * p.inv_tau);
+            } else if (p.mode == 3) {
+                at[0] = xq[u];
+                at[CS] = xk[u] * cc[u];
+                at[2 * CS] = ss[u];
             } else {
                 const float lo = cc[u];
                 const float f = lo + (1.f - lo) / (1.f + expf(-xk[u]));
@@ -375,7 +387,7 @@ __global__ void scan_chain_kernel(const ScanParams p) {
 // A warp per (token, head).
 template <typename T>
 __global__ void head_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ w, const T* __restrict__ gate,
-                                      int ldg, T* __restrict__ out, int ld_out, int n_pairs, int H, int dv, float eps,
+                                      int ldg, const float* __restrict__ sig, T* __restrict__ out, int ld_out, int n_pairs, int H, int dv, float eps,
                                       float scale) {
     const int pair = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
     if (pair >= n_pairs) return;
@@ -393,6 +405,7 @@ __global__ void head_norm_gate_kernel(const float* __restrict__ o, const float* 
             const float z = to_float(gate[(size_t)t * ldg + h * dv + j]);
             y *= z / (1.f + expf(-z));
         }
+        if (sig != nullptr) y /= 1.f + expf(-sig[(size_t)t * H * dv + h * dv + j]);
         out[(size_t)t * ld_out + h * dv + j] = from_float<T>(y);
     }
 }
@@ -570,7 +583,8 @@ extern "C" long long fd_linear_scan_scratch_floats(int T, int n_rows, int H, int
 // at k_col - H * d columns each - and v at v_col (H * dv columns).  state [slots, H, d, dv] and out [T, H * dv] float.
 // mode 0: decay [H], cos_t / sin_t [table_len, rot / 2] (unused when rot == 0), k_scale.  mode 1: lower [H * d].
 // mode 2: gate [T, gate_ld] float (the decay's pre-activation, H * d columns from the pointer on), q_scale, inv_tau.
-// silu (mode 0, rot 0): q, k and v pass silu.
+// silu (mode 0, rot 0): q, k and v pass silu.  mode 3: step [T, H, 2] float (step size, decay); rep heads share a q and a k
+// head (H / rep * d columns each).
 // max_q_len: the longest portion of the step; with scratch memory (fd_linear_scan_scratch_floats floats for the step's T
 // tokens) portions longer than two segments run in segments side by side, otherwise each in one CTA per head and tile.
 extern "C" int fd_linear_scan(const void* proj, int ld, int dtype, int q_col, int k_col, int v_col, float* state,
@@ -579,11 +593,11 @@ extern "C" int fd_linear_scan(const void* proj, int ld, int dtype, int q_col, in
                               const int* row_q_start, const int* row_q_len, const int* row_ctx_len, int n_rows, int H,
                               int d, int dv, int write_state, int* status, int T, int max_q_len, float* scratch,
                               long long scratch_floats, const float* gate, int gate_ld, float q_scale, float inv_tau, int silu,
-                              cudaStream_t stream) {
+                              const float* step, int rep, cudaStream_t stream) {
     if (n_rows == 0) return 0;
     FD_REQUIRE(H > 0 && d > 0 && dv > 0 && d <= 256, -2, "linear_scan: %d heads of %d x %d (d at most 256)", H, d, dv);
-    FD_REQUIRE(mode >= 0 && mode <= 2, -2, "linear_scan: unknown mode %d", mode);
-    FD_REQUIRE(mode == 1 ? lower != nullptr : (mode == 2 ? gate != nullptr && gate_ld >= H * d : decay != nullptr), -2,
+    FD_REQUIRE(mode >= 0 && mode <= 3, -2, "linear_scan: unknown mode %d", mode);
+    FD_REQUIRE(mode == 3 ? step != nullptr && rep >= 1 && H % rep == 0 : mode == 1 ? lower != nullptr : (mode == 2 ? gate != nullptr && gate_ld >= H * d : decay != nullptr), -2,
                "linear_scan: the mode's constants are missing");
     FD_REQUIRE(rot >= 0 && rot % 2 == 0 && rot <= d && (rot == 0 || mode != 0 || (cos_t && sin_t)), -2,
                "linear_scan: %d rotated dimensions of %d", rot, d);
@@ -594,6 +608,7 @@ extern "C" int fd_linear_scan(const void* proj, int ld, int dtype, int q_col, in
     p.rot = mode == 0 ? rot : 0; p.k_scale = k_scale;
     p.silu = mode == 0 && silu;
     FD_REQUIRE(!p.silu || p.rot == 0, -2, "linear_scan: silu on q, k and v goes without a rotation");
+    p.step = step; p.rep = mode == 3 ? rep : 1;
     p.gate = gate; p.gate_ld = gate_ld; p.q_scale = q_scale; p.inv_tau = inv_tau;
     p.row_slot = row_slot; p.row_q_start = row_q_start; p.row_q_len = row_q_len; p.row_ctx_len = row_ctx_len;
     p.H = H; p.d = d; p.dv = dv; p.mode = mode; p.write_state = write_state; p.status = status;
@@ -619,8 +634,8 @@ extern "C" int fd_linear_scan(const void* proj, int ld, int dtype, int q_col, in
 }
 
 // o [T, H * dv] float; w [dv] float or null; gate: pointer to the first gate column of a packed projection with row
-// stride ldg (dtype as out), or null; out: pointer to the first output column, row stride ld_out.
-extern "C" int fd_head_norm_gate(const float* o, const float* w, const void* gate, int ldg, void* out, int ld_out,
+// stride ldg (dtype as out), or null; sig [T, H * dv] float: the result is multiplied by its sigmoid, or null; out: pointer to the first output column, row stride ld_out.
+extern "C" int fd_head_norm_gate(const float* o, const float* w, const void* gate, int ldg, const float* sig, void* out, int ld_out,
                                  int dtype, int T, int H, int dv, float eps, float scale, cudaStream_t stream) {
     const long long pairs = (long long)T * H;
     if (pairs == 0) return 0;
@@ -628,9 +643,9 @@ extern "C" int fd_head_norm_gate(const float* o, const float* w, const void* gat
     const dim3 grid((unsigned)((pairs + 3) / 4));
     if (dtype == 0)
         return launch("head_norm_gate", head_norm_gate_kernel<float>, grid, dim3(128), 0, stream, dim3(1, 1, 1), o, w,
-                      (const float*)gate, ldg, (float*)out, ld_out, (int)pairs, H, dv, eps, scale);
+                      (const float*)gate, ldg, sig, (float*)out, ld_out, (int)pairs, H, dv, eps, scale);
     return launch("head_norm_gate", head_norm_gate_kernel<bf16>, grid, dim3(128), 0, stream, dim3(1, 1, 1), o, w,
-                  (const bf16*)gate, ldg, (bf16*)out, ld_out, (int)pairs, H, dv, eps, scale);
+                  (const bf16*)gate, ldg, sig, (bf16*)out, ld_out, (int)pairs, H, dv, eps, scale);
 }
 
 // o [T, n] float; w [n] float; gate: pointer to the first gate column of a packed projection with row stride ldg (dtype as

@@ -1,0 +1,73 @@
+// Short causal convolution over time of one channel, for the kernels that prepare a recurrence's inputs.
+//
+// y[t] = bias + sum_k w[k] u[t - (taps - 1) + k], zeros before the sequence's start.  The values of earlier steps come from
+// the sequence's ring, float [slots, taps, C]: the value of position p lies at place p % taps.  A ring of `taps` places
+// (one more than a token needs) lets a step of single tokens write its own value, at the place of the value that no
+// one reads any more, while other CTAs still read the earlier ones.  A place whose position would lie before the start is
+// never read, so a slot's old contents do not matter.  The taps are added in the order k = 0, 1, ... after the bias,
+// from the same values wherever they come from: how a prompt is cut changes no bit.
+#pragma once
+
+#include "common.cuh"
+
+namespace fd {
+
+constexpr int SC_TOK = 8;             // tokens of a tile at most
+constexpr int SC_TAPS = 4;            // more taps than this take the plain loop
+
+struct ConvMeta {                     // what the tokens of a tile need to know, in shared memory
+    int slot[SC_TOK], i[SC_TOK], pos[SC_TOK], single[SC_TOK];     // slot -1: padding row; i: place in its row's new tokens
+};
+
+// threads 0 .. nt - 1 fill the tile's entries; the caller synchronises
+__device__ __forceinline__ void conv_meta(ConvMeta& m, int t0, int nt, const int* tok_row, const int* tok_pos,
+                                          const int* row_slot, const int* row_q_start, const int* row_q_len) {
+    if (threadIdx.x < nt) {
+        const int t = t0 + threadIdx.x, r = tok_row[t];
+        m.slot[threadIdx.x] = row_slot[r];
+        m.i[threadIdx.x] = t - row_q_start[r];
+        m.pos[threadIdx.x] = tok_pos[t];
+        m.single[threadIdx.x] = row_q_len[r] == 1;
+    }
+}
+
+// The nt <= SC_TOK tokens from t0 on of channel c of C (column `col` points at it in token 0's row, rows of ld elements);
+// rows that bring a single token leave their value in the ring when `keep` is set.
+template <typename T>
+__device__ __forceinline__ void conv_channel(const T* __restrict__ col, int ld, const float* __restrict__ w, float bias, int taps,
+                                             float* ring, int c, int C, const ConvMeta& m, int t0, int nt, bool keep,
+                                             float y[SC_TOK]) {
+    float wk[SC_TAPS];
+#pragma unroll
+    for (int k = 0; k < SC_TAPS; ++k) wk[k] = k < taps ? w[k] : 0.f;
+#pragma unroll
+    for (int tt = 0; tt < SC_TOK; ++tt) {
+        y[tt] = 0.f;
+        if (tt >= nt || m.slot[tt] < 0) continue;
+        const int t = t0 + tt, i = m.i[tt], pos = m.pos[tt];
+        float* rg = ring + (size_t)m.slot[tt] * taps * C + c;
+        auto value = [&](int back) -> float {
+            if (back <= i) return to_float(col[(size_t)(t - back) * ld]);
+            return back <= pos ? rg[(size_t)((pos - back) % taps) * C] : 0.f;
+        };
+        float a = bias;
+        const float cur = value(0);
+        if (taps <= SC_TAPS) {
+            float u[SC_TAPS];
+#pragma unroll
+            for (int k = 0; k < SC_TAPS; ++k) u[k] = k < taps - 1 ? value(taps - 1 - k) : (k == taps - 1 ? cur : 0.f);
+#pragma unroll
+            for (int k = 0; k < SC_TAPS; ++k) if (k < taps) a = fmaf(wk[k], u[k], a);
+        } else {
+            for (int k = 0; k < taps; ++k) a = fmaf(w[k], value(taps - 1 - k), a);
+        }
+        if (keep && taps > 1 && m.single[tt]) rg[(size_t)(pos % taps) * C] = cur;
+        y[tt] = a;
+    }
+}
+
+__device__ __forceinline__ float sc_silu(float z) { return z / (1.f + expf(-z)); }
+__device__ __forceinline__ float sc_sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
+__device__ __forceinline__ float sc_softplus(float z) { return z > 0.f ? z + log1pf(expf(-z)) : log1pf(expf(z)); }
+
+}  // namespace fd

@@ -94,24 +94,31 @@ def _declare(L: ctypes.CDLL) -> None:
         "fd_attn_simt_qt": [I],
         "fd_attn_decode_group": [I, I, I],
         "fd_attention_simt": [P, P, P, P, I, P, I, I, I, P, P, P, P, P, I, I, I, I, I, I, F, I, I, I, I, I, P, P, P],
-        "fd_attention": [P, P, P, P, I, P, I, I, I, P, P, P, P, P, I, I, I, I, I, I, F, I, I, I, I, I, P, P, P, P, c_ulonglong, P],
+        "fd_attention": [P, P, P, P, I, P, I, I, I, P, P, P, P, P, I, I, I, I, I, I, F, I, I, I, I, I, P, P, P, P, c_ulonglong, I, F, P],
         "fd_attention_mma_sync": [P, P, P, P, I, P, I, I, I, P, P, P, P, P, I, I, I, I, I, I, F, I, I, I, I, I, P, P, P, P],
         "fd_attention_dense": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, F, I, P, P, I, P, P],
         "fd_conv_rope_append": [P, I, I, P, P, P, P, P, I, I, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, P, I, P, P, F, I, I, P],
-        "fd_attention_ext": [P, P, P, P, I, P, I, I, I, P, P, P, P, P, I, I, I, I, I, I, F, I, I, I, I, I, P, P, F, I, P, I, I, I, P, I, P],
+        "fd_attention_ext": [P, P, P, P, I, P, I, I, I, P, P, P, P, P, I, I, I, I, I, I, F, I, I, I, I, I, P, P, F, I, P, I, I, I, P, I, I, F, P],
         "fd_attn_head_mix": [P, P, P, I, I, I, I, I, I, F, P],
         "fd_add_dyn_tanh": [P, I, P, I, P, P, F, P, I, P, I, I, P],
         "fd_quad_exp_act": [P, P, I, P, LL, P],
         "fd_scale_f32": [P, LL, F, P],
         "fd_axpy_f32": [P, P, I, LL, F, I, P],
-        "fd_linear_scan": [P, I, I, I, I, I, P, P, I, P, P, P, P, I, I, F, P, P, P, P, I, I, I, I, I, P, I, I, P, LL, P, I, F, F, I, P],
+        "fd_linear_scan": [P, I, I, I, I, I, P, P, I, P, P, P, P, I, I, F, P, P, P, P, I, I, I, I, I, P, I, I, P, LL, P, I, F, F, I, P, I, P],
         "fd_row_norm_gate": [P, P, P, I, P, I, I, I, F, P],
-        "fd_head_norm_gate": [P, P, P, I, P, I, I, I, I, I, F, F, P],
+        "fd_head_norm_gate": [P, P, P, I, P, P, I, I, I, I, I, F, F, P],
+        "fd_delta_prepare": [P, I, I, I, I, I, I, I, I, P, P, I, I, P, I, P, P, I, P, P, F, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, P],
+        "fd_delta_scan": [P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, P],
+        "fd_conv_ring_update": [P, I, I, P, P, P, P, P, I, I, I, P],
+        "fd_ssd_prepare": [P, I, I, I, I, I, P, P, P, I, I, P, P, P, P, P, P, P, P, P, I, I, P],
+        "fd_ssd_gate_norm": [P, P, I, P, P, I, P, P, I, I, I, I, I, I, F, F, P],
+        "fd_rope_norm_append": [P, I, I, P, P, P, P, P, P, F, P, P, I, I, I, I, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, I, P, P],
         "fd_low_rank_expand": [P, I, P, P, P, I, I, I, I, P],
         "fd_conv_state_update": [P, I, I, P, P, P, P, I, I, I, P],
         "fd_gate_mul": [P, P, I, P, I, I, I, P],
         "fd_add_concat": [P, I, P, P, P, I, I, I, P],
         "fd_relu2": [P, P, I, LL, P],
+        "fd_relu2_cols": [P, I, P, I, I, I, I, P],
         "fd_moe_tile_rows": [I, I],
         "fd_moe_route": [P, P, I, P, P, P, P, P, I, I, I, I, I, I, I, I, F, P],
         "fd_glu_mul": [P, P, I, I, I, I, I, F, P],
@@ -722,16 +729,17 @@ def _counters(device, n: int) -> torch.Tensor:
 
 def _attention(fn_name, q, k_pool, v_pool, out, block_table, tok_row, row_slot, row_q_start, row_q_len,
                row_ctx_len, n_rows, max_q_len, n_q, n_kv, head_dim, scale, window, n_splits, split_len,
-               scratch, status, prefetch=None, prefetch_bytes=0, chunk=0) -> None:
+               scratch, status, prefetch=None, prefetch_bytes=0, chunk=0, out_col=None, out_scale=1.0) -> None:
     T = q.shape[0]
     num_blocks, _, block_size, _ = k_pool.shape
     v_dim = v_pool.shape[-1]
-    assert q.dtype == k_pool.dtype == out.dtype and k_pool.shape[-1] == head_dim and out.shape[-1] == n_q * v_dim
+    assert q.dtype == k_pool.dtype == out.dtype and k_pool.shape[-1] == head_dim
+    assert out.shape[-1] == n_q * v_dim or (out_col is not None and out_col + n_q * v_dim <= out.shape[-1])
     assert v_pool.shape[:3] == k_pool.shape[:3]
     if n_splits > 1:
         assert scratch is not None and scratch.dtype == torch.float32
         assert scratch.numel() >= attention_scratch_floats(T, n_q, v_dim, n_splits)
-    args = [_ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(out), _dt(q.dtype), _ptr(block_table), block_table.shape[1],
+    args = [_ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(out) + (out_col or 0) * out.element_size(), _dt(q.dtype), _ptr(block_table), block_table.shape[1],
             num_blocks, block_size, _ptr(tok_row), _ptr(row_slot), _ptr(row_q_start), _ptr(row_q_len),
             _ptr(row_ctx_len), n_rows, T, max_q_len, n_q, n_kv, head_dim, float(scale), int(window), int(v_dim),
             int(chunk), n_splits, split_len, _ptr(scratch)]
@@ -741,7 +749,7 @@ def _attention(fn_name, q, k_pool, v_pool, out, block_table, tok_row, row_slot, 
         args.append(_ptr(_counters(q.device, n_rows * n_q)) if fused else None)
     args.append(_ptr(status))
     if fn_name == "fd_attention":
-        args += list(_prefetch_args(prefetch, prefetch_bytes))
+        args += list(_prefetch_args(prefetch, prefetch_bytes)) + [0 if out_col is None else out.shape[-1], float(out_scale)]
     args.append(_stream())
     _check(getattr(lib(), fn_name)(*args))
 
@@ -752,7 +760,8 @@ def attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, out: 
               n_rows: int, max_q_len: int, n_q: int, n_kv: int, head_dim: int, scale: float,
               window: int = 0, n_splits: int = 1, split_len: int = 0,
               scratch: Optional[torch.Tensor] = None, status: Optional[torch.Tensor] = None,
-              prefetch: Optional[torch.Tensor] = None, prefetch_bytes: int = 0, chunk: int = 0) -> None:
+              prefetch: Optional[torch.Tensor] = None, prefetch_bytes: int = 0, chunk: int = 0,
+              out_col: Optional[int] = None, out_scale: float = 1.0) -> None:
     """Causal GQA attention of the step's tokens over the paged cache, by the
     fastest kernel that takes the sizes (tensor cores for bfloat16 decode steps
     with head size 64 or 128; the CUDA-core kernel otherwise).  ``window`` > 0: a query
@@ -760,10 +769,11 @@ def attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, out: 
     ``chunk`` positions, counted from the start of the sequence.  The size of a value head
     is that of ``v_pool`` (the tensor-core kernels take it equal to the key's).  ``prefetch``: a
     tensor that a later kernel streams; the tensor-core decode kernel asks L2 for its
-    first ``prefetch_bytes`` when its own reads are through (the other kernels do not)."""
+    first ``prefetch_bytes`` when its own reads are through (the other kernels do not).  ``out_col``: the heads go to the
+    columns from there on of a wider ``out`` (columns and rows at multiples of 8); ``out_scale`` multiplies them."""
     _attention("fd_attention", q, k_pool, v_pool, out, block_table, tok_row, row_slot, row_q_start, row_q_len,
                row_ctx_len, n_rows, max_q_len, n_q, n_kv, head_dim, scale, window, n_splits, split_len,
-               scratch, status, prefetch, prefetch_bytes, chunk=chunk)
+               scratch, status, prefetch, prefetch_bytes, chunk=chunk, out_col=out_col, out_scale=out_scale)
 
 
 def attention_mma_sync(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, out: torch.Tensor,
@@ -800,39 +810,42 @@ def attention_ext(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, o
                   window: int = 0, n_splits: int = 1, split_len: int = 0,
                   scratch: Optional[torch.Tensor] = None, status: Optional[torch.Tensor] = None, chunk: int = 0,
                   softcap: float = 0.0, keep_first: int = 0, sink: Optional[torch.Tensor] = None,
-                  all_value_heads: bool = False, tensor_cores: bool = True, value_dim: int = 0) -> None:
+                  all_value_heads: bool = False, tensor_cores: bool = True, value_dim: int = 0,
+                  out_col: Optional[int] = None, out_scale: float = 1.0) -> None:
     """Attention with more options, on the CUDA cores; prompt steps in bfloat16 whose key and value heads both have 64
     or 128 dimensions run on the tensor cores unless ``tensor_cores`` is False, and so do decode steps in bfloat16 whose
-    only option is ``sink`` (the split-keys decode kernel, at the sizes it takes).  ``softcap`` > 0: the scaled scores
+    only options are ``softcap`` and ``sink`` (the split-keys decode kernel, at the sizes it takes).  ``softcap`` > 0: the scaled scores
     become softcap * tanh(score / softcap).  ``keep_first``: with a window, keys at positions below it stay
     visible.  ``sink`` [n_q] float32: exp(sink[h]) is one more term of head h's softmax denominator; it has
     no key and no value.  ``all_value_heads``: every query head's weights are applied to each of the ``n_kv``
     value heads; ``out`` is then float32 [T, n_q, n_kv, dv] (for ``attn_head_mix``).  Otherwise ``out`` is
     [T, n_q * dv] in q's dtype, or float32 if it is given so.  ``value_dim`` (with ``v_pool`` the same memory as
-    ``k_pool``): the values are the first so many columns of the keys."""
+    ``k_pool``): the values are the first so many columns of the keys.  ``out_col``, ``out_scale``: as in ``attention``."""
     T = q.shape[0]
     num_blocks, _, block_size, _ = k_pool.shape
     assert not value_dim or v_pool.data_ptr() == k_pool.data_ptr()
     v_dim = value_dim or v_pool.shape[-1]
     v_rep = n_kv if all_value_heads else 1
     assert q.dtype == k_pool.dtype == v_pool.dtype and k_pool.shape[-1] == head_dim
-    assert out.dtype in (q.dtype, torch.float32) and out.numel() == T * n_q * v_rep * v_dim
+    assert out.dtype in (q.dtype, torch.float32)
+    assert out.numel() == T * n_q * v_rep * v_dim or (out_col is not None and out_col + n_q * v_rep * v_dim <= out.shape[-1])
     assert not all_value_heads or out.dtype == torch.float32
     assert sink is None or (sink.dtype == torch.float32 and sink.numel() == n_q)
     if n_splits > 1:
         assert scratch is not None and scratch.dtype == torch.float32
         assert scratch.numel() >= attention_scratch_floats(T, n_q * v_rep, v_dim, n_splits)
-    # a bfloat16 decode step whose only option is the keyless term may run on the tensor-core decode kernel, which
+    # a bfloat16 decode step whose only options are the cap and the keyless term may run on the tensor-core decode kernel, which
     # merges its own splits when it is given counters
-    fused = (n_splits > 1 and max_q_len == 1 and q.dtype == torch.bfloat16 and tensor_cores and sink is not None
-             and not softcap and not (keep_first and window) and not all_value_heads and out.dtype == q.dtype)
+    fused = (n_splits > 1 and max_q_len == 1 and q.dtype == torch.bfloat16 and tensor_cores and (sink is not None or softcap)
+             and not (keep_first and window) and not all_value_heads and out.dtype == q.dtype)
     _check(lib().fd_attention_ext(
-        _ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(out), _dt(q.dtype), _ptr(block_table), block_table.shape[1],
+        _ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(out) + (out_col or 0) * out.element_size(), _dt(q.dtype), _ptr(block_table), block_table.shape[1],
         num_blocks, block_size, _ptr(tok_row), _ptr(row_slot), _ptr(row_q_start), _ptr(row_q_len), _ptr(row_ctx_len),
         n_rows, T, max_q_len, n_q, n_kv, head_dim, float(scale), int(window), int(v_dim), int(chunk), n_splits,
         split_len, _ptr(scratch), _ptr(status), float(softcap), int(keep_first), _ptr(sink), v_rep,
         int(out.dtype == torch.float32 and q.dtype != torch.float32 or all_value_heads), int(tensor_cores),
-        _ptr(_counters(q.device, n_rows * n_q)) if fused else None, k_pool.shape[-1] if value_dim else 0, _stream()))
+        _ptr(_counters(q.device, n_rows * n_q)) if fused else None, k_pool.shape[-1] if value_dim else 0,
+        0 if out_col is None else out.shape[-1], float(out_scale), _stream()))
 
 
 def attention_dense_takes(key_size: int, rot_size: int, v_size: int) -> bool:
@@ -918,7 +931,7 @@ def axpy_f32(y: torch.Tensor, x: torch.Tensor, s: float, accumulate: bool = True
     _check(lib().fd_axpy_f32(_ptr(y), _ptr(x), _dt(x.dtype), y.numel(), float(s), int(accumulate), _stream()))
 
 
-SCAN_DECAY, SCAN_GATED, SCAN_CHANNEL_DECAY = 0, 1, 2
+SCAN_DECAY, SCAN_GATED, SCAN_CHANNEL_DECAY, SCAN_STEP = 0, 1, 2, 3
 
 
 def linear_scan(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, state: torch.Tensor, out: torch.Tensor,
@@ -928,7 +941,8 @@ def linear_scan(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, state: t
                 lower: Optional[torch.Tensor] = None, cos: Optional[torch.Tensor] = None,
                 sin: Optional[torch.Tensor] = None, rot_dims: int = 0, k_scale: float = 1.0, max_q_len: int = 0,
                 scratch: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, gate_col: int = 0,
-                q_scale: float = 1.0, tau: float = 1.0, silu: bool = False) -> None:
+                q_scale: float = 1.0, tau: float = 1.0, silu: bool = False, step: Optional[torch.Tensor] = None,
+                qk_heads: int = 0) -> None:
     """The recurrence S_t = diag(a_t) S_(t-1) + b_t v_t^T, o_t = S_t^T q_t per sequence and head over the step's
     tokens, from ``state`` [slots, heads, head_dim, v_head_dim] (float32, updated when ``write_state``) to ``out``
     [T, heads * v_head_dim] (float32).  q, k and v are column ranges of ``proj`` [T, ld].  ``SCAN_DECAY``: a = decay[h],
@@ -936,18 +950,25 @@ def linear_scan(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, state: t
     ``SCAN_GATED``: the k columns hold the gate's pre-activation z; a = lower + (1 - lower) sigmoid(z), b = 1 - a,
     q = silu of the q columns.  ``SCAN_CHANNEL_DECAY``: a = sigmoid(z)^(1 / tau) per key channel with z the columns
     ``gate_col ...`` of ``gate`` [T, ldg] (float32), b = the k columns, q = the q columns times ``q_scale``.
+    ``SCAN_STEP``: a = step[t, h, 1] for every channel and b = step[t, h, 0] times the k columns, ``step`` float32
+    [T, heads, 2]; ``qk_heads`` (0: as many as heads) heads of q and k, each shared by heads / qk_heads neighbours.
     ``silu`` (``SCAN_DECAY`` without a rotation): q, k and v pass silu on their way in.  With ``scratch`` (float32, ``linear_scan_scratch_floats`` elements) and ``max_q_len`` (the
     longest portion of the step), portions longer than two segments are cut into segments that run side by side."""
     T = proj.shape[0]
     assert state.dtype == out.dtype == torch.float32 and state.shape[1:] == (n_heads, head_dim, v_head_dim)
     assert out.shape == (T, n_heads * v_head_dim) and proj.is_contiguous()
-    assert max(q_col, k_col) + n_heads * head_dim <= proj.shape[1] and v_col + n_heads * v_head_dim <= proj.shape[1]
+    qk_heads = qk_heads or n_heads
+    assert n_heads % qk_heads == 0 and (qk_heads == n_heads or mode == SCAN_STEP)
+    assert max(q_col, k_col) + qk_heads * head_dim <= proj.shape[1] and v_col + n_heads * v_head_dim <= proj.shape[1]
     if mode == SCAN_DECAY:
         assert decay is not None and decay.dtype == torch.float32 and decay.numel() == n_heads
         if rot_dims:
             assert cos.dtype == torch.float32 and cos.shape[1] == rot_dims // 2 and sin.shape == cos.shape
     elif mode == SCAN_GATED:
         assert lower is not None and lower.dtype == torch.float32 and lower.numel() == n_heads * head_dim
+        rot_dims = 0
+    elif mode == SCAN_STEP:
+        assert step is not None and step.dtype == torch.float32 and step.shape == (T, n_heads, 2)
         rot_dims = 0
     else:
         assert gate is not None and gate.dtype == torch.float32 and gate.shape[0] == T and gate.is_contiguous()
@@ -961,7 +982,8 @@ def linear_scan(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, state: t
                                 _ptr(scratch) if scratch is not None else None,
                                 scratch.numel() if scratch is not None else 0,
                                 _col_ptr(gate, gate_col) if gate is not None else None,
-                                gate.shape[1] if gate is not None else 0, float(q_scale), 1.0 / float(tau), int(silu), _stream()))
+                                gate.shape[1] if gate is not None else 0, float(q_scale), 1.0 / float(tau), int(silu), _ptr(step), n_heads // qk_heads,
+                                _stream()))
 
 
 def linear_scan_segment() -> int:
@@ -999,18 +1021,141 @@ def row_norm_gate(o: torch.Tensor, weight: torch.Tensor, gate: torch.Tensor, gat
 
 def head_norm_gate(o: torch.Tensor, out: torch.Tensor, first_col: int, n_heads: int, v_head_dim: int, eps: float,
                    weight: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, gate_col: int = 0,
-                   scale: float = 1.0) -> None:
+                   scale: float = 1.0, sigmoid_gate: Optional[torch.Tensor] = None) -> None:
     """out[t, first_col + h dv + j] = scale * o[t, h, j] / sqrt(mean_j o[t, h, :]^2 + eps) [* weight[j]]
     [* silu(gate[t, gate_col + h dv + j])].  ``o`` float32 [T, heads * dv]; ``weight`` float32 [dv]; ``gate`` a packed
-    projection [T, ldg] in out's dtype."""
+    projection [T, ldg] in out's dtype.  ``sigmoid_gate`` float32 [T, heads * dv]: the result times its sigmoid."""
     T = o.shape[0]
+    assert sigmoid_gate is None or (sigmoid_gate.dtype == torch.float32 and sigmoid_gate.shape == o.shape)
     assert o.dtype == torch.float32 and o.shape == (T, n_heads * v_head_dim) and out.shape[0] == T
     assert first_col + n_heads * v_head_dim <= out.shape[1]
     assert weight is None or (weight.dtype == torch.float32 and weight.numel() == v_head_dim)
     assert gate is None or (gate.dtype == out.dtype and gate.shape[0] == T and gate_col + n_heads * v_head_dim <= gate.shape[1])
     _check(lib().fd_head_norm_gate(_ptr(o), _ptr(weight), _col_ptr(gate, gate_col) if gate is not None else None,
-                                   gate.shape[1] if gate is not None else 0, _col_ptr(out, first_col), out.shape[1],
-                                   _dt(out.dtype), T, n_heads, v_head_dim, float(eps), float(scale), _stream()))
+                                   gate.shape[1] if gate is not None else 0, _ptr(sigmoid_gate),
+                                   _col_ptr(out, first_col), out.shape[1], _dt(out.dtype), T, n_heads, v_head_dim, float(eps), float(scale), _stream()))
+
+
+def delta_prepare(proj: torch.Tensor, cols, conv_w: torch.Tensor, ring: Optional[torch.Tensor], keep: bool, A_log: torch.Tensor,
+                  dt_bias: torch.Tensor, q_scale: float, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, g: torch.Tensor,
+                  beta: torch.Tensor, gate_z: Optional[torch.Tensor], tok_row: torch.Tensor, tok_pos: torch.Tensor,
+                  row_slot: torch.Tensor, row_q_start: torch.Tensor, row_q_len: torch.Tensor, n_heads: int, n_qk_heads: int,
+                  head_dim: int, v_head_dim: int, a2: Optional[torch.Tensor] = None, z_a: Optional[torch.Tensor] = None,
+                  g2: Optional[torch.Tensor] = None) -> None:
+    """What enters the gated delta rule, as float32.  ``cols``: first columns in ``proj`` [T, ld] of q, k, v, beta's
+    pre-activation, and the narrow vectors of decay and gate.  q, k, v: a causal convolution per channel (``conv_w`` float32
+    [C, taps], C = 2 n_qk_heads head_dim + n_heads v_head_dim; earlier values from ``ring`` float32 [slots, taps, C]) and silu;
+    every head of q and k a unit vector, q times ``q_scale``.  g = exp(-exp(A_log[h]) softplus(z + dt_bias)) per key channel,
+    z = ``a2`` [n_heads head_dim, R] times the narrow vector, or ``z_a`` float32 [T, n_heads head_dim].  beta = its sigmoid.
+    ``gate_z`` [T, n_heads v_head_dim] <- ``g2`` times the gate's narrow vector, if g2 is given.  ``keep``: rows that bring a
+    single token leave their values in the ring (longer rows: ``conv_ring_update``).  Outputs q, k [T, n_qk_heads, dp],
+    g [T, n_heads, dp], v [T, n_heads, dvp] with dp, dvp the head sizes rounded up to 4."""
+    T = proj.shape[0]
+    up4 = lambda n: -(-n // 4) * 4
+    C = 2 * n_qk_heads * head_dim + n_heads * v_head_dim
+    taps = conv_w.shape[1]
+    assert proj.is_contiguous() and conv_w.shape == (C, taps) and (taps == 1 or ring.shape[1:] == (taps, C))
+    assert q.shape == k.shape == (T, n_qk_heads, up4(head_dim)) and g.shape == (T, n_heads, up4(head_dim))
+    assert v.shape == (T, n_heads, up4(v_head_dim)) and beta.shape == (T, n_heads)
+    for t in (conv_w, ring, A_log, dt_bias, q, k, v, g, beta, gate_z, z_a):
+        assert t is None or t.dtype == torch.float32
+    assert A_log.numel() == n_heads and dt_bias.numel() == n_heads * head_dim
+    assert (a2 is None) != (z_a is None) and (a2 is None or (a2.dtype == proj.dtype and a2.shape[0] == n_heads * head_dim))
+    assert z_a is None or z_a.shape == (T, n_heads * head_dim)
+    assert g2 is None or (g2.dtype == proj.dtype and g2.shape[0] == n_heads * v_head_dim and gate_z.shape == (T, n_heads * v_head_dim))
+    qc, kc, vc, bc, ac, gc = cols
+    ld = proj.shape[1]
+    assert max(qc, kc) + n_qk_heads * head_dim <= ld and vc + n_heads * v_head_dim <= ld and bc + n_heads <= ld
+    assert (a2 is None or ac + a2.shape[1] <= ld) and (g2 is None or gc + g2.shape[1] <= ld)
+    _check(lib().fd_delta_prepare(
+        _ptr(proj), ld, _dt(proj.dtype), qc, kc, vc, bc, ac, gc, _ptr(conv_w), _ptr(ring), taps, int(keep), _ptr(a2),
+        a2.shape[1] if a2 is not None else 0, _ptr(z_a), _ptr(g2), g2.shape[1] if g2 is not None else 0, _ptr(A_log), _ptr(dt_bias),
+        float(q_scale), _ptr(q), _ptr(k), _ptr(v), _ptr(g), _ptr(beta), _ptr(gate_z), _ptr(tok_row), _ptr(tok_pos), _ptr(row_slot),
+        _ptr(row_q_start), _ptr(row_q_len), T, n_heads, n_qk_heads, head_dim, v_head_dim, _stream()))
+
+
+def delta_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, g: torch.Tensor, beta: torch.Tensor, state: torch.Tensor,
+               out: torch.Tensor, row_slot: torch.Tensor, row_q_start: torch.Tensor, row_q_len: torch.Tensor, n_rows: int,
+               write_state: bool) -> None:
+    """S <- diag(g) S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q, per sequence and head over the step's tokens, from
+    ``state`` [slots, heads, d, dv] (float32, updated when ``write_state``) to ``out`` [T, heads * dv] float32.  The inputs are
+    those ``delta_prepare`` leaves."""
+    H, d, dv = state.shape[1:]
+    T, Hk = q.shape[:2]
+    for t in (q, k, v, g, beta, state, out):
+        assert t.dtype == torch.float32
+    assert out.shape == (T, H * dv) and k.shape == q.shape and g.shape[:2] == (T, H) and v.shape[:2] == (T, H)
+    _check(lib().fd_delta_scan(_ptr(q), _ptr(k), _ptr(v), _ptr(g), _ptr(beta), _ptr(state), _ptr(out), _ptr(row_slot),
+                               _ptr(row_q_start), _ptr(row_q_len), n_rows, H, Hk, d, dv, int(write_state), _stream()))
+
+
+def conv_ring_update(proj: torch.Tensor, first_col: int, ring: torch.Tensor, row_slot: torch.Tensor, row_q_start: torch.Tensor,
+                     row_q_len: torch.Tensor, row_ctx_len: torch.Tensor, n_rows: int) -> None:
+    """ring[slot, p % taps] <- the columns ``first_col ...`` of ``proj`` for the last taps - 1 positions p of every row that
+    brings more than one token; ``ring`` float32 [slots, taps, C]."""
+    taps, C = ring.shape[1:]
+    assert ring.dtype == torch.float32 and first_col + C <= proj.shape[1]
+    _check(lib().fd_conv_ring_update(_col_ptr(proj, first_col), proj.shape[1], _dt(proj.dtype), _ptr(ring), _ptr(row_slot),
+                                     _ptr(row_q_start), _ptr(row_q_len), _ptr(row_ctx_len), n_rows, C, taps, _stream()))
+
+
+def ssd_prepare(proj: torch.Tensor, col: int, dt_col: int, conv_w: torch.Tensor, conv_b: torch.Tensor, ring: Optional[torch.Tensor],
+                keep: bool, dt_bias: torch.Tensor, A_log: torch.Tensor, xbc: torch.Tensor, step: torch.Tensor, tok_row: torch.Tensor,
+                tok_pos: torch.Tensor, row_slot: torch.Tensor, row_q_start: torch.Tensor, row_q_len: torch.Tensor) -> None:
+    """``xbc`` float32 [T, C] <- silu of the causal convolution (``conv_w`` [C, taps], bias ``conv_b`` [C], float32; earlier
+    values from ``ring`` [slots, taps, C]) of the C columns of ``proj`` from ``col`` on; ``step`` float32 [T, heads, 2] <- (dt,
+    exp(-exp(A_log) dt)) with dt = softplus of the columns from ``dt_col`` on plus ``dt_bias``."""
+    T, C, H, taps = proj.shape[0], xbc.shape[1], dt_bias.numel(), conv_w.shape[1]
+    for t in (conv_w, conv_b, ring, dt_bias, A_log, xbc, step):
+        assert t is None or t.dtype == torch.float32
+    assert conv_w.shape == (C, taps) and conv_b.numel() == C and (taps == 1 or ring.shape[1:] == (taps, C))
+    assert xbc.shape[0] == T and step.shape == (T, H, 2) and A_log.numel() == H
+    _check(lib().fd_ssd_prepare(_ptr(proj), proj.shape[1], _dt(proj.dtype), col, C, dt_col, _ptr(conv_w), _ptr(conv_b), _ptr(ring),
+                                taps, int(keep), _ptr(dt_bias), _ptr(A_log), _ptr(xbc), _ptr(step), _ptr(tok_row), _ptr(tok_pos),
+                                _ptr(row_slot), _ptr(row_q_start), _ptr(row_q_len), T, H, _stream()))
+
+
+def ssd_gate_norm(y: torch.Tensor, xbc: torch.Tensor, D: torch.Tensor, proj: torch.Tensor, z_col: int, weight: torch.Tensor,
+                  out: torch.Tensor, first_col: int, parts: int, eps: float, scale: float = 1.0) -> None:
+    """out[t, first_col ...] = scale * weight * norm((y + D_h x) * silu(z)): x the first columns of ``xbc``, z the columns of ``proj``
+    from ``z_col`` on, the norm over each of ``parts`` equal parts.  ``y`` float32 [T, inner]; ``D`` float32, one per head."""
+    T, inner = y.shape
+    assert y.dtype == xbc.dtype == D.dtype == weight.dtype == torch.float32 and weight.numel() == inner and inner % D.numel() == 0
+    assert proj.dtype == out.dtype and z_col + inner <= proj.shape[1] and first_col + inner <= out.shape[1] and inner <= xbc.shape[1]
+    _check(lib().fd_ssd_gate_norm(_ptr(y), _ptr(xbc), xbc.shape[1], _ptr(D), _col_ptr(proj, z_col), proj.shape[1], _ptr(weight),
+                                  _col_ptr(out, first_col), out.shape[1], _dt(out.dtype), T, inner, inner // D.numel(), parts,
+                                  float(eps), float(scale), _stream()))
+
+
+VALUES_PLAIN, VALUES_SOURCE, VALUES_MIXED = 0, 1, 2
+
+
+def rope_norm_append(proj: torch.Tensor, first_col: int, q_out: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
+                     block_table: torch.Tensor, q_weight: Optional[torch.Tensor], k_weight: Optional[torch.Tensor], eps: float,
+                     cos: Optional[torch.Tensor], sin: Optional[torch.Tensor], rot_dims: int, head_norm: bool,
+                     tok_row: torch.Tensor, tok_pos: torch.Tensor, row_slot: torch.Tensor, n_q: int, n_kv: int, head_dim: int,
+                     v_head_dim: int, write_kv: bool, status: torch.Tensor, q_count: int = 0, k_count: int = 0, head_count: int = 0,
+                     value_mode: int = VALUES_PLAIN, v_first: Optional[torch.Tensor] = None, lam: Optional[torch.Tensor] = None) -> None:
+    """From the columns of ``proj`` from ``first_col`` on - q, k, v side by side - to ``q_out`` [T, n_q head_dim] and the paged
+    cache: q and k RMS-normed over their whole projections (``q_weight``, ``k_weight`` float32, or None: not), their first
+    ``rot_dims`` dimensions turned (i paired with i + rot_dims / 2), and by ``head_norm`` every head divided by its own root mean
+    square.  The means run over ``q_count`` / ``k_count`` / ``head_count`` values (0: all).  ``value_mode``: VALUES_SOURCE also leaves
+    the values in ``v_first`` [T, n_kv v_head_dim]; VALUES_MIXED stores (1 - lam) v + lam v_first, ``lam`` one float32."""
+    T = proj.shape[0]
+    num_blocks, _, block_size, _ = k_pool.shape
+    assert proj.dtype == q_out.dtype == k_pool.dtype == v_pool.dtype and q_out.shape == (T, n_q * head_dim)
+    assert k_pool.shape[1] == n_kv and k_pool.shape[3] == head_dim and v_pool.shape[3] == v_head_dim
+    assert first_col + (n_q + n_kv) * head_dim + n_kv * v_head_dim <= proj.shape[1]
+    assert q_weight is None or (q_weight.dtype == k_weight.dtype == torch.float32 and q_weight.numel() == n_q * head_dim
+                                and k_weight.numel() == n_kv * head_dim)
+    assert value_mode == VALUES_PLAIN or (v_first.dtype == proj.dtype and v_first.shape == (T, n_kv * v_head_dim))
+    assert value_mode != VALUES_MIXED or (lam.dtype == torch.float32 and lam.numel() == 1)
+    _check(lib().fd_rope_norm_append(
+        _col_ptr(proj, first_col), proj.shape[1], _dt(proj.dtype), _ptr(q_out), _ptr(k_pool), _ptr(v_pool), _ptr(v_first),
+        _ptr(q_weight), _ptr(k_weight), float(eps), _ptr(cos) if rot_dims else None, _ptr(sin) if rot_dims else None,
+        cos.shape[0] if rot_dims else 0, rot_dims, int(head_norm), value_mode, _ptr(lam), _ptr(tok_row), _ptr(tok_pos),
+        _ptr(row_slot), _ptr(block_table), block_table.shape[1], num_blocks, block_size, T, n_q, n_kv, head_dim, v_head_dim,
+        q_count or n_q * head_dim, k_count or n_kv * head_dim, head_count or head_dim, int(write_kv), _ptr(status), _stream()))
 
 
 # ---------------------------------------------------------------------------
@@ -1141,6 +1286,13 @@ def relu2(x: torch.Tensor, out: torch.Tensor) -> None:
     """out = max(x, 0)^2."""
     assert x.shape == out.shape and x.dtype == out.dtype
     _check(lib().fd_relu2(_ptr(x), _ptr(out), _dt(x.dtype), x.numel(), _stream()))
+
+
+def relu2_cols(x: torch.Tensor, x_col: int, out: torch.Tensor, out_col: int, n_cols: int) -> None:
+    """out[:, out_col ...] = max(x[:, x_col ...], 0)^2 for ``n_cols`` columns; one rounding."""
+    assert x.dtype == out.dtype and x.shape[0] == out.shape[0] and x_col + n_cols <= x.shape[1] and out_col + n_cols <= out.shape[1]
+    _check(lib().fd_relu2_cols(_col_ptr(x, x_col), x.shape[1], _col_ptr(out, out_col), out.shape[1], _dt(x.dtype), x.shape[0],
+                               n_cols, _stream()))
 
 
 def moe_tile_rows(dtype: torch.dtype = torch.float32, n_pairs: int = 0, n_experts: int = 1, k_sizes=()) -> int:

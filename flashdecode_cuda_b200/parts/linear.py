@@ -98,3 +98,19 @@ def matmul(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out: 
         if bias is not None:
             out.add_(bias.to(out.dtype))
     return out
+
+
+NARROW_PRODUCT_ROWS = 128      # bfloat16 steps of more tokens expand narrow vectors with a product of their own
+
+
+def narrow_product(ctx, proj: torch.Tensor, first_col: int, w: torch.Tensor, name: Optional[str],
+                   out: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+    """x w^T as float32 [T, N] for x = the columns of ``proj`` from ``first_col`` on, as many as w [N, R] has - a low-rank
+    projection's second matrix - in a bfloat16 step of more than ``NARROW_PRODUCT_ROWS`` tokens; None for any other
+    step, whose consumer expands the vector itself.  ``out`` (else workspace memory called ``name``): where it goes."""
+    if proj.dtype != torch.bfloat16 or proj.shape[0] <= NARROW_PRODUCT_ROWS:
+        return None
+    if out is None:
+        out = ctx.ws.get(name, (proj.shape[0], w.shape[0]), torch.float32)
+    torch.mm(proj[:, first_col:first_col + w.shape[1]], w.t(), out_dtype=torch.float32, out=out)
+    return out

@@ -150,42 +150,73 @@ class GatedMLP(FeedForward):
 
 @register_part("feed_forward", "dense_act")
 class DenseActMLP(FeedForward):
-    """down( act(up(x)) ), no gate and no biases, with the two-parameter activation ``quad_exp``:
+    """down( act(up(x)) ), no gate and no biases.  ``activation`` ``relu2``: max(z, 0)^2; ``quad_exp``, with two parameters:
 
         act(z) = softplus(p) z^2 + z / 2                          for z > 0
                  (1/2 + softplus(q)) (exp(z) - 1 - z) + z / 2     for z <= 0
 
     (p, q) are the tensor ``<prefix>.act`` [2].  Tensors ``<prefix>.up`` / ``.down`` (stored [out, in]).  The
-    activation is computed in float32 and rounded once."""
+    activation is computed in float32 and rounded once.  With ``relu2`` it can be a branch beside mixers that read the
+    same input (``parts.parallel``): up rides in their packed input product, down in their output product."""
+
+    out_name = "down"
 
     def __init__(self, prefix: str, hidden_size: int, intermediate_size: int, activation: str = "quad_exp"):
-        if activation != "quad_exp":
-            raise ValueError(f"{prefix}: unknown activation {activation!r}; known: quad_exp")
+        if activation not in ("quad_exp", "relu2"):
+            raise ValueError(f"{prefix}: unknown activation {activation!r}; known: quad_exp, relu2")
         self.prefix, self.hidden_size, self.inter, self.activation = prefix, hidden_size, intermediate_size, activation
 
     def tensor_specs(self) -> List[TensorSpec]:
         p, H, I = self.prefix, self.hidden_size, self.inter
-        return [TensorSpec(f"{p}.up", (I, H), init="unit"), TensorSpec(f"{p}.down", (H, I), init="unit"),
-                TensorSpec(f"{p}.act", (2,), "vector", init="half")]
+        specs = [TensorSpec(f"{p}.up", (I, H), init="unit"), TensorSpec(f"{p}.down", (H, I), init="unit")]
+        if self.activation == "quad_exp":
+            specs.append(TensorSpec(f"{p}.act", (2,), "vector", init="half"))
+        return specs
 
     def bind(self, tensors: Dict[str, torch.Tensor], rt: Runtime) -> None:
         self.rt = rt
         p = self.prefix
-        self.w_up, self.w_down = tensors[f"{p}.up"], tensors[f"{p}.down"]
-        self.pq = tensors.pop(f"{p}.act").float().contiguous()
+        self.w_in, self.w_o = tensors[f"{p}.up"], tensors[f"{p}.down"]
+        self.pq = tensors.pop(f"{p}.act").float().contiguous() if self.activation == "quad_exp" else None
 
     def weight_bytes(self) -> int:
-        return (self.w_up.numel() + self.w_down.numel()) * self.w_down.element_size()
+        return sum(w.numel() * w.element_size() for w in (self.w_in, self.w_o) if w is not None)
 
     def first_weights(self) -> Optional[torch.Tensor]:
-        return self.w_up
+        return self.w_in
+
+    # --- as a branch beside mixers ----------------------------------------
+    @property
+    def shares_products(self) -> bool:
+        return self.activation == "relu2"
+
+    def kv_request(self):
+        return None
+
+    def state_requests(self) -> list:
+        return []
+
+    def in_proj(self):
+        return self.w_in, None
+
+    def out_proj(self) -> torch.Tensor:
+        return self.w_o
+
+    def inner(self, ctx, proj: torch.Tensor, col0: int, lc, act: torch.Tensor, act_col: int = 0, scale: float = 1.0) -> torch.Tensor:
+        if scale != 1.0:
+            raise ValueError(f"{self.prefix}: this feed-forward enters a sum with the weight 1 only")
+        K.relu2_cols(proj, col0, act, act_col, self.inter)
+        return act
 
     def forward(self, ctx, x: torch.Tensor, parts_ok: bool = False) -> torch.Tensor:
         T, ws = ctx.T, ctx.ws
         up = ws.get("ffn_up", (T, self.inter), x.dtype)
-        matmul(x, self.w_up, None, up, status=self.rt.status)
+        matmul(x, self.w_in, None, up, status=self.rt.status)
         act = ws.get("ffn_act", (T, self.inter), x.dtype)
-        K.quad_exp_act(up, self.pq, act)
+        if self.activation == "relu2":
+            K.relu2(up, act)
+        else:
+            K.quad_exp_act(up, self.pq, act)
         out = ws.get("ffn_out", (T, self.hidden_size), x.dtype)
-        return matmul(act, self.w_down, None, out, target_ctas=4 * self.rt.sm_count, status=self.rt.status,
+        return matmul(act, self.w_o, None, out, target_ctas=4 * self.rt.sm_count, status=self.rt.status,
                       upcoming=ctx.upcoming)

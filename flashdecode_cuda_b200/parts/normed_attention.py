@@ -16,10 +16,11 @@ from .base import KVRequest, LayerCache, Mixer, Runtime
 from .linear import matmul
 
 
-def decode_splits(ctx, n_q: int, n_kv: int, v_dim: int, dtype: torch.dtype, rt: Runtime, head_dim: int = 0):
+def decode_splits(ctx, n_q: int, n_kv: int, v_dim: int, dtype: torch.dtype, rt: Runtime, head_dim: int = 0, window: int = 0):
     """(n_splits, split_len, scratch) of a step's attention: a step of single tokens cuts every sequence's keys into
     splits (float32: of a fixed length, so that where a sequence's partial sums are cut depends on its own length only;
-    bfloat16: by the batch's size); any other step does not."""
+    bfloat16: by the batch's size and, if ``window`` is given, for the keys it shows, so that the CTAs that find keys are
+    about as many as the SMs); any other step does not."""
     if ctx.max_q_len != 1:
         return 1, 0, None
     if dtype == torch.float32:
@@ -28,7 +29,12 @@ def decode_splits(ctx, n_q: int, n_kv: int, v_dim: int, dtype: torch.dtype, rt: 
     else:
         # (the tensor-core kernel cuts a large group of query heads into several, each with CTAs of its own)
         heads = K.attention_decode_heads(n_q, n_kv, head_dim, v_dim) if head_dim else n_kv
-        n_splits, split_len = plan_splits(ctx.n_rows, heads, ctx.kv_len_bound, rt.sm_count)
+        bound = ctx.kv_len_bound
+        n_splits, split_len = plan_splits(ctx.n_rows, heads, min(bound, window + 32) if window else bound, rt.sm_count)
+        n_splits = max(1, -(-bound // split_len))
+        if window and n_splits > 64:                # bounded scratch memory and merge
+            split_len = -(-(-(-bound // 64)) // 32) * 32
+            n_splits = -(-bound // split_len)
     scratch = None
     if n_splits > 1:
         scratch = ctx.ws.get("attn_scratch", (K.attention_scratch_floats(ctx.T, n_q, v_dim, n_splits),), torch.float32)
@@ -37,6 +43,16 @@ def decode_splits(ctx, n_q: int, n_kv: int, v_dim: int, dtype: torch.dtype, rt: 
 
 def _up8(n: int) -> int:
     return -(-n // 8) * 8
+
+
+def tensor_core_sizes(head_dim: int, v_head_dim: int):
+    """(key, value) head sizes as the kernels should see them: both 64 or both 128, which the tensor-core attention kernels
+    take, where filling up with zeros costs at most 60 % more of the cache; else the next multiples of 8."""
+    widest = max(head_dim, v_head_dim)
+    size = 64 if widest <= 64 else 128
+    if widest <= 128 and 2 * size <= 1.6 * (head_dim + v_head_dim):
+        return size, size
+    return _up8(head_dim), _up8(v_head_dim)
 
 
 def _head_sizes_ok(prefix: str, **sizes: int) -> None:
@@ -82,22 +98,38 @@ def _pad_split_heads(w: torch.Tensor, n_heads: int, *parts) -> torch.Tensor:
 class QKNormedAttention(Mixer):
     """For the mixer's input h [T, hidden]:
 
-        q, k, v = W_q h, W_k h, W_v h                           (no biases)
+        q, k, v = W_q h, W_k h, W_v h                           (``bias``: + ``.q.b``, ``.k.b``, ``.v.b``)
         q       = q / sqrt(mean(q^2) + eps) * w_q               over ALL of q's n_heads * head_dim values at once,
         k       = k / sqrt(mean(k^2) + eps) * w_k               likewise; then both are split into heads
+        q, k    = rotation of every head's first ``rot_dims`` dimensions (i paired with i + rot_dims / 2), if any
+        q, k    = x / sqrt(mean(x^2) + eps) per head, without a weight                  (``head_norm``)
+        v       = (1 - lam) v + lam v_first                     (``value_mix``, below)
         a       = softmax over the visible keys of (q . k) * scale; query head h reads key/value head
                   h // (n_heads / n_kv_heads); value heads have ``v_head_dim`` dimensions
         out     = W_o a
 
-    Nothing is rotated: positions enter through visibility alone.  Visible keys of the query at position i: j <= i,
-    and with a ``window`` only i - j < window.  ``qk_norm`` False: q and k are used as projected.  One packed
+    Without ``rot_dims`` positions enter through visibility alone.  Visible keys of the query at position i: j <= i,
+    and with a ``window`` only i - j < window.  ``qk_norm`` False: q and k are used as projected.  ``softcap``: score <-
+    softcap * tanh(score / softcap) after scaling.  ``sink``: exp(``.sink``[h]) is one more term of head h's denominator,
+    without key or value.  ``value_mix``: "source" leaves the layer's values of the step's tokens for other layers,
+    "mix" mixes them into its own values with lam = ``.vmix`` before they are cached; ``value_group`` names what they
+    share.  One packed
     product gives q, k and v.  Tensors ``<prefix>.q`` / ``.k`` / ``.v`` / ``.o`` (stored [out, in]), ``.q.norm``,
-    ``.k.norm``.  The norms are float32 in both dtypes.
+    ``.k.norm``.  Norms, rotation, scores, softmax and mixing are float32 in both dtypes.  Other mixers, or a feed-forward,
+    may share its input and output products (``parts.parallel``).
     """
 
+    shares_products = True
+
     def __init__(self, prefix: str, hidden_size: int, n_heads: int, n_kv_heads: int, head_dim: int, v_head_dim: int,
-                 scale: float, eps: float, window: Optional[int] = None, qk_norm: bool = True):
+                 scale: float, eps: float, window: Optional[int] = None, qk_norm: bool = True, bias: bool = False,
+                 position=None, rot_dims: int = 0, head_norm: bool = False, softcap: Optional[float] = None, sink: bool = False,
+                 value_mix: Optional[str] = None, value_group: str = "values"):
         _head_sizes_ok(prefix, head_size=head_dim, value_head_size=v_head_dim)
+        if rot_dims < 0 or rot_dims % 2 or rot_dims > head_dim or (rot_dims and position is None):
+            raise ValueError(f"{prefix}: {rot_dims} rotated dimensions of {head_dim}: they must be even and given a position part")
+        if value_mix not in (None, "source", "mix") or (softcap is not None and not softcap > 0):
+            raise ValueError(f"{prefix}: value mixing {value_mix!r} (None, 'source' or 'mix'), a soft cap of {softcap} (positive or None)")
         if n_kv_heads < 1 or n_heads % n_kv_heads != 0 or n_heads // n_kv_heads > 64:
             raise ValueError(f"{prefix}: {n_heads} query heads for {n_kv_heads} key/value heads: the kernels take whole "
                              f"groups of up to 64 query heads per key/value head")
@@ -105,8 +137,14 @@ class QKNormedAttention(Mixer):
             raise ValueError(f"{prefix}: a window of {window} positions")
         self.prefix, self.hidden_size = prefix, hidden_size
         self.n_q, self.n_kv, self.d, self.dv = n_heads, n_kv_heads, head_dim, v_head_dim
-        self.dp, self.dvp = _up8(head_dim), _up8(v_head_dim)         # head sizes as the kernels see them
+        # head sizes as the kernels see them
+        self.dp, self.dvp = tensor_core_sizes(head_dim, v_head_dim)
         self.scale, self.eps, self.window, self.qk_norm = float(scale), float(eps), window, qk_norm
+        self.bias, self.position, self.rot_dims, self.head_norm = bool(bias), position, int(rot_dims), bool(head_norm)
+        self.softcap, self.has_sink, self.value_mix, self.value_group = softcap, bool(sink), value_mix, value_group
+        self.extended = bool(softcap or sink)
+        # what the plain append kernel does not have
+        self.turned = bool(rot_dims or head_norm or value_mix)
 
     def _sizes(self):
         return (("q", self.n_q * self.d), ("k", self.n_kv * self.d), ("v", self.n_kv * self.dv))
@@ -117,6 +155,12 @@ class QKNormedAttention(Mixer):
         if self.qk_norm:
             specs += [TensorSpec(f"{p}.q.norm", (self.n_q * self.d,), "vector", init="norm"),
                       TensorSpec(f"{p}.k.norm", (self.n_kv * self.d,), "vector", init="norm")]
+        if self.bias:
+            specs += [TensorSpec(f"{p}.{n}.b", (c,), "vector", init="bias") for n, c in self._sizes()]
+        if self.has_sink:
+            specs.append(TensorSpec(f"{p}.sink", (self.n_q,), "vector", init="sink"))
+        if self.value_mix:          # (the source's own constant is never read)
+            specs.append(TensorSpec(f"{p}.vmix", (), "vector", optional=self.value_mix == "source", init="half"))
         specs.append(TensorSpec(f"{p}.o", (H, self.n_q * self.dv), init="unit"))
         return specs
 
@@ -128,6 +172,11 @@ class QKNormedAttention(Mixer):
         p = self.prefix
         heads = {"q": (self.n_q, self.d, self.dp), "k": (self.n_kv, self.d, self.dp), "v": (self.n_kv, self.dv, self.dvp)}
         self.w_in = torch.cat([_pad_heads(tensors.pop(f"{p}.{n}"), *heads[n]) for n, _ in self._sizes()], dim=0).contiguous()
+        self.b_in = None
+        if self.bias:
+            self.b_in = torch.cat([_pad_heads(tensors.pop(f"{p}.{n}.b"), *heads[n]) for n, _ in self._sizes()]).contiguous()
+        self.sink_w = tensors.pop(f"{p}.sink").float().contiguous() if self.has_sink else None
+        self.lam = tensors.pop(f"{p}.vmix").float().reshape(1).contiguous() if self.value_mix == "mix" else None
         self.q_norm = self.k_norm = None
         if self.qk_norm:
             self.q_norm = _pad_heads(tensors[f"{p}.q.norm"].float(), *heads["q"]).contiguous()
@@ -139,24 +188,52 @@ class QKNormedAttention(Mixer):
         self.w_o = w_o
 
     def weight_bytes(self) -> int:
-        return self.w_in.numel() * self.w_in.element_size() + self.w_o.numel() * self.w_o.element_size()
+        return sum(w.numel() * w.element_size() for w in (self.w_in, self.w_o) if w is not None)
 
     def first_weights(self) -> Optional[torch.Tensor]:
         return self.w_in
 
+    def in_proj(self):
+        return self.w_in, self.b_in
+
+    def out_proj(self) -> torch.Tensor:
+        return self.w_o
+
+    def inner(self, ctx, proj: torch.Tensor, col0: int, lc: LayerCache, act: torch.Tensor, act_col: int = 0,
+              scale: float = 1.0) -> torch.Tensor:
+        T, ws, rt = ctx.T, ctx.ws, self.rt
+        q = ws.get("nat_q", (T, self.n_q * self.dp), proj.dtype)
+        counts = dict(q_count=self.n_q * self.d, k_count=self.n_kv * self.d)
+        if self.turned or col0:
+            v_first = None
+            if self.value_mix:
+                v_first = ws.get(f"first_{self.value_group}", (T, self.n_kv * self.dvp), proj.dtype)
+            mode = {None: K.VALUES_PLAIN, "source": K.VALUES_SOURCE, "mix": K.VALUES_MIXED}[self.value_mix]
+            rope = self.position
+            K.rope_norm_append(proj, col0, q, lc.k_pool, lc.v_pool, lc.group.table, self.q_norm, self.k_norm, self.eps,
+                               rope.cos if self.rot_dims else None, rope.sin if self.rot_dims else None, self.rot_dims,
+                               self.head_norm, ctx.tok_row, ctx.tok_pos, ctx.row_slot, self.n_q, self.n_kv, self.dp, self.dvp,
+                               lc.writes, rt.status, head_count=self.d, value_mode=mode, v_first=v_first, lam=self.lam, **counts)
+        else:
+            K.norm_append(proj, q, self.q_norm, self.k_norm, self.eps, ctx.tok_row, ctx.tok_pos, ctx.row_slot, lc.k_pool,
+                          lc.v_pool, lc.group.table, self.n_kv, lc.writes, rt.status, **counts)
+        n_splits, split_len, scratch = decode_splits(ctx, self.n_q, self.n_kv, self.dvp, proj.dtype, rt, self.dp,
+                                                     (self.window or 0) if self.turned else 0)
+        args = (q, lc.k_pool, lc.v_pool, act, lc.group.table, ctx.tok_row, ctx.row_slot, ctx.row_q_start, ctx.row_q_len,
+                ctx.row_ctx_len, ctx.n_rows, ctx.max_q_len, self.n_q, self.n_kv, self.dp, self.scale, self.window or 0, n_splits,
+                split_len, scratch, rt.status)
+        if self.extended:
+            K.attention_ext(*args, softcap=self.softcap or 0.0, sink=self.sink_w, out_col=act_col, out_scale=scale)
+        else:
+            K.attention(*args, out_col=act_col, out_scale=scale)
+        return act
+
     def forward(self, ctx, x: torch.Tensor, lc: LayerCache) -> torch.Tensor:
         T, ws, rt = ctx.T, ctx.ws, self.rt
         proj = ws.get("nat_proj", (T, self.w_in.shape[0]), x.dtype)
-        matmul(x, self.w_in, None, proj, status=rt.status)
-        q = ws.get("nat_q", (T, self.n_q * self.dp), x.dtype)
-        K.norm_append(proj, q, self.q_norm, self.k_norm, self.eps, ctx.tok_row, ctx.tok_pos, ctx.row_slot, lc.k_pool,
-                      lc.v_pool, lc.group.table, self.n_kv, lc.writes, rt.status, q_count=self.n_q * self.d,
-                      k_count=self.n_kv * self.d)
+        matmul(x, self.w_in, self.b_in, proj, status=rt.status)
         attn = ws.get("nat_attn", (T, self.n_q * self.dvp), x.dtype)
-        n_splits, split_len, scratch = decode_splits(ctx, self.n_q, self.n_kv, self.dvp, x.dtype, rt, self.dp)
-        K.attention(q, lc.k_pool, lc.v_pool, attn, lc.group.table, ctx.tok_row, ctx.row_slot, ctx.row_q_start,
-                    ctx.row_q_len, ctx.row_ctx_len, ctx.n_rows, ctx.max_q_len, self.n_q, self.n_kv, self.dp, self.scale,
-                    self.window or 0, n_splits, split_len, scratch, rt.status)
+        self.inner(ctx, proj, 0, lc, attn)
         out = ws.get("mixer_out", (T, self.hidden_size), x.dtype)
         return matmul(attn, self.w_o, None, out, target_ctas=4 * rt.sm_count, status=rt.status)
 

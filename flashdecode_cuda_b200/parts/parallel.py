@@ -23,8 +23,9 @@ class ParallelMixers(Mixer):
     are run as ONE input product over the stacked input matrices, each branch's inner work on its columns, and ONE
     output product over the branches' activations laid side by side with the stacked output matrices:
     sum_b scale_b W_b a_b = [W_1 | W_2 | ...] [scale_1 a_1 ; scale_2 a_2 ; ...].  The scale enters each branch's
-    activations in float32 before their one rounding.  Other branches run whole, and the weighted sum of the outputs is
-    taken in float32.  At most one branch may keep keys; every branch's per-sequence state is kept under
+    activations in float32 before their one rounding.  A feed-forward that reads the same input as the mixers is one more
+    such branch.  A branch's activations start at a multiple of 8 columns, and the row's length is a multiple of 32 (columns
+    of zeros fill up).  Other branches run whole, and the weighted sum of the outputs is taken in float32.  At most one branch may keep keys; every branch's per-sequence state is kept under
     ``<name>.<its own name>``."""
 
     def __init__(self, prefix: str, branches: Sequence[Mixer], names: Sequence[str], scales: Sequence[float],
@@ -68,20 +69,31 @@ class ParallelMixers(Mixer):
             self.b_in = torch.cat([bias.float() if bias is not None
                                    else torch.zeros(w.shape[0], dtype=torch.float32, device=w.device)
                                    for w, bias in ins]).contiguous()
-        self.w_o = torch.cat([b.out_proj() for b in self.branches], dim=1).contiguous()
-        self.in_cols, self.act_cols = [], []
+            if rt.dtype == torch.bfloat16 and torch.equal(self.b_in.to(torch.bfloat16).float(), self.b_in):
+                self.b_in = self.b_in.to(torch.bfloat16)         # as stored: the library product then adds it in its epilogue
+        self.in_cols, self.act_cols, self.gaps = [], [], []
         c = a = 0
+        outs = [b.out_proj() for b in self.branches]
+        cols = []                                   # the stacked output matrix: the branches' columns and the zeros between
+        for i, w in enumerate(outs):
+            n = w.shape[1]
+            unit = 32 if i + 1 == len(outs) else 8
+            fill = -(a + n) % unit
+            cols += [w] + ([w.new_zeros((w.shape[0], fill))] if fill else [])
+            self.act_cols.append(a)
+            if fill:
+                self.gaps.append((a + n, a + n + fill))
+            a += n + fill
+        self.w_o = torch.cat(cols, dim=1).contiguous()
+        self.n_act = a
         for b, (w, _) in zip(self.branches, ins):
             self.in_cols.append(c)
-            self.act_cols.append(a)
             # the branch keeps views of the stacked matrices instead of copies of its own (rows of w_in are
             # contiguous; its columns of w_o are not, so alone it can no longer run)
             b.w_in = self.w_in[c:c + w.shape[0]]
             c += w.shape[0]
-            a += b.out_proj().shape[1]
             b.w_o = None
-            tensors.pop(f"{b.prefix}.o", None)
-        self.n_act = a
+            tensors.pop(f"{b.prefix}.{getattr(b, 'out_name', 'o')}", None)
 
     def weight_bytes(self) -> int:
         if not self.fused:
@@ -103,6 +115,8 @@ class ParallelMixers(Mixer):
             proj = ws.get("par_proj", (T, self.w_in.shape[0]), x.dtype)
             matmul(x, self.w_in, self.b_in, proj, status=rt.status)
             act = ws.get("par_act", (T, self.n_act), x.dtype)
+            for lo, hi in self.gaps:
+                act[:, lo:hi].zero_()
             for i, b in enumerate(self.branches):
                 b.inner(ctx, proj, self.in_cols[i], self._sub(lc, i), act, self.act_cols[i], self.scales[i])
             out = ws.get("mixer_out", (T, self.hidden_size), x.dtype)

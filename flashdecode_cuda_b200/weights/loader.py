@@ -127,6 +127,8 @@ def random_tensor(spec: TensorSpec, seed: int, dtype: torch.dtype, device="cpu")
             t = torch.sigmoid(t)
         elif spec.init == "decay_bias":         # pre-activation of a decay near one: sigmoid(2 + N(0, 1))
             t = 2.0 + t
+        elif spec.init == "step_bias":           # pre-activation of a step size: softplus(-2 + N(0, 1)), about 0.1
+            t = t - 2.0
         elif spec.init == "unit_rows":          # rows of a lookup table whose entries multiply activations: about one
             pass
         elif spec.init == "conv_small":          # a convolution that is added to its own input

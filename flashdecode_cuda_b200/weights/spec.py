@@ -19,7 +19,7 @@ class TensorSpec:
     N(0, 1 / fan-in) (products that keep their input's scale), ``bias`` N(0, 0.02),
     ``lane_read`` 1 / n + N(0, 0.1), ``lane_mix`` the unit matrix + N(0, 0.1), ``half`` 0.5 + N(0, 0.1),
     ``sink`` N(0, 0.5), ``unit_interval`` sigmoid(N(0, 1)), ``unit_rows`` N(0, 1),
-    ``decay_bias`` 2 + N(0, 1), ``depth`` N(0, 0.1) and one more on the last, ``conv_small`` N(0, 0.2), ``zeros``."""
+    ``decay_bias`` 2 + N(0, 1), ``step_bias`` -2 + N(0, 1) (a softplus of about 0.1), ``depth`` N(0, 0.1) and one more on the last, ``conv_small`` N(0, 0.2), ``zeros``."""
 
     name: str
     shape: Tuple[int, ...]
