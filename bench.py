@@ -34,7 +34,8 @@ attention with a rotated key part and lightning attention, routed feed-forwards,
 depth) beside the Nizazen design at equal sizes.  ``--compare botusun`` measures the Botusun design (six
 layers, two of them twice: linear attention with a decay per key channel and windowed attention over convolved, normed keys, dense and routed
 feed-forwards, a contribution of the token itself after every layer) beside the Revelix design at equal sizes.  ``--compare revelix`` for the Revelix design (eight layers that alternate retention and attention beside a gated
-recurrence, each with a dense feed-forward).  ``--compare lonasun`` leaves all of that aside and measures the Lonasun design beside the Qwen2 dense decoder of the
+recurrence, each with a dense feed-forward), ``--compare bifatar`` for the Bifatar design (eight layers of state-space mixers,
+attention beside a delta rule and capped attention, each with its feed-forward beside the mixer) beside the Revelix design.  ``--compare lonasun`` leaves all of that aside and measures the Lonasun design beside the Qwen2 dense decoder of the
 same width, heads, layer runs and feed-forward work per token (random weights, a window as long as Lonasun's chunk):
 prefill and decode throughput of both at a few layer sizes, and for every mixer and feed-forward the device time of
 its kernels against the least time its operations and bytes need at the measured peaks.  It prints one JSON line of
@@ -450,10 +451,32 @@ def gulozen_configs(sz: dict):
     return gulo, niza
 
 
+def bifatar_configs(sz: dict):
+    """(Bifatar config dictionary, Revelix config dictionary) of equal width and layers.  Bifatar: eight layers in the order
+    state-space mixer, attention beside a delta rule, capped windowed attention, each with a feed-forward beside its mixer.
+    Beside it the closest design the library has, Revelix at the sizes of ``--compare revelix``: the same attention heads, head
+    size and window, delta rules of the same heads and state as its gated recurrences, state-space mixers with as many
+    state elements as its retention layers, and feed-forwards of the same size."""
+    reve, _ = revelix_configs(sz)
+    rot = {"base": 1000000.0, "dims": sz["rot"]}
+    heads = {"dim": sz["dim"], "heads": sz["heads"], "kv_heads": sz["kv"], "rot": rot, "scale": sz["dim"] ** -0.5, "vdim": sz["dim"]}
+    att = dict(heads, mask={"size": sz["window"]}, softcap=50.0, v_mix=True, scale=1.0)
+    ssm = {"conv": 4, "groups": 2, "heads": sz["ret_heads"] * sz["ret_dim"] * sz["ret_vdim"] // (64 * 128), "norm_groups": 2,
+           "state": 128, "vdim": 64}
+    right = {"conv": 4, "dim": sz["rec_dim"], "heads": sz["rec_heads"], "kv_heads": sz["rec_heads"], "vdim": sz["rec_vdim"],
+             "rank": sz["rec_dim"]}
+    par = {"left": heads, "right": right, "left_scale": 1.0, "right_scale": 1.0}
+    mlp = {"ff": sz["ff"], "kind": "dense"}
+    kinds = ([("mamba2", ssm), ("parallel", par), ("attention", att)] * 3)[:8]
+    bifa = {"architecture": "Bifatar", "vocab": COMPARE_VOCAB, "width": sz["width"], "norm": {"eps": 1e-5},
+            "layers": [{"type": t, "mixer": m, "mlp": mlp} for t, m in kinds]}
+    return bifa, reve
+
+
 # design -> (sizes, function of a size that gives both configurations, the key of the model that stands beside it)
 COMPARISONS = {"lonasun": (COMPARE_SIZES, compare_configs, "qwen2"), "nizazen": (NIZAZEN_SIZES, nizazen_configs, "qwen2"),
                "revelix": (REVELIX_SIZES, revelix_configs, "qwen2"), "botusun": (REVELIX_SIZES, botusun_configs, "revelix"),
-               "gulozen": (GULOZEN_SIZES, gulozen_configs, "nizazen")}
+               "gulozen": (GULOZEN_SIZES, gulozen_configs, "nizazen"), "bifatar": (REVELIX_SIZES, bifatar_configs, "revelix")}
 
 
 def compare_one(cfgd: dict, pk: dict, batch: int, context: int, prompt: int, steps: int, warmup: int, seed: int) -> dict:
@@ -577,8 +600,14 @@ def compare_main(args) -> int:
             "prefill_tok_s": round(entry[design]["prefill"]["tok_s"] / entry[beside]["prefill"]["tok_s"], 3),
             "decode_tok_s": round(entry[design]["decode"]["tok_s"] / entry[beside]["decode"]["tok_s"], 3)}
         for phase in ("prefill", "decode"):
-            for part in ("mixer", "feed_forward"):
-                a, b = entry[design][phase]["parts"][part], entry[beside][phase]["parts"][part]
+            ours_parts, its_parts = entry[design][phase]["parts"], entry[beside][phase]["parts"]
+            if "feed_forward" not in ours_parts:           # feed-forwards that ride in the mixers' products: both together
+                for parts in (ours_parts, its_parts):
+                    both = [parts[k] for k in ("mixer", "feed_forward") if k in parts]
+                    ms, need = sum(p["ms"] for p in both), sum(p["roofline_ms"] for p in both)
+                    parts["layer"] = {"ms": round(ms, 4), "roofline_ms": round(need, 4), "frac": round(need / ms, 4)}
+            for part in ("mixer", "feed_forward") if "feed_forward" in ours_parts else ("layer",):
+                a, b = ours_parts[part], its_parts[part]
                 entry["ratios"][f"{phase}_{part}_frac"] = [a["frac"], b["frac"], round(a["frac"] / b["frac"], 3)]
         sizes[name] = entry
     print(json.dumps({"compare": design, "beside": {"qwen2": "Qwen2ForCausalLM", "revelix": "Revelix", "nizazen": "Nizazen"}[beside], "dtype": "bf16", "data": "synthetic: random weights",
@@ -797,7 +826,7 @@ def main() -> int:
     ap.add_argument("--no-fp32", action="store_true", help="skip the float32 point (slow at the larger presets)")
     ap.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"],
                     help="float32: the main run through the true 32-bit path (with --no-points)")
-    ap.add_argument("--compare", default="", choices=["", "lonasun", "nizazen", "revelix", "botusun", "gulozen"],
+    ap.add_argument("--compare", default="", choices=["", "lonasun", "nizazen", "revelix", "botusun", "gulozen", "bifatar"],
                     help="measure this design beside the closest dense model at equal sizes instead of the default run")
     ap.add_argument("--compare-sizes", default="", help="with --compare: names of the sizes to run, with commas (default: all)")
     ap.add_argument("--device", default="cuda", choices=["cuda", "cpu"],

@@ -10,7 +10,15 @@
 //  * delta_scan: the recurrence.  A CTA of 128 threads takes one sequence of the step, one head and 16 value columns; 8
 //    adjacent lanes share a column and each holds NR adjacent rows of it in registers.  Tokens come to shared memory a chunk
 //    ahead with cp.async.  Per token the lanes add up S^T k and S^T q of the decayed state with shuffles that run side
-//    by side; the read-out after the write is o = S^T q + (k . q) u, with k . q worked out once per token and chunk.
+//    by side; the read-out after the write is o = S^T q + (k . q) u, with k . q added up beside them.
+//    Rows of up to DR_SINGLE tokens only; longer ones:
+//  * delta_blocks and delta_block_scan: four tokens at a time.  With c_i the product of the block's decays up to token i, the
+//    corrections of a block follow from S^T (c_i k_i) alone and from products of the block's own keys,
+//        u_i = beta_i (v_i - S^T (c_i k_i) - sum_(j<i) A_ij u_j),      o_i = S^T (c_i q_i) + sum_(j<=i) P_ij u_j,
+//        S <- c_4 S + sum_j (g_(j+1) .. g_4 k_j) u_j^T,     A_ij = sum_c k_i k_j g_(j+1) .. g_i,  P_ij the same with q_i,
+//    in which decays are only multiplied, never divided.  The first kernel leaves the 13 vectors and 16 products of
+//    every block (nothing in it depends on the state); the second walks the blocks, one reduction over the lanes per block
+//    instead of one per token, two value columns per thread, blocks three ahead on their way with cp.async.
 //  * conv_ring_update: after a step with longer portions, the last values of every row go to its ring.
 //
 // State, decays, step sizes, unit vectors, sums: float.  A sequence's tokens are walked in order, so the sums of every
@@ -27,6 +35,9 @@ constexpr int DR_THREADS = 128;
 constexpr int DR_DS = 8;                       // lanes that share a column
 constexpr int DR_VT = DR_THREADS / DR_DS;      // value columns of a CTA
 constexpr int DR_TC = 16;                      // tokens of a chunk
+constexpr int DR_SINGLE = 16;                  // the most tokens of a row that is walked token by token
+constexpr int DB_THREADS = 64;                 // block form: 8 lanes share two columns
+constexpr int DB_TOK = 4, DB_VECS = 13, DB_SCAL = 20, DB_STAGES = 4;
 
 struct DeltaParams {
     const void* proj; int ld;                  // [T, ld]
@@ -78,7 +89,8 @@ __device__ __forceinline__ void expand_row(const T* __restrict__ w, const float*
 }
 
 // grid (token tiles, units): q heads, k heads, v heads, decay heads, gate heads
-template <typename T>
+// NARROW: decay heads (and gate heads, if any) expand their narrow vectors here
+template <typename T, bool NARROW>
 __global__ void __launch_bounds__(256)
 delta_prepare_kernel(const DeltaParams p) {
     __shared__ ConvMeta meta;
@@ -142,13 +154,13 @@ delta_prepare_kernel(const DeltaParams p) {
     const int h = is_gate ? u - p.H : u;
     const int R = is_gate ? p.R2 : p.R, col = is_gate ? p.g_col : p.a_col;
     const T* w = static_cast<const T*>(is_gate ? p.g2 : p.a2);
-    if (w != nullptr)
+    if (NARROW && w != nullptr)
         for (int e = tid; e < SC_TOK * R; e += blockDim.x) {
             const int tt = e / R, r = e - tt * R;
             x_s[e] = tt < nt ? to_float(proj[(size_t)(t0 + tt) * p.ld + col + r]) : 0.f;
         }
     __syncthreads();
-    if (is_gate) {
+    if (NARROW && is_gate) {
         for (int j = tid; j < p.dv; j += blockDim.x) {
             float z[SC_TOK];
             expand_row<T>(w + (size_t)(h * p.dv + j) * R, x_s, R, z);
@@ -163,7 +175,7 @@ delta_prepare_kernel(const DeltaParams p) {
     for (int j = tid; j < p.dp; j += blockDim.x) {
         float z[SC_TOK];
         const bool active = j < p.d;
-        if (active && w != nullptr) {
+        if (NARROW && active && w != nullptr) {
             expand_row<T>(w + (size_t)(h * p.d + j) * R, x_s, R, z);
         } else {
 #pragma unroll
@@ -182,7 +194,12 @@ struct DeltaScan {
     float* state; float* out;                  // [slots, H, d, dv], [T, H dv]
     const int* row_slot; const int* row_q_start; const int* row_q_len;
     int H, Hk, d, dv, dp, dvp, write_state;
+    float* blocks; float* scal;                // block form: [block slots, H, DB_VECS, dp], [block slots, H, DB_SCAL]; or null
+    int max_blocks;                            // blocks of the longest row
 };
+
+// Block b of step row r has the slot q_start / 4 + r + b: slots of different rows never meet.
+__device__ __forceinline__ int block_slot(int q_start, int r, int b) { return q_start / DB_TOK + r + b; }
 
 // floats of NR rows in shared memory: 4 apart from a multiple of 32 banks, so that the DS lanes of a column read different banks
 template <int NR> __host__ __device__ constexpr int dr_stride() { return NR == 4 ? 4 : NR + 4; }
@@ -191,15 +208,16 @@ template <int NR>
 __global__ void __launch_bounds__(DR_THREADS)
 delta_scan_kernel(const DeltaScan p) {
     constexpr int CS = DR_DS * dr_stride<NR>();              // floats of a token's k, q or g
-    constexpr int TS = 3 * CS + DR_VT + 4;                   // and of the token: k, q, g, v, [beta, k . q]
+    constexpr int TS = 3 * CS + DR_VT + 4;                   // and of the token: k, q, g, v, beta
     extern __shared__ __align__(16) float sm[];              // two chunks, filled in turn
     const int tiles = (p.dv + DR_VT - 1) / DR_VT;
     const int r = blockIdx.x / tiles, tile = blockIdx.x - r * tiles, h = blockIdx.y;
     const int slot = p.row_slot[r];
     if (slot < 0) return;
     const int q_start = p.row_q_start[r], q_len = p.row_q_len[r];
+    if (p.blocks != nullptr && q_len > DR_SINGLE) return;    // a row of the block form
     const int hk = h / (p.H / p.Hk);
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int tid = threadIdx.x;
     const int vl = tid / DR_DS, ds = tid % DR_DS;
     const int col = tile * DR_VT + vl;
     const bool live = col < p.dv;
@@ -220,18 +238,24 @@ delta_scan_kernel(const DeltaScan p) {
         const int n = min(DR_TC, q_len - c0);
         float* dst = sm + buf * DR_TC * TS;
         const int per = p.dp >> 2;                           // 16-byte pieces of a token's k, q or g
-        for (int e = tid; e < n * per * 3; e += DR_THREADS) {
-            const int which = e / (n * per), rest = e - which * n * per;
-            const int tt = rest / per, i = (rest - tt * per) * 4;
-            const size_t t = q_start + c0 + tt;
+        const size_t t = q_start + c0;
+        for (int piece = tid; piece < 3 * per; piece += DR_THREADS) {      // a thread's piece of every token of the chunk
+            const int which = piece >= 2 * per ? 2 : (piece >= per ? 1 : 0);
+            const int i = (piece - which * per) * 4;
             const float* src = which == 2 ? p.g + (t * p.H + h) * p.dp + i : (which == 1 ? p.q : p.k) + (t * p.Hk + hk) * p.dp + i;
-            cp_async16(smem_u32(dst + tt * TS + which * CS + (i / NR) * dr_stride<NR>() + i % NR), src, 16);
+            const size_t step = (size_t)(which == 2 ? p.H : p.Hk) * p.dp;
+            uint32_t at = smem_u32(dst + which * CS + (i / NR) * dr_stride<NR>() + i % NR);
+#pragma unroll 4
+            for (int tt = 0; tt < n; ++tt, src += step, at += TS * 4) cp_async16(at, src, 16);
         }
-        for (int e = tid; e < n * (DR_VT / 4); e += DR_THREADS) {
-            const int tt = e / (DR_VT / 4), i = (e - tt * (DR_VT / 4)) * 4;
-            const size_t t = q_start + c0 + tt;
+        if (tid < n * (DR_VT / 4)) {
+            const int tt = tid / (DR_VT / 4), i = (tid % (DR_VT / 4)) * 4;
             const bool in = tile * DR_VT + i < p.dvp;
-            cp_async16(smem_u32(dst + tt * TS + 3 * CS + i), in ? p.v + (t * p.H + h) * p.dvp + tile * DR_VT + i : p.v, in ? 16 : 0);
+            cp_async16(smem_u32(dst + tt * TS + 3 * CS + i), in ? p.v + ((t + tt) * p.H + h) * p.dvp + tile * DR_VT + i : p.v, in ? 16 : 0);
+        } else if (tid >= DR_THREADS - DR_TC && tid - (DR_THREADS - DR_TC) < n) {
+            const int tt = tid - (DR_THREADS - DR_TC);
+            asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_u32(dst + tt * TS + 3 * CS + DR_VT)),
+                         "l"(p.beta + (t + tt) * p.H + h) : "memory");
         }
         cp_async_commit();
     };
@@ -243,28 +267,14 @@ delta_scan_kernel(const DeltaScan p) {
         if (c0 + DR_TC < q_len) { issue(c0 + DR_TC, (it + 1) & 1); cp_async_wait<1>(); }
         else cp_async_wait<0>();
         __syncthreads();
-        // k . q of the chunk's tokens, a warp per token
-        for (int tt = warp; tt < n; tt += DR_THREADS / 32) {
-            float a = 0.f;
-            for (int i = lane; i < p.dp; i += 32) {
-                const float* at = buf + tt * TS + (i / NR) * dr_stride<NR>() + i % NR;
-                a = fmaf(at[0], at[CS], a);
-            }
-            a = warp_sum(a);
-            if (lane == 0) {
-                buf[tt * TS + 3 * CS + DR_VT] = p.beta[(size_t)(q_start + c0 + tt) * p.H + h];
-                buf[tt * TS + 3 * CS + DR_VT + 1] = a;
-            }
-        }
-        __syncthreads();
         const float* mine = buf + ds * dr_stride<NR>();
 #pragma unroll 1
         for (int tt = 0; tt < n; ++tt) {
             const float* tk = mine + tt * TS;
-            const float2 bk = *reinterpret_cast<const float2*>(buf + tt * TS + 3 * CS + DR_VT);
+            const float beta = buf[tt * TS + 3 * CS + DR_VT];
             const float v = buf[tt * TS + 3 * CS + vl];
             float kk[NR];
-            float sk[4] = {0.f, 0.f, 0.f, 0.f}, sq[4] = {0.f, 0.f, 0.f, 0.f};
+            float sk[4] = {0.f, 0.f, 0.f, 0.f}, sq[4] = {0.f, 0.f, 0.f, 0.f}, kq[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
             for (int i = 0; i < NR; i += 4) {
                 const float4 k4 = *reinterpret_cast<const float4*>(tk + i);
@@ -276,17 +286,21 @@ delta_scan_kernel(const DeltaScan p) {
                 sk[2] = fmaf(S[i + 2], k4.z, sk[2]); sk[3] = fmaf(S[i + 3], k4.w, sk[3]);
                 sq[0] = fmaf(S[i], q4.x, sq[0]); sq[1] = fmaf(S[i + 1], q4.y, sq[1]);
                 sq[2] = fmaf(S[i + 2], q4.z, sq[2]); sq[3] = fmaf(S[i + 3], q4.w, sq[3]);
+                kq[0] = fmaf(k4.x, q4.x, kq[0]); kq[1] = fmaf(k4.y, q4.y, kq[1]);
+                kq[2] = fmaf(k4.z, q4.z, kq[2]); kq[3] = fmaf(k4.w, q4.w, kq[3]);
             }
             float ak = (sk[0] + sk[1]) + (sk[2] + sk[3]), aq = (sq[0] + sq[1]) + (sq[2] + sq[3]);
+            float akq = (kq[0] + kq[1]) + (kq[2] + kq[3]);
 #pragma unroll
             for (int off = 1; off < DR_DS; off <<= 1) {
                 ak += __shfl_xor_sync(0xffffffffu, ak, off);
                 aq += __shfl_xor_sync(0xffffffffu, aq, off);
+                akq += __shfl_xor_sync(0xffffffffu, akq, off);
             }
-            const float un = bk.x * (v - ak);
+            const float un = beta * (v - ak);
 #pragma unroll
             for (int i = 0; i < NR; ++i) S[i] = fmaf(kk[i], un, S[i]);
-            if (ds == 0 && live) p.out[((size_t)(q_start + c0 + tt) * p.H + h) * p.dv + col] = fmaf(bk.y, un, aq);
+            if (ds == 0 && live) p.out[((size_t)(q_start + c0 + tt) * p.H + h) * p.dv + col] = fmaf(akq, un, aq);
         }
         __syncthreads();                                     // the chunk is through before its place is filled again
     }
@@ -295,6 +309,224 @@ delta_scan_kernel(const DeltaScan p) {
         for (int i = 0; i < NR; ++i) {
             const int row = ds * NR + i;
             if (row < p.d) st[(size_t)row * p.dv + col] = S[i];
+        }
+    }
+}
+
+// grid (rows x blocks, heads), a thread per key channel.  Vectors of a block: c_i k_i (4), c_i q_i (4), g_(j+1) .. g_4 k_j (4), c_4.
+// Scalars: A_10, A_20, A_21, A_30, A_31, A_32, P_00, P_10, P_11, P_20, .. P_33, then beta_0 .. beta_3.
+__global__ void __launch_bounds__(256)
+delta_blocks_kernel(const DeltaScan p) {
+    __shared__ float red[16][8];
+    const int r = blockIdx.x / p.max_blocks, b = blockIdx.x - r * p.max_blocks, h = blockIdx.y;
+    const int q_start = p.row_q_start[r], q_len = p.row_q_len[r];
+    if (p.row_slot[r] < 0 || q_len <= DR_SINGLE || b * DB_TOK >= q_len) return;
+    const int n = min(DB_TOK, q_len - b * DB_TOK);
+    const int hk = h / (p.H / p.Hk), tid = threadIdx.x;
+    const bool active = tid < p.dp;
+    float k[4], q[4], g[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        k[i] = q[i] = 0.f; g[i] = 1.f;                       // tokens the row does not have change nothing
+        if (active && i < n) {
+            const size_t t = q_start + b * DB_TOK + i;
+            k[i] = p.k[(t * p.Hk + hk) * p.dp + tid];
+            q[i] = p.q[(t * p.Hk + hk) * p.dp + tid];
+            g[i] = p.g[(t * p.H + h) * p.dp + tid];
+        }
+    }
+    const size_t slot = (size_t)block_slot(q_start, r, b) * p.H + h;
+    if (active) {
+        float* out = p.blocks + slot * DB_VECS * p.dp + tid;
+        float c = 1.f;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            c *= g[i];
+            out[i * p.dp] = c * k[i];
+            out[(4 + i) * p.dp] = c * q[i];
+        }
+        out[12 * p.dp] = c;
+        float tail = 1.f;
+#pragma unroll
+        for (int j = 3; j >= 0; --j) {
+            out[(8 + j) * p.dp] = tail * k[j];
+            tail *= g[j];
+        }
+    }
+    // products of the block's own keys and queries, the decays between the two tokens on them
+    float x[16];
+    int at_a = 0, at_p = 6;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        float w[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            w[j] = 1.f;
+#pragma unroll
+            for (int e = 0; e < 4; ++e) if (e > j && e <= i) w[j] *= g[e];
+        }
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            if (j < i) x[at_a++] = k[i] * k[j] * w[j];
+            if (j <= i) x[at_p++] = q[i] * k[j] * w[j];
+        }
+    }
+    const int lane = tid & 31, warp = tid >> 5, n_warps = blockDim.x >> 5;
+#pragma unroll
+    for (int e = 0; e < 16; ++e) {
+        const float s = warp_sum(x[e]);
+        if (lane == 0) red[e][warp] = s;
+    }
+    __syncthreads();
+    if (tid < 16) {
+        float s = 0.f;
+        for (int w = 0; w < n_warps; ++w) s += red[tid][w];
+        p.scal[slot * DB_SCAL + tid] = s;
+    } else if (tid < DB_SCAL) {
+        const int i = tid - 16;
+        p.scal[slot * DB_SCAL + tid] = i < n ? p.beta[(size_t)(q_start + b * DB_TOK + i) * p.H + h] : 0.f;
+    }
+}
+
+template <int NR>
+__global__ void __launch_bounds__(DB_THREADS)
+delta_block_scan_kernel(const DeltaScan p) {
+    constexpr int CS = DR_DS * dr_stride<NR>();
+    constexpr int VT = DB_THREADS / DR_DS * 2;               // value columns of a CTA
+    constexpr int BS = DB_VECS * CS + DB_TOK * VT + DB_SCAL; // floats of a block in shared memory
+    extern __shared__ __align__(16) float sm[];
+    const int tiles = (p.dv + VT - 1) / VT;
+    const int r = blockIdx.x / tiles, tile = blockIdx.x - r * tiles, h = blockIdx.y;
+    const int slot = p.row_slot[r];
+    const int q_start = p.row_q_start[r], q_len = p.row_q_len[r];
+    if (slot < 0 || q_len <= DR_SINGLE) return;
+    const int tid = threadIdx.x, vl = tid / DR_DS, ds = tid % DR_DS;
+    const int col = tile * VT + vl * 2;
+    const bool live0 = col < p.dv, live1 = col + 1 < p.dv;
+    float* st = p.state + ((size_t)slot * p.H + h) * p.d * p.dv;
+    float S[NR][2];
+#pragma unroll
+    for (int i = 0; i < NR; ++i) {
+        const int row = ds * NR + i;
+        S[i][0] = live0 && row < p.d ? st[(size_t)row * p.dv + col] : 0.f;
+        S[i][1] = live1 && row < p.d ? st[(size_t)row * p.dv + col + 1] : 0.f;
+    }
+    if (p.dp < DR_DS * NR) {                                 // places of channels at or beyond dp are never filled: zero once
+        for (int e = tid; e < DB_STAGES * BS; e += DB_THREADS) sm[e] = 0.f;
+        __syncthreads();
+    }
+    const int n_blocks = (q_len + DB_TOK - 1) / DB_TOK;
+    const int per = p.dp >> 2;
+    const size_t slot0 = (size_t)block_slot(q_start, r, 0);
+    auto issue = [&](int b) {
+        if (b < n_blocks) {
+            float* dst = sm + (b % DB_STAGES) * BS;
+            const size_t bs = (slot0 + b) * p.H + h;
+            const float* src = p.blocks + bs * DB_VECS * p.dp;
+            for (int piece = tid; piece < per; piece += DB_THREADS) {
+                const int i = piece * 4;
+                uint32_t at = smem_u32(dst + (i / NR) * dr_stride<NR>() + i % NR);
+                const float* s = src + i;
+#pragma unroll
+                for (int v = 0; v < DB_VECS; ++v, s += p.dp, at += CS * 4) cp_async16(at, s, 16);
+            }
+            if (tid >= DB_THREADS - 4 * VT / 4) {            // v: VT / 4 pieces of each of the four tokens
+                const int e = tid - (DB_THREADS - 4 * VT / 4), tt = e / (VT / 4), i = (e % (VT / 4)) * 4;
+                const int t = b * DB_TOK + tt;
+                const bool in = tile * VT + i < p.dvp && t < q_len;
+                cp_async16(smem_u32(dst + DB_VECS * CS + tt * VT + i),
+                           in ? p.v + ((size_t)(q_start + t) * p.H + h) * p.dvp + tile * VT + i : p.v, in ? 16 : 0);
+            } else if (tid >= 32 && tid < 32 + DB_SCAL / 4) {
+                const int e = tid - 32;
+                cp_async16(smem_u32(dst + DB_VECS * CS + DB_TOK * VT + e * 4), p.scal + bs * DB_SCAL + e * 4, 16);
+            }
+        }
+        cp_async_commit();
+    };
+#pragma unroll
+    for (int b = 0; b < DB_STAGES - 1; ++b) issue(b);
+    for (int b = 0; b < n_blocks; ++b) {
+        cp_async_wait<DB_STAGES - 2>();
+        __syncthreads();                                     // block b is there, and everyone is through with block b - 1
+        issue(b + DB_STAGES - 1);
+        const float* buf = sm + (b % DB_STAGES) * BS;
+        const float* mine = buf + ds * dr_stride<NR>();
+        float dk[4][2], dq[4][2];
+#pragma unroll
+        for (int t = 0; t < 4; ++t) dk[t][0] = dk[t][1] = dq[t][0] = dq[t][1] = 0.f;
+#pragma unroll
+        for (int i = 0; i < NR; i += 4) {
+#pragma unroll
+            for (int t = 0; t < 4; ++t) {
+                const float4 k4 = *reinterpret_cast<const float4*>(mine + t * CS + i);
+                const float4 q4 = *reinterpret_cast<const float4*>(mine + (4 + t) * CS + i);
+#pragma unroll
+                for (int c = 0; c < 2; ++c) {
+                    dk[t][c] = fmaf(S[i + 3][c], k4.w, fmaf(S[i + 2][c], k4.z, fmaf(S[i + 1][c], k4.y, fmaf(S[i][c], k4.x, dk[t][c]))));
+                    dq[t][c] = fmaf(S[i + 3][c], q4.w, fmaf(S[i + 2][c], q4.z, fmaf(S[i + 1][c], q4.y, fmaf(S[i][c], q4.x, dq[t][c]))));
+                }
+            }
+        }
+#pragma unroll
+        for (int off = 1; off < DR_DS; off <<= 1)
+#pragma unroll
+            for (int t = 0; t < 4; ++t)
+#pragma unroll
+                for (int c = 0; c < 2; ++c) {
+                    dk[t][c] += __shfl_xor_sync(0xffffffffu, dk[t][c], off);
+                    dq[t][c] += __shfl_xor_sync(0xffffffffu, dq[t][c], off);
+                }
+        const float* v_s = buf + DB_VECS * CS + vl * 2;
+        const float4* sc = reinterpret_cast<const float4*>(buf + DB_VECS * CS + DB_TOK * VT);
+        const float4 s0 = sc[0], s1 = sc[1], s2 = sc[2], s3 = sc[3], be = sc[4];
+        const float A[6] = {s0.x, s0.y, s0.z, s0.w, s1.x, s1.y};
+        const float P[10] = {s1.z, s1.w, s2.x, s2.y, s2.z, s2.w, s3.x, s3.y, s3.z, s3.w};
+        const float beta[4] = {be.x, be.y, be.z, be.w};
+        float u[4][2], o[4][2];
+#pragma unroll
+        for (int c = 0; c < 2; ++c)
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                float s = v_s[i * VT + c] - dk[i][c];
+#pragma unroll
+                for (int j = 0; j < 4; ++j) if (j < i) s = fmaf(-A[i * (i - 1) / 2 + j], u[j][c], s);
+                u[i][c] = beta[i] * s;
+                float a = dq[i][c];
+#pragma unroll
+                for (int j = 0; j < 4; ++j) if (j <= i) a = fmaf(P[i * (i + 1) / 2 + j], u[j][c], a);
+                o[i][c] = a;
+            }
+#pragma unroll
+        for (int i = 0; i < NR; i += 4) {
+            const float4 c4 = *reinterpret_cast<const float4*>(mine + 12 * CS + i);
+#pragma unroll
+            for (int c = 0; c < 2; ++c) { S[i][c] *= c4.x; S[i + 1][c] *= c4.y; S[i + 2][c] *= c4.z; S[i + 3][c] *= c4.w; }
+#pragma unroll
+            for (int t = 0; t < 4; ++t) {
+                const float4 k4 = *reinterpret_cast<const float4*>(mine + (8 + t) * CS + i);
+#pragma unroll
+                for (int c = 0; c < 2; ++c) {
+                    S[i][c] = fmaf(k4.x, u[t][c], S[i][c]); S[i + 1][c] = fmaf(k4.y, u[t][c], S[i + 1][c]);
+                    S[i + 2][c] = fmaf(k4.z, u[t][c], S[i + 2][c]); S[i + 3][c] = fmaf(k4.w, u[t][c], S[i + 3][c]);
+                }
+            }
+        }
+        if (ds < 4 && b * DB_TOK + ds < q_len) {             // lane t of the first four writes token t's two columns
+            float a = o[0][0], c = o[0][1];
+#pragma unroll
+            for (int t = 1; t < 4; ++t) if (ds == t) { a = o[t][0]; c = o[t][1]; }
+            float* out = p.out + ((size_t)(q_start + b * DB_TOK + ds) * p.H + h) * p.dv + col;
+            if (live0) out[0] = a;
+            if (live1) out[1] = c;
+        }
+    }
+    cp_async_wait<0>();
+    if (p.write_state) {
+#pragma unroll
+        for (int i = 0; i < NR; ++i) {
+            const int row = ds * NR + i;
+            if (row < p.d && live0) st[(size_t)row * p.dv + col] = S[i][0];
+            if (row < p.d && live1) st[(size_t)row * p.dv + col + 1] = S[i][1];
         }
     }
 }
@@ -323,7 +555,21 @@ static int launch_delta_scan(const DeltaScan& p, int n_rows, cudaStream_t stream
         configured = true;
     }
     const int tiles = (p.dv + DR_VT - 1) / DR_VT;
-    return launch("delta_scan", k, dim3((unsigned)tiles * n_rows, p.H), dim3(DR_THREADS), smem, stream, dim3(1, 1, 1), p);
+    const dim3 one(1, 1, 1);
+    int rc = launch("delta_scan", k, dim3((unsigned)tiles * n_rows, p.H), dim3(DR_THREADS), smem, stream, one, p);
+    if (rc || p.blocks == nullptr) return rc;
+    constexpr int VT = DB_THREADS / DR_DS * 2;
+    constexpr size_t bsmem = DB_STAGES * (size_t)(DB_VECS * DR_DS * dr_stride<NR>() + DB_TOK * VT + DB_SCAL) * sizeof(float);
+    auto kb = delta_block_scan_kernel<NR>;
+    static bool block_configured = false;
+    if (!block_configured) {
+        cudaError_t e = cudaFuncSetAttribute(kb, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bsmem);
+        if (e != cudaSuccess) return fail(-3, "delta_scan: cannot get %zu bytes of shared memory: %s", bsmem, cudaGetErrorString(e));
+        block_configured = true;
+    }
+    rc = launch("delta_blocks", delta_blocks_kernel, dim3((unsigned)n_rows * p.max_blocks, p.H), dim3((p.dp + 31) / 32 * 32), 0, stream, one, p);
+    if (rc) return rc;
+    return launch("delta_block_scan", kb, dim3((unsigned)((p.dv + VT - 1) / VT) * n_rows, p.H), dim3(DB_THREADS), bsmem, stream, one, p);
 }
 
 }  // namespace fd
@@ -362,21 +608,41 @@ extern "C" int fd_delta_prepare(const void* proj, int ld, int dtype, int q_col, 
     const size_t smem = (size_t)SC_TOK * r_max * sizeof(float);
     const dim3 grid((T + p.tpc - 1) / p.tpc, 2 * Hk + 2 * H + (g2 ? H : 0));
     FD_REQUIRE(grid.y <= 65535, -2, "delta_prepare: %d heads", H);
-    if (dtype == 0) return launch("delta_prepare", delta_prepare_kernel<float>, grid, dim3(threads), smem, stream, dim3(1, 1, 1), p);
-    return launch("delta_prepare", delta_prepare_kernel<bf16>, grid, dim3(threads), smem, stream, dim3(1, 1, 1), p);
+    const bool narrow = a2 != nullptr || g2 != nullptr;
+    if (dtype == 0) {
+        if (narrow) return launch("delta_prepare", delta_prepare_kernel<float, true>, grid, dim3(threads), smem, stream, dim3(1, 1, 1), p);
+        return launch("delta_prepare", delta_prepare_kernel<float, false>, grid, dim3(threads), smem, stream, dim3(1, 1, 1), p);
+    }
+    if (narrow) return launch("delta_prepare", delta_prepare_kernel<bf16, true>, grid, dim3(threads), smem, stream, dim3(1, 1, 1), p);
+    return launch("delta_prepare", delta_prepare_kernel<bf16, false>, grid, dim3(threads), smem, stream, dim3(1, 1, 1), p);
 }
 
 // q, k [T, Hk, dp], g [T, H, dp], v [T, H, dvp], beta [T, H] as fd_delta_prepare leaves them; state [slots, H, d, dv] and
-// out [T, H dv] float.
+// out [T, H dv] float.  max_q_len: the longest row of the step; rows of more than 16 tokens take the block form and need scratch
+// memory, fd_delta_scan_scratch_floats floats (without it every row is walked token by token).
+extern "C" int fd_delta_scan_single() { return DR_SINGLE; }
+extern "C" long long fd_delta_scan_scratch_floats(int T, int n_rows, int H, int d) {
+    return (long long)(T / DB_TOK + n_rows + 1) * H * (DB_VECS * ((d + 3) / 4 * 4) + DB_SCAL);
+}
 extern "C" int fd_delta_scan(const float* q, const float* k, const float* v, const float* g, const float* beta, float* state,
                              float* out, const int* row_slot, const int* row_q_start, const int* row_q_len, int n_rows, int H,
-                             int Hk, int d, int dv, int write_state, cudaStream_t stream) {
+                             int Hk, int d, int dv, int write_state, int T, int max_q_len, float* scratch, long long scratch_floats,
+                             cudaStream_t stream) {
     if (n_rows == 0) return 0;
     FD_REQUIRE(H > 0 && Hk > 0 && H % Hk == 0 && d > 0 && d <= 256 && dv > 0, -2, "delta_scan: %d heads on %d of %d x %d (keys up to 256)", H, Hk, d, dv);
     FD_REQUIRE(H <= 65535 && (long long)n_rows * ((dv + DR_VT - 1) / DR_VT) < (1ll << 31), -2, "delta_scan: %d rows", n_rows);
     auto al = [](const void* x) { return (uintptr_t)x % 16 == 0; };
     FD_REQUIRE(al(q) && al(k) && al(v) && al(g), -2, "delta_scan: 16-byte alignment");
-    DeltaScan p = {q, k, v, g, beta, state, out, row_slot, row_q_start, row_q_len, H, Hk, d, dv, (d + 3) / 4 * 4, (dv + 3) / 4 * 4, write_state};
+    DeltaScan p = {q, k, v, g, beta, state, out, row_slot, row_q_start, row_q_len, H, Hk, d, dv, (d + 3) / 4 * 4, (dv + 3) / 4 * 4, write_state,
+                   nullptr, nullptr, 0};
+    if (scratch != nullptr && max_q_len > DR_SINGLE) {
+        FD_REQUIRE(scratch_floats >= fd_delta_scan_scratch_floats(T, n_rows, H, d) && (uintptr_t)scratch % 16 == 0, -2,
+                   "delta_scan: %lld floats of scratch memory for %d tokens", scratch_floats, T);
+        p.blocks = scratch;
+        p.scal = scratch + (long long)(T / DB_TOK + n_rows + 1) * H * DB_VECS * p.dp;
+        p.max_blocks = (max_q_len + DB_TOK - 1) / DB_TOK;
+        FD_REQUIRE((long long)n_rows * p.max_blocks < (1ll << 31), -2, "delta_scan: %d rows of %d tokens", n_rows, max_q_len);
+    }
     if (d <= 32) return launch_delta_scan<4>(p, n_rows, stream);
     if (d <= 64) return launch_delta_scan<8>(p, n_rows, stream);
     if (d <= 128) return launch_delta_scan<16>(p, n_rows, stream);

@@ -17,6 +17,7 @@ constexpr int SC_TAPS = 4;            // more taps than this take the plain loop
 
 struct ConvMeta {                     // what the tokens of a tile need to know, in shared memory
     int slot[SC_TOK], i[SC_TOK], pos[SC_TOK], single[SC_TOK];     // slot -1: padding row; i: place in its row's new tokens
+    int one_row;                      // the tile's tokens all belong to one row (and none is padding)
 };
 
 // threads 0 .. nt - 1 fill the tile's entries; the caller synchronises
@@ -28,6 +29,7 @@ __device__ __forceinline__ void conv_meta(ConvMeta& m, int t0, int nt, const int
         m.i[threadIdx.x] = t - row_q_start[r];
         m.pos[threadIdx.x] = tok_pos[t];
         m.single[threadIdx.x] = row_q_len[r] == 1;
+        if (threadIdx.x == 0) m.one_row = m.slot[0] >= 0 && tok_row[t0 + nt - 1] == r;
     }
 }
 
@@ -40,6 +42,36 @@ __device__ __forceinline__ void conv_channel(const T* __restrict__ col, int ld, 
     float wk[SC_TAPS];
 #pragma unroll
     for (int k = 0; k < SC_TAPS; ++k) wk[k] = k < taps ? w[k] : 0.f;
+    if (m.one_row && !m.single[0] && taps <= SC_TAPS) {
+        // consecutive tokens of one row: every value once, all loads under way together; place SC_TAPS - 1 + j is token t0 + j
+        float u[SC_TOK + SC_TAPS - 1];
+        const int i0 = m.i[0], pos0 = m.pos[0];
+        const float* rg = ring + (size_t)m.slot[0] * taps * C + c;
+#pragma unroll
+        for (int e = 0; e < SC_TOK + SC_TAPS - 1; ++e) {
+            const int j = e - (SC_TAPS - 1);
+            u[e] = 0.f;
+            if (j >= nt || -j >= taps) continue;
+            if (i0 + j >= 0) u[e] = to_float(col[(size_t)(t0 + j) * ld]);
+            else if (pos0 + j >= 0) u[e] = rg[(size_t)((pos0 + j) % taps) * C];
+        }
+        // the weights moved to the end, so that tap k of `taps` meets the place it would meet below
+        float we[SC_TAPS];
+#pragma unroll
+        for (int e = 0; e < SC_TAPS; ++e) {
+            we[e] = 0.f;
+#pragma unroll
+            for (int k = 0; k < SC_TAPS; ++k) if (k < taps && SC_TAPS - taps + k == e) we[e] = wk[k];
+        }
+#pragma unroll
+        for (int tt = 0; tt < SC_TOK; ++tt) {
+            float a = bias;
+#pragma unroll
+            for (int e = 0; e < SC_TAPS; ++e) if (e >= SC_TAPS - taps) a = fmaf(we[e], u[tt + e], a);
+            y[tt] = tt < nt ? a : 0.f;
+        }
+        return;
+    }
 #pragma unroll
     for (int tt = 0; tt < SC_TOK; ++tt) {
         y[tt] = 0.f;

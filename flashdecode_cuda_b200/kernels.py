@@ -108,11 +108,15 @@ def _declare(L: ctypes.CDLL) -> None:
         "fd_row_norm_gate": [P, P, P, I, P, I, I, I, F, P],
         "fd_head_norm_gate": [P, P, P, I, P, P, I, I, I, I, I, F, F, P],
         "fd_delta_prepare": [P, I, I, I, I, I, I, I, I, P, P, I, I, P, I, P, P, I, P, P, F, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, P],
-        "fd_delta_scan": [P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, P],
+        "fd_delta_scan": [P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, P, LL, P],
+        "fd_delta_scan_single": [],
         "fd_conv_ring_update": [P, I, I, P, P, P, P, P, I, I, I, P],
-        "fd_ssd_prepare": [P, I, I, I, I, I, P, P, P, I, I, P, P, P, P, P, P, P, P, P, I, I, P],
+        "fd_ssd_prepare": [P, I, I, I, I, I, P, P, P, I, I, P, P, P, P, I, P, P, P, P, P, P, I, I, P],
+        "fd_ssd_chunks_takes": [I, I],
+        "fd_ssd_chunk": [],
+        "fd_ssd_chunks": [P, I, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, P, LL, P],
         "fd_ssd_gate_norm": [P, P, I, P, P, I, P, P, I, I, I, I, I, I, F, F, P],
-        "fd_rope_norm_append": [P, I, I, P, P, P, P, P, P, F, P, P, I, I, I, I, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, I, P, P],
+        "fd_rope_norm_append": [P, I, I, P, P, P, P, P, P, F, P, P, I, I, I, I, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, I, I, P, P],
         "fd_low_rank_expand": [P, I, P, P, P, I, I, I, I, P],
         "fd_conv_state_update": [P, I, I, P, P, P, P, I, I, I, P],
         "fd_gate_mul": [P, P, I, P, I, I, I, P],
@@ -156,6 +160,10 @@ def _declare(L: ctypes.CDLL) -> None:
     L.fd_linear_scan_segment.restype = I
     L.fd_linear_scan_scratch_floats.argtypes = [I, I, I, I, I]
     L.fd_linear_scan_scratch_floats.restype = LL
+    L.fd_delta_scan_scratch_floats.argtypes = [I, I, I, I]
+    L.fd_delta_scan_scratch_floats.restype = LL
+    L.fd_ssd_chunks_scratch_floats.argtypes = [I, I, I, I, I]
+    L.fd_ssd_chunks_scratch_floats.restype = LL
     L.fd_sample_scratch_words.argtypes = [I, I]
     L.fd_sample_scratch_words.restype = LL
 
@@ -1076,17 +1084,27 @@ def delta_prepare(proj: torch.Tensor, cols, conv_w: torch.Tensor, ring: Optional
 
 def delta_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, g: torch.Tensor, beta: torch.Tensor, state: torch.Tensor,
                out: torch.Tensor, row_slot: torch.Tensor, row_q_start: torch.Tensor, row_q_len: torch.Tensor, n_rows: int,
-               write_state: bool) -> None:
+               write_state: bool, max_q_len: int = 0, scratch: Optional[torch.Tensor] = None) -> None:
     """S <- diag(g) S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q, per sequence and head over the step's tokens, from
     ``state`` [slots, heads, d, dv] (float32, updated when ``write_state``) to ``out`` [T, heads * dv] float32.  The inputs are
-    those ``delta_prepare`` leaves."""
+    those ``delta_prepare`` leaves.  With ``scratch`` (float32, ``delta_scan_scratch_floats`` elements) and ``max_q_len`` (the longest
+    row), rows of more than ``delta_scan_single()`` tokens are walked four tokens at a time."""
     H, d, dv = state.shape[1:]
     T, Hk = q.shape[:2]
     for t in (q, k, v, g, beta, state, out):
         assert t.dtype == torch.float32
     assert out.shape == (T, H * dv) and k.shape == q.shape and g.shape[:2] == (T, H) and v.shape[:2] == (T, H)
     _check(lib().fd_delta_scan(_ptr(q), _ptr(k), _ptr(v), _ptr(g), _ptr(beta), _ptr(state), _ptr(out), _ptr(row_slot),
-                               _ptr(row_q_start), _ptr(row_q_len), n_rows, H, Hk, d, dv, int(write_state), _stream()))
+                               _ptr(row_q_start), _ptr(row_q_len), n_rows, H, Hk, d, dv, int(write_state), T, int(max_q_len), _ptr(scratch),
+                               scratch.numel() if scratch is not None else 0, _stream()))
+
+
+def delta_scan_single() -> int:
+    return lib().fd_delta_scan_single()
+
+
+def delta_scan_scratch_floats(T: int, n_rows: int, n_heads: int, head_dim: int) -> int:
+    return int(lib().fd_delta_scan_scratch_floats(T, n_rows, n_heads, head_dim))
 
 
 def conv_ring_update(proj: torch.Tensor, first_col: int, ring: torch.Tensor, row_slot: torch.Tensor, row_q_start: torch.Tensor,
@@ -1101,18 +1119,53 @@ def conv_ring_update(proj: torch.Tensor, first_col: int, ring: torch.Tensor, row
 
 def ssd_prepare(proj: torch.Tensor, col: int, dt_col: int, conv_w: torch.Tensor, conv_b: torch.Tensor, ring: Optional[torch.Tensor],
                 keep: bool, dt_bias: torch.Tensor, A_log: torch.Tensor, xbc: torch.Tensor, step: torch.Tensor, tok_row: torch.Tensor,
-                tok_pos: torch.Tensor, row_slot: torch.Tensor, row_q_start: torch.Tensor, row_q_len: torch.Tensor) -> None:
+                tok_pos: torch.Tensor, row_slot: torch.Tensor, row_q_start: torch.Tensor, row_q_len: torch.Tensor,
+                xbc16: Optional[torch.Tensor] = None, float_cols: Optional[int] = None) -> None:
     """``xbc`` float32 [T, C] <- silu of the causal convolution (``conv_w`` [C, taps], bias ``conv_b`` [C], float32; earlier
     values from ``ring`` [slots, taps, C]) of the C columns of ``proj`` from ``col`` on; ``step`` float32 [T, heads, 2] <- (dt,
-    exp(-exp(A_log) dt)) with dt = softplus of the columns from ``dt_col`` on plus ``dt_bias``."""
+    exp(-exp(A_log) dt)) with dt = softplus of the columns from ``dt_col`` on plus ``dt_bias``.  ``xbc16`` bfloat16 [T, C]: receives
+    all columns rounded, and ``xbc`` only its first ``float_cols``."""
     T, C, H, taps = proj.shape[0], xbc.shape[1], dt_bias.numel(), conv_w.shape[1]
     for t in (conv_w, conv_b, ring, dt_bias, A_log, xbc, step):
         assert t is None or t.dtype == torch.float32
     assert conv_w.shape == (C, taps) and conv_b.numel() == C and (taps == 1 or ring.shape[1:] == (taps, C))
     assert xbc.shape[0] == T and step.shape == (T, H, 2) and A_log.numel() == H
+    assert xbc16 is None or (xbc16.dtype == torch.bfloat16 and xbc16.shape == xbc.shape)
     _check(lib().fd_ssd_prepare(_ptr(proj), proj.shape[1], _dt(proj.dtype), col, C, dt_col, _ptr(conv_w), _ptr(conv_b), _ptr(ring),
-                                taps, int(keep), _ptr(dt_bias), _ptr(A_log), _ptr(xbc), _ptr(step), _ptr(tok_row), _ptr(tok_pos),
+                                taps, int(keep), _ptr(dt_bias), _ptr(A_log), _ptr(xbc), _ptr(xbc16),
+                                C if float_cols is None else int(float_cols), _ptr(step), _ptr(tok_row), _ptr(tok_pos),
                                 _ptr(row_slot), _ptr(row_q_start), _ptr(row_q_len), T, H, _stream()))
+
+
+def ssd_chunks_takes(state_size: int, v_head_dim: int) -> bool:
+    """Whether ``ssd_chunks`` takes a state of these sizes."""
+    return bool(lib().fd_ssd_chunks_takes(state_size, v_head_dim))
+
+
+def ssd_chunk() -> int:
+    """Tokens of a chunk of ``ssd_chunks``."""
+    return lib().fd_ssd_chunk()
+
+
+def ssd_chunks_scratch_floats(T: int, n_rows: int, n_heads: int, state_size: int, v_head_dim: int) -> int:
+    return int(lib().fd_ssd_chunks_scratch_floats(T, n_rows, n_heads, state_size, v_head_dim))
+
+
+def ssd_chunks(xbc16: torch.Tensor, step: torch.Tensor, A_log: torch.Tensor, state: torch.Tensor, y: torch.Tensor, n_groups: int,
+               row_slot: torch.Tensor, row_q_start: torch.Tensor, row_q_len: torch.Tensor, n_rows: int, max_q_len: int,
+               write_state: bool, scratch: torch.Tensor) -> None:
+    """The recurrence S_t = exp(-exp(A_log) dt) S_(t-1) + dt B_t x_t^T, y_t = S_t^T C_t in chunks on the tensor cores.  ``xbc16``
+    bfloat16 [T, ld]: x, B, C side by side; ``step`` float32 [T, heads, 2]: dt first; ``state`` float32 [slots, heads, N, dv],
+    updated when ``write_state``; ``y`` float32 [T, heads * dv]; ``scratch`` float32."""
+    H, N, dv = state.shape[1:]
+    T = xbc16.shape[0]
+    assert xbc16.dtype == torch.bfloat16 and xbc16.shape[1] == H * dv + 2 * n_groups * N and step.shape == (T, H, 2)
+    for t in (step, A_log, state, y, scratch):
+        assert t.dtype == torch.float32
+    assert y.shape == (T, H * dv) and A_log.numel() == H
+    _check(lib().fd_ssd_chunks(_ptr(xbc16), xbc16.shape[1], _ptr(step), _ptr(A_log), _ptr(state), _ptr(y), _ptr(row_slot),
+                               _ptr(row_q_start), _ptr(row_q_len), n_rows, T, int(max_q_len), H, n_groups, N, dv, int(write_state),
+                               _ptr(scratch), scratch.numel(), _stream()))
 
 
 def ssd_gate_norm(y: torch.Tensor, xbc: torch.Tensor, D: torch.Tensor, proj: torch.Tensor, z_col: int, weight: torch.Tensor,
@@ -1135,12 +1188,13 @@ def rope_norm_append(proj: torch.Tensor, first_col: int, q_out: torch.Tensor, k_
                      cos: Optional[torch.Tensor], sin: Optional[torch.Tensor], rot_dims: int, head_norm: bool,
                      tok_row: torch.Tensor, tok_pos: torch.Tensor, row_slot: torch.Tensor, n_q: int, n_kv: int, head_dim: int,
                      v_head_dim: int, write_kv: bool, status: torch.Tensor, q_count: int = 0, k_count: int = 0, head_count: int = 0,
-                     value_mode: int = VALUES_PLAIN, v_first: Optional[torch.Tensor] = None, lam: Optional[torch.Tensor] = None) -> None:
+                     value_mode: int = VALUES_PLAIN, v_first: Optional[torch.Tensor] = None, lam: Optional[torch.Tensor] = None, v_count: int = 0) -> None:
     """From the columns of ``proj`` from ``first_col`` on - q, k, v side by side - to ``q_out`` [T, n_q head_dim] and the paged
     cache: q and k RMS-normed over their whole projections (``q_weight``, ``k_weight`` float32, or None: not), their first
     ``rot_dims`` dimensions turned (i paired with i + rot_dims / 2), and by ``head_norm`` every head divided by its own root mean
     square.  The means run over ``q_count`` / ``k_count`` / ``head_count`` values (0: all).  ``value_mode``: VALUES_SOURCE also leaves
-    the values in ``v_first`` [T, n_kv v_head_dim]; VALUES_MIXED stores (1 - lam) v + lam v_first, ``lam`` one float32."""
+    the values in ``v_first`` [T, n_kv v_count]; VALUES_MIXED stores (1 - lam) v + lam v_first, ``lam`` one float32; ``v_count`` (0:
+    all): the dimensions of a value head that are not padding."""
     T = proj.shape[0]
     num_blocks, _, block_size, _ = k_pool.shape
     assert proj.dtype == q_out.dtype == k_pool.dtype == v_pool.dtype and q_out.shape == (T, n_q * head_dim)
@@ -1148,14 +1202,15 @@ def rope_norm_append(proj: torch.Tensor, first_col: int, q_out: torch.Tensor, k_
     assert first_col + (n_q + n_kv) * head_dim + n_kv * v_head_dim <= proj.shape[1]
     assert q_weight is None or (q_weight.dtype == k_weight.dtype == torch.float32 and q_weight.numel() == n_q * head_dim
                                 and k_weight.numel() == n_kv * head_dim)
-    assert value_mode == VALUES_PLAIN or (v_first.dtype == proj.dtype and v_first.shape == (T, n_kv * v_head_dim))
+    assert value_mode == VALUES_PLAIN or (v_first.dtype == proj.dtype and v_first.shape == (T, n_kv * (v_count or v_head_dim)))
     assert value_mode != VALUES_MIXED or (lam.dtype == torch.float32 and lam.numel() == 1)
     _check(lib().fd_rope_norm_append(
         _col_ptr(proj, first_col), proj.shape[1], _dt(proj.dtype), _ptr(q_out), _ptr(k_pool), _ptr(v_pool), _ptr(v_first),
         _ptr(q_weight), _ptr(k_weight), float(eps), _ptr(cos) if rot_dims else None, _ptr(sin) if rot_dims else None,
         cos.shape[0] if rot_dims else 0, rot_dims, int(head_norm), value_mode, _ptr(lam), _ptr(tok_row), _ptr(tok_pos),
         _ptr(row_slot), _ptr(block_table), block_table.shape[1], num_blocks, block_size, T, n_q, n_kv, head_dim, v_head_dim,
-        q_count or n_q * head_dim, k_count or n_kv * head_dim, head_count or head_dim, int(write_kv), _ptr(status), _stream()))
+        q_count or n_q * head_dim, k_count or n_kv * head_dim, head_count or head_dim, v_count or v_head_dim,
+        int(write_kv), _ptr(status), _stream()))
 
 
 # ---------------------------------------------------------------------------

@@ -22,7 +22,8 @@ LAUNCHERS = ["embed", "add_rmsnorm", "silu_mul", "rope_append", "gemv_qkv_rope",
              "conv_state_update", "gate_mul", "add_concat", "relu2", "moe_route", "moe_align", "moe_gemm", "moe_combine",
              "moe_gather", "gemm_tc_grouped", "glu_mul", "softcap", "lanes_norm", "lanes_fill", "norm_append", "head_gemm",
              "attention_ext", "attn_head_mix", "add_dyn_tanh", "quad_exp_act", "scale_", "axpy_f32", "linear_scan",
-             "head_norm_gate", "row_norm_gate", "rope_heads", "post_norm", "stream_conv", "attention_dense", "add_cast", "side_gate_mul", "token_side_row", "add_row_vector", "low_rank_expand"]
+             "head_norm_gate", "row_norm_gate", "rope_heads", "post_norm", "stream_conv", "attention_dense", "add_cast", "side_gate_mul", "token_side_row", "add_row_vector", "low_rank_expand",
+             "rope_norm_append", "delta_prepare", "delta_scan", "conv_ring_update", "ssd_prepare", "ssd_chunks", "ssd_gate_norm", "relu2_cols"]
 
 
 class PartTimer:
@@ -174,8 +175,14 @@ def part_work(part, ctx_lens: Sequence[int], q_lens: Sequence[int], real_choice_
         for b in part.branches:
             if type(b).__name__ == "ConvGatedAttention":
                 f, y = _conv_attention_inner(b, ctx_lens, q_lens, el)
-            elif type(b).__name__ in ("Retention", "GatedLinearRecurrence"):
+            elif type(b).__name__ in ("Retention", "GatedLinearRecurrence", "Mamba2", "GatedDeltaRule"):
                 f, y = _recurrence_inner(b, q_lens)
+            elif type(b).__name__ == "QKNormedAttention":
+                pairs = visible_pairs(ctx_lens, q_lens, b.window, None)
+                f = 2.0 * b.n_q * (b.d + b.dv) * pairs
+                y = keys_read(ctx_lens, q_lens, b.window, None) * b.n_kv * (b.d + b.dv) * el
+            elif type(b).__name__ == "DenseActMLP":
+                f, y = 0.0, 0.0                      # nothing beside its two products, which are counted below
             else:
                 f, y = part_work(b, ctx_lens, q_lens)
                 y -= act
@@ -233,8 +240,12 @@ def _conv_attention_inner(part, ctx_lens, q_lens, el: int) -> Tuple[float, float
 
 def _recurrence_inner(part, q_lens) -> Tuple[float, float]:
     """(operations, bytes) of a matrix-state recurrence between its two products: per token and state element one
-    multiply-add to move the state on and one to read it; every row's float32 state read and written once."""
+    multiply-add to move the state on and one to read it (the delta rule: one more to read what is there before the
+    write, and the product of its narrow vectors); every row's float32 state read and written once."""
     elements = part.n_heads * part.d * part.dv
+    if type(part).__name__ == "GatedDeltaRule":
+        narrow = 2 * sum(q_lens) * part.n_heads * (part.d * part.ra + part.dv * part.rg)
+        return float(6 * sum(q_lens) * elements + narrow), float(2 * len(q_lens) * elements * 4)
     return float(4 * sum(q_lens) * elements), float(2 * len(q_lens) * elements * 4)
 
 

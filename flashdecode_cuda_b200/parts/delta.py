@@ -127,7 +127,11 @@ class GatedDeltaRule(Mixer):
         if ring is not None and lc.writes and ctx.max_q_len > 1:
             K.conv_ring_update(proj, col0, ring, ctx.row_slot, ctx.row_q_start, ctx.row_q_len, ctx.row_ctx_len, ctx.n_rows)
         o = ws.get("scan_out", (T, H * dv), f32)
-        K.delta_scan(q, k, v, g, beta, lc.states["state"], o, ctx.row_slot, ctx.row_q_start, ctx.row_q_len, ctx.n_rows, lc.writes)
+        scratch = None
+        if ctx.max_q_len > K.delta_scan_single():
+            scratch = ws.get("delta_blocks", (K.delta_scan_scratch_floats(T, ctx.n_rows, H, d),), f32)
+        K.delta_scan(q, k, v, g, beta, lc.states["state"], o, ctx.row_slot, ctx.row_q_start, ctx.row_q_len, ctx.n_rows, lc.writes,
+                     ctx.max_q_len, scratch)
         K.head_norm_gate(o, act, act_col, H, dv, self.eps, self.norm_w, None, 0, scale, sigmoid_gate=gate_z)
         return act
 

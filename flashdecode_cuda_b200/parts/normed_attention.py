@@ -207,13 +207,14 @@ class QKNormedAttention(Mixer):
         if self.turned or col0:
             v_first = None
             if self.value_mix:
-                v_first = ws.get(f"first_{self.value_group}", (T, self.n_kv * self.dvp), proj.dtype)
+                v_first = ws.get(f"first_{self.value_group}", (T, self.n_kv * self.dv), proj.dtype)
             mode = {None: K.VALUES_PLAIN, "source": K.VALUES_SOURCE, "mix": K.VALUES_MIXED}[self.value_mix]
             rope = self.position
             K.rope_norm_append(proj, col0, q, lc.k_pool, lc.v_pool, lc.group.table, self.q_norm, self.k_norm, self.eps,
                                rope.cos if self.rot_dims else None, rope.sin if self.rot_dims else None, self.rot_dims,
                                self.head_norm, ctx.tok_row, ctx.tok_pos, ctx.row_slot, self.n_q, self.n_kv, self.dp, self.dvp,
-                               lc.writes, rt.status, head_count=self.d, value_mode=mode, v_first=v_first, lam=self.lam, **counts)
+                               lc.writes, rt.status, head_count=self.d, value_mode=mode, v_first=v_first, lam=self.lam,
+                               v_count=self.dv, **counts)
         else:
             K.norm_append(proj, q, self.q_norm, self.k_norm, self.eps, ctx.tok_row, ctx.tok_pos, ctx.row_slot, lc.k_pool,
                           lc.v_pool, lc.group.table, self.n_kv, lc.writes, rt.status, **counts)

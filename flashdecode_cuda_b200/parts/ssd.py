@@ -14,6 +14,9 @@ from .base import LayerCache, Runtime
 from .recurrent import _StateMixer
 
 
+CHUNKED_FROM = 32         # bfloat16 steps with a portion of more tokens than this take the recurrence in chunks
+
+
 @register_part("mixer", "mamba2")
 class Mamba2(_StateMixer):
     """For the mixer's input h [T, hidden], with ``n_heads`` heads of ``v_head_dim`` channels (together ``inner``), a state of
@@ -76,13 +79,22 @@ class Mamba2(_StateMixer):
         y = ws.get("scan_out", (T, self.inner_size), torch.float32)
         ring = lc.states.get("ring")
         x_col = col0 + self.inner_size
+        # long portions in bfloat16: chunks on the tensor cores, from the convolved channels rounded; x itself also as floats
+        chunked = proj.dtype == torch.bfloat16 and ctx.max_q_len > CHUNKED_FROM and K.ssd_chunks_takes(self.d, self.dv)
+        xbc16 = ws.get("ssd_xbc16", (T, self.n_conv), torch.bfloat16) if chunked else None
         K.ssd_prepare(proj, x_col, x_col + self.n_conv, self.conv_w, self.conv_b, ring, lc.writes, self.dt_bias, self.A_log, xbc, step,
-                      ctx.tok_row, ctx.tok_pos, ctx.row_slot, ctx.row_q_start, ctx.row_q_len)
+                      ctx.tok_row, ctx.tok_pos, ctx.row_slot, ctx.row_q_start, ctx.row_q_len, xbc16=xbc16,
+                      float_cols=self.inner_size if chunked else None)
         if ring is not None and lc.writes and ctx.max_q_len > 1:
             K.conv_ring_update(proj, x_col, ring, ctx.row_slot, ctx.row_q_start, ctx.row_q_len, ctx.row_ctx_len, ctx.n_rows)
         b_col = self.inner_size
-        K.linear_scan(xbc, b_col + self.groups * self.d, b_col, 0, lc.states["state"], y, K.SCAN_STEP, ctx.row_slot,
-                      ctx.row_q_start, ctx.row_q_len, ctx.row_ctx_len, ctx.n_rows, self.n_heads, self.d, self.dv, lc.writes,
-                      rt.status, max_q_len=ctx.max_q_len, scratch=self.scan_scratch(ctx), step=step, qk_heads=self.groups)
+        if chunked:
+            n = K.ssd_chunks_scratch_floats(T, ctx.n_rows, self.n_heads, self.d, self.dv)
+            K.ssd_chunks(xbc16, step, self.A_log, lc.states["state"], y, self.groups, ctx.row_slot, ctx.row_q_start, ctx.row_q_len,
+                         ctx.n_rows, ctx.max_q_len, lc.writes, ws.get("ssd_chunks", (n,), torch.float32))
+        else:
+            K.linear_scan(xbc, b_col + self.groups * self.d, b_col, 0, lc.states["state"], y, K.SCAN_STEP, ctx.row_slot,
+                          ctx.row_q_start, ctx.row_q_len, ctx.row_ctx_len, ctx.n_rows, self.n_heads, self.d, self.dv, lc.writes,
+                          rt.status, max_q_len=ctx.max_q_len, scratch=self.scan_scratch(ctx), step=step, qk_heads=self.groups)
         K.ssd_gate_norm(y, xbc, self.D, proj, col0, self.norm_w, act, act_col, self.norm_groups, self.eps, scale)
         return act
