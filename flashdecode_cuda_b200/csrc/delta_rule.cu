@@ -4,8 +4,8 @@
 //
 //  * delta_prepare: everything that enters the recurrence, as floats.  q, k and v pass a short causal convolution over time
 //    per channel (short_conv.cuh) and silu; every head of q and k becomes a unit vector, x / sqrt(sum x^2 + 1e-6), and q is
-//    multiplied by a constant; g = exp(-exp(A_h) softplus(z + bias)) per key channel with z a narrow vector times a matrix
-//    (or handed over); beta = sigmoid of a column per head; by option the output gate's pre-activation from its own
+//    multiplied by a constant; the log decay log g = -exp(A_h) softplus(z + bias) per key channel with z a narrow vector times
+//    a matrix (or handed over); beta = sigmoid of a column per head; by option the output gate's pre-activation from its own
 //    narrow vector.
 //  * delta_scan: the recurrence.  A CTA of 128 threads takes one sequence of the step, one head and 16 value columns; 8
 //    adjacent lanes share a column and each holds NR adjacent rows of it in registers.  Tokens come to shared memory a chunk
@@ -18,7 +18,7 @@
 //        S <- c_4 S + sum_j (g_(j+1) .. g_4 k_j) u_j^T,     A_ij = sum_c k_i k_j g_(j+1) .. g_i,  P_ij the same with q_i,
 //    in which decays are only multiplied, never divided.  The first kernel leaves the 13 vectors and 16 products of
 //    every block (nothing in it depends on the state); the second walks the blocks, one reduction over the lanes per block
-//    instead of one per token, two value columns per thread, blocks three ahead on their way with cp.async.
+//    instead of one per token, blocks three ahead on their way with cp.async.
 //  * conv_ring_update: after a step with longer portions, the last values of every row go to its ring.
 //
 // State, decays, step sizes, unit vectors, sums: float.  A sequence's tokens are walked in order, so the sums of every
@@ -36,7 +36,7 @@ constexpr int DR_DS = 8;                       // lanes that share a column
 constexpr int DR_VT = DR_THREADS / DR_DS;      // value columns of a CTA
 constexpr int DR_TC = 16;                      // tokens of a chunk
 constexpr int DR_SINGLE = 16;                  // the most tokens of a row that is walked token by token
-constexpr int DB_THREADS = 64;                 // block form: 8 lanes share two columns
+constexpr int DB_VT = 8;                       // block form: value columns of a CTA
 constexpr int DB_TOK = 4, DB_VECS = 13, DB_SCAL = 20, DB_STAGES = 4;
 
 struct DeltaParams {
@@ -114,7 +114,7 @@ delta_prepare_kernel(const DeltaParams p) {
 #pragma unroll
         for (int tt = 0; tt < SC_TOK; ++tt) {
             if (tt >= nt) continue;
-            y[tt] = active ? sc_silu(y[tt]) : 0.f;
+            y[tt] = active ? sc_silu<T>(y[tt]) : 0.f;
             const float s = warp_sum(y[tt] * y[tt]);
             if ((tid & 31) == 0) red[tt][tid >> 5] = s;
         }
@@ -122,14 +122,14 @@ delta_prepare_kernel(const DeltaParams p) {
         if (tid >= p.dp) return;
         float* out = is_q ? p.q : p.k;
         const int nw = blockDim.x >> 5;
-        for (int tt = 0; tt < nt; ++tt) {
-            if (meta.slot[tt] < 0) continue;
+        const float scale = is_q ? p.q_scale : 1.f;
+        out += ((size_t)t0 * p.Hk + h) * p.dp + tid;
+#pragma unroll
+        for (int tt = 0; tt < SC_TOK; ++tt) {
+            if (tt >= nt || meta.slot[tt] < 0) continue;
             float total = 0.f;
             for (int w = 0; w < nw; ++w) total += red[tt][w];
-            float val = 0.f;
-#pragma unroll
-            for (int e = 0; e < SC_TOK; ++e) if (e == tt) val = y[e];
-            out[((size_t)(t0 + tt) * p.Hk + h) * p.dp + tid] = val / sqrtf(total + DELTA_UNIT_EPS) * (is_q ? p.q_scale : 1.f);
+            out[(size_t)tt * p.Hk * p.dp] = y[tt] * (scale * rsqrtf(total + DELTA_UNIT_EPS));
         }
         return;
     }
@@ -145,7 +145,7 @@ delta_prepare_kernel(const DeltaParams p) {
 #pragma unroll
             for (int tt = 0; tt < SC_TOK; ++tt)
                 if (tt < nt && meta.slot[tt] >= 0)
-                    p.v[((size_t)(t0 + tt) * p.H + u) * p.dvp + j] = active ? sc_silu(y[tt]) : 0.f;
+                    p.v[((size_t)(t0 + tt) * p.H + u) * p.dvp + j] = active ? sc_silu<T>(y[tt]) : 0.f;
         }
         return;
     }
@@ -185,17 +185,18 @@ delta_prepare_kernel(const DeltaParams p) {
         const float b = active ? p.dt_bias[h * p.d + j] : 0.f;
 #pragma unroll
         for (int tt = 0; tt < SC_TOK; ++tt)
-            if (tt < nt) p.g[((size_t)(t0 + tt) * p.H + h) * p.dp + j] = active ? expf(-rate * sc_softplus(z[tt] + b)) : 0.f;
+            if (tt < nt) p.g[((size_t)(t0 + tt) * p.H + h) * p.dp + j] = active ? -rate * sc_softplus(z[tt] + b) : 0.f;
     }
 }
 
 struct DeltaScan {
-    const float* q; const float* k; const float* v; const float* g; const float* beta;
+    const float* q; const float* k; const float* v; const float* g; const float* beta;      // g: log decays
     float* state; float* out;                  // [slots, H, d, dv], [T, H dv]
     const int* row_slot; const int* row_q_start; const int* row_q_len;
     int H, Hk, d, dv, dp, dvp, write_state;
     float* blocks; float* scal;                // block form: [block slots, H, DB_VECS, dp], [block slots, H, DB_SCAL]; or null
     int max_blocks;                            // blocks of the longest row
+    int short_only;                            // rows of more than DR_SINGLE tokens are not walked token by token
 };
 
 // Block b of step row r has the slot q_start / 4 + r + b: slots of different rows never meet.
@@ -215,7 +216,7 @@ delta_scan_kernel(const DeltaScan p) {
     const int slot = p.row_slot[r];
     if (slot < 0) return;
     const int q_start = p.row_q_start[r], q_len = p.row_q_len[r];
-    if (p.blocks != nullptr && q_len > DR_SINGLE) return;    // a row of the block form
+    if (p.short_only && q_len > DR_SINGLE) return;           // a row of another form
     const int hk = h / (p.H / p.Hk);
     const int tid = threadIdx.x;
     const int vl = tid / DR_DS, ds = tid % DR_DS;
@@ -266,6 +267,12 @@ delta_scan_kernel(const DeltaScan p) {
         float* buf = sm + (it & 1) * DR_TC * TS;
         if (c0 + DR_TC < q_len) { issue(c0 + DR_TC, (it + 1) & 1); cp_async_wait<1>(); }
         else cp_async_wait<0>();
+        __syncthreads();
+        for (int i = tid; i < n * p.dp; i += DR_THREADS) {   // the decays from their logarithms
+            const int tt = i / p.dp, ch = i - tt * p.dp;
+            float* at = buf + tt * TS + 2 * CS + (ch / NR) * dr_stride<NR>() + ch % NR;
+            *at = expf(*at);
+        }
         __syncthreads();
         const float* mine = buf + ds * dr_stride<NR>();
 #pragma unroll 1
@@ -332,7 +339,7 @@ delta_blocks_kernel(const DeltaScan p) {
             const size_t t = q_start + b * DB_TOK + i;
             k[i] = p.k[(t * p.Hk + hk) * p.dp + tid];
             q[i] = p.q[(t * p.Hk + hk) * p.dp + tid];
-            g[i] = p.g[(t * p.H + h) * p.dp + tid];
+            g[i] = expf(p.g[(t * p.H + h) * p.dp + tid]);
         }
     }
     const size_t slot = (size_t)block_slot(q_start, r, b) * p.H + h;
@@ -388,11 +395,37 @@ delta_blocks_kernel(const DeltaScan p) {
     }
 }
 
-template <int NR>
-__global__ void __launch_bounds__(DB_THREADS)
+// two floats in one register pair: sm_100 multiplies and adds both in one instruction
+typedef unsigned long long f32x2;
+__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
+    f32x2 d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+    return d;
+}
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
+    f32x2 d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+__device__ __forceinline__ f32x2 pair2(float lo, float hi) {
+    f32x2 d;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
+    return d;
+}
+__device__ __forceinline__ float2 split2(f32x2 a) {
+    float2 d;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(d.x), "=f"(d.y) : "l"(a));
+    return d;
+}
+
+// DS lanes share a column and hold NR rows of it each.  What bounds the time is the chain of a block's own steps (loads, sums, the
+// reduction, the four corrections, the update), one block after the other: so the sums run in eight chains side by side.
+template <int NR, int DS>
+__global__ void __launch_bounds__(DS * DB_VT)
 delta_block_scan_kernel(const DeltaScan p) {
-    constexpr int CS = DR_DS * dr_stride<NR>();
-    constexpr int VT = DB_THREADS / DR_DS * 2;               // value columns of a CTA
+    constexpr int DB_THREADS = DS * DB_VT, WARPS = DB_THREADS / 32;
+    constexpr int CS = DS * dr_stride<NR>();
+    constexpr int VT = DB_VT;
     constexpr int BS = DB_VECS * CS + DB_TOK * VT + DB_SCAL; // floats of a block in shared memory
     extern __shared__ __align__(16) float sm[];
     const int tiles = (p.dv + VT - 1) / VT;
@@ -400,18 +433,17 @@ delta_block_scan_kernel(const DeltaScan p) {
     const int slot = p.row_slot[r];
     const int q_start = p.row_q_start[r], q_len = p.row_q_len[r];
     if (slot < 0 || q_len <= DR_SINGLE) return;
-    const int tid = threadIdx.x, vl = tid / DR_DS, ds = tid % DR_DS;
-    const int col = tile * VT + vl * 2;
-    const bool live0 = col < p.dv, live1 = col + 1 < p.dv;
+    const int tid = threadIdx.x, lane = tid & 31, vl = tid / DS, ds = tid % DS;
+    const int col = tile * VT + vl;
+    const bool live = col < p.dv;
     float* st = p.state + ((size_t)slot * p.H + h) * p.d * p.dv;
-    float S[NR][2];
+    f32x2 S[NR / 2];                                         // rows ds * NR + 2 i and the next of the thread's column
 #pragma unroll
-    for (int i = 0; i < NR; ++i) {
-        const int row = ds * NR + i;
-        S[i][0] = live0 && row < p.d ? st[(size_t)row * p.dv + col] : 0.f;
-        S[i][1] = live1 && row < p.d ? st[(size_t)row * p.dv + col + 1] : 0.f;
+    for (int i = 0; i < NR / 2; ++i) {
+        const int row = ds * NR + 2 * i;
+        S[i] = pair2(live && row < p.d ? st[(size_t)row * p.dv + col] : 0.f, live && row + 1 < p.d ? st[(size_t)(row + 1) * p.dv + col] : 0.f);
     }
-    if (p.dp < DR_DS * NR) {                                 // places of channels at or beyond dp are never filled: zero once
+    if (p.dp < DS * NR) {                                 // places of channels at or beyond dp are never filled: zero once
         for (int e = tid; e < DB_STAGES * BS; e += DB_THREADS) sm[e] = 0.f;
         __syncthreads();
     }
@@ -423,21 +455,23 @@ delta_block_scan_kernel(const DeltaScan p) {
             float* dst = sm + (b % DB_STAGES) * BS;
             const size_t bs = (slot0 + b) * p.H + h;
             const float* src = p.blocks + bs * DB_VECS * p.dp;
-            for (int piece = tid; piece < per; piece += DB_THREADS) {
+            for (int piece = lane; piece < per; piece += 32) {      // the warps take the vectors in turn
                 const int i = piece * 4;
-                uint32_t at = smem_u32(dst + (i / NR) * dr_stride<NR>() + i % NR);
-                const float* s = src + i;
+                const uint32_t at = smem_u32(dst + (i / NR) * dr_stride<NR>() + i % NR);
+                const float* from = src + i;
 #pragma unroll
-                for (int v = 0; v < DB_VECS; ++v, s += p.dp, at += CS * 4) cp_async16(at, s, 16);
+                for (int e = 0; e < (DB_VECS + WARPS - 1) / WARPS; ++e) {
+                    const int v = (tid >> 5) + e * WARPS;
+                    if (v < DB_VECS) cp_async16(at + v * CS * 4, from + v * p.dp, 16);
+                }
             }
-            if (tid >= DB_THREADS - 4 * VT / 4) {            // v: VT / 4 pieces of each of the four tokens
-                const int e = tid - (DB_THREADS - 4 * VT / 4), tt = e / (VT / 4), i = (e % (VT / 4)) * 4;
-                const int t = b * DB_TOK + tt;
+            if (tid >= 32 && tid < 32 + DB_TOK * VT / 4) {
+                const int e = tid - 32, tt = e / (VT / 4), i = (e % (VT / 4)) * 4, t = b * DB_TOK + tt;
                 const bool in = tile * VT + i < p.dvp && t < q_len;
                 cp_async16(smem_u32(dst + DB_VECS * CS + tt * VT + i),
                            in ? p.v + ((size_t)(q_start + t) * p.H + h) * p.dvp + tile * VT + i : p.v, in ? 16 : 0);
-            } else if (tid >= 32 && tid < 32 + DB_SCAL / 4) {
-                const int e = tid - 32;
+            } else if (tid >= 48 && tid < 48 + DB_SCAL / 4) {
+                const int e = tid - 48;
                 cp_async16(smem_u32(dst + DB_VECS * CS + DB_TOK * VT + e * 4), p.scal + bs * DB_SCAL + e * 4, 16);
             }
         }
@@ -451,82 +485,90 @@ delta_block_scan_kernel(const DeltaScan p) {
         issue(b + DB_STAGES - 1);
         const float* buf = sm + (b % DB_STAGES) * BS;
         const float* mine = buf + ds * dr_stride<NR>();
-        float dk[4][2], dq[4][2];
+        f32x2 ak[4], aq[4];
 #pragma unroll
-        for (int t = 0; t < 4; ++t) dk[t][0] = dk[t][1] = dq[t][0] = dq[t][1] = 0.f;
+        for (int t = 0; t < 4; ++t) ak[t] = aq[t] = 0ull;    // two zeros
 #pragma unroll
         for (int i = 0; i < NR; i += 4) {
+            ulonglong2 k4[4], q4[4];
 #pragma unroll
             for (int t = 0; t < 4; ++t) {
-                const float4 k4 = *reinterpret_cast<const float4*>(mine + t * CS + i);
-                const float4 q4 = *reinterpret_cast<const float4*>(mine + (4 + t) * CS + i);
-#pragma unroll
-                for (int c = 0; c < 2; ++c) {
-                    dk[t][c] = fmaf(S[i + 3][c], k4.w, fmaf(S[i + 2][c], k4.z, fmaf(S[i + 1][c], k4.y, fmaf(S[i][c], k4.x, dk[t][c]))));
-                    dq[t][c] = fmaf(S[i + 3][c], q4.w, fmaf(S[i + 2][c], q4.z, fmaf(S[i + 1][c], q4.y, fmaf(S[i][c], q4.x, dq[t][c]))));
-                }
+                k4[t] = *reinterpret_cast<const ulonglong2*>(mine + t * CS + i);
+                q4[t] = *reinterpret_cast<const ulonglong2*>(mine + (4 + t) * CS + i);
             }
+#pragma unroll
+            for (int t = 0; t < 4; ++t) { ak[t] = fma2(S[i / 2], k4[t].x, ak[t]); aq[t] = fma2(S[i / 2], q4[t].x, aq[t]); }
+#pragma unroll
+            for (int t = 0; t < 4; ++t) { ak[t] = fma2(S[i / 2 + 1], k4[t].y, ak[t]); aq[t] = fma2(S[i / 2 + 1], q4[t].y, aq[t]); }
+        }
+        // what the update needs from memory, and the decay, while the reduction runs
+        ulonglong2 w4[4][NR / 4];
+#pragma unroll
+        for (int t = 0; t < 4; ++t)
+#pragma unroll
+            for (int i = 0; i < NR / 4; ++i) w4[t][i] = *reinterpret_cast<const ulonglong2*>(mine + (8 + t) * CS + i * 4);
+#pragma unroll
+        for (int i = 0; i < NR / 4; ++i) {
+            const ulonglong2 c4 = *reinterpret_cast<const ulonglong2*>(mine + 12 * CS + i * 4);
+            S[2 * i] = mul2(S[2 * i], c4.x);
+            S[2 * i + 1] = mul2(S[2 * i + 1], c4.y);
+        }
+        float dk[4], dq[4];
+#pragma unroll
+        for (int t = 0; t < 4; ++t) {
+            const float2 a = split2(ak[t]), c = split2(aq[t]);
+            dk[t] = a.x + a.y;
+            dq[t] = c.x + c.y;
         }
 #pragma unroll
-        for (int off = 1; off < DR_DS; off <<= 1)
+        for (int off = 1; off < DS; off <<= 1)
 #pragma unroll
-            for (int t = 0; t < 4; ++t)
-#pragma unroll
-                for (int c = 0; c < 2; ++c) {
-                    dk[t][c] += __shfl_xor_sync(0xffffffffu, dk[t][c], off);
-                    dq[t][c] += __shfl_xor_sync(0xffffffffu, dq[t][c], off);
-                }
-        const float* v_s = buf + DB_VECS * CS + vl * 2;
+            for (int t = 0; t < 4; ++t) {
+                dk[t] += __shfl_xor_sync(0xffffffffu, dk[t], off);
+                dq[t] += __shfl_xor_sync(0xffffffffu, dq[t], off);
+            }
+        const float* v_s = buf + DB_VECS * CS + vl;
         const float4* sc = reinterpret_cast<const float4*>(buf + DB_VECS * CS + DB_TOK * VT);
         const float4 s0 = sc[0], s1 = sc[1], s2 = sc[2], s3 = sc[3], be = sc[4];
         const float A[6] = {s0.x, s0.y, s0.z, s0.w, s1.x, s1.y};
         const float P[10] = {s1.z, s1.w, s2.x, s2.y, s2.z, s2.w, s3.x, s3.y, s3.z, s3.w};
         const float beta[4] = {be.x, be.y, be.z, be.w};
-        float u[4][2], o[4][2];
+        float u[4];
 #pragma unroll
-        for (int c = 0; c < 2; ++c)
+        for (int i = 0; i < 4; ++i) {
+            float s = v_s[i * VT] - dk[i];
 #pragma unroll
-            for (int i = 0; i < 4; ++i) {
-                float s = v_s[i * VT + c] - dk[i][c];
-#pragma unroll
-                for (int j = 0; j < 4; ++j) if (j < i) s = fmaf(-A[i * (i - 1) / 2 + j], u[j][c], s);
-                u[i][c] = beta[i] * s;
-                float a = dq[i][c];
-#pragma unroll
-                for (int j = 0; j < 4; ++j) if (j <= i) a = fmaf(P[i * (i + 1) / 2 + j], u[j][c], a);
-                o[i][c] = a;
-            }
-#pragma unroll
-        for (int i = 0; i < NR; i += 4) {
-            const float4 c4 = *reinterpret_cast<const float4*>(mine + 12 * CS + i);
-#pragma unroll
-            for (int c = 0; c < 2; ++c) { S[i][c] *= c4.x; S[i + 1][c] *= c4.y; S[i + 2][c] *= c4.z; S[i + 3][c] *= c4.w; }
-#pragma unroll
-            for (int t = 0; t < 4; ++t) {
-                const float4 k4 = *reinterpret_cast<const float4*>(mine + (8 + t) * CS + i);
-#pragma unroll
-                for (int c = 0; c < 2; ++c) {
-                    S[i][c] = fmaf(k4.x, u[t][c], S[i][c]); S[i + 1][c] = fmaf(k4.y, u[t][c], S[i + 1][c]);
-                    S[i + 2][c] = fmaf(k4.z, u[t][c], S[i + 2][c]); S[i + 3][c] = fmaf(k4.w, u[t][c], S[i + 3][c]);
-                }
-            }
+            for (int j = 0; j < 4; ++j) if (j < i) s = fmaf(-A[i * (i - 1) / 2 + j], u[j], s);
+            u[i] = beta[i] * s;
         }
-        if (ds < 4 && b * DB_TOK + ds < q_len) {             // lane t of the first four writes token t's two columns
-            float a = o[0][0], c = o[0][1];
 #pragma unroll
-            for (int t = 1; t < 4; ++t) if (ds == t) { a = o[t][0]; c = o[t][1]; }
-            float* out = p.out + ((size_t)(q_start + b * DB_TOK + ds) * p.H + h) * p.dv + col;
-            if (live0) out[0] = a;
-            if (live1) out[1] = c;
+        for (int i = 0; i < 4; ++i) {
+#pragma unroll
+            for (int j = 0; j < 4; ++j) if (j <= i) dq[i] = fmaf(P[i * (i + 1) / 2 + j], u[j], dq[i]);
+        }
+        f32x2 uu[4];
+#pragma unroll
+        for (int t = 0; t < 4; ++t) uu[t] = pair2(u[t], u[t]);
+#pragma unroll
+        for (int t = 0; t < 4; ++t)
+#pragma unroll
+            for (int i = 0; i < NR / 4; ++i) {
+                S[2 * i] = fma2(w4[t][i].x, uu[t], S[2 * i]);
+                S[2 * i + 1] = fma2(w4[t][i].y, uu[t], S[2 * i + 1]);
+            }
+        if (ds < 4 && b * DB_TOK + ds < q_len && live) {     // lane t of the first four writes token t
+            const float o = ds == 0 ? dq[0] : ds == 1 ? dq[1] : ds == 2 ? dq[2] : dq[3];
+            p.out[((size_t)(q_start + b * DB_TOK + ds) * p.H + h) * p.dv + col] = o;
         }
     }
     cp_async_wait<0>();
-    if (p.write_state) {
+    if (p.write_state && live) {
 #pragma unroll
-        for (int i = 0; i < NR; ++i) {
-            const int row = ds * NR + i;
-            if (row < p.d && live0) st[(size_t)row * p.dv + col] = S[i][0];
-            if (row < p.d && live1) st[(size_t)row * p.dv + col + 1] = S[i][1];
+        for (int i = 0; i < NR / 2; ++i) {
+            const int row = ds * NR + 2 * i;
+            const float2 x = split2(S[i]);
+            if (row < p.d) st[(size_t)row * p.dv + col] = x.x;
+            if (row + 1 < p.d) st[(size_t)(row + 1) * p.dv + col] = x.y;
         }
     }
 }
@@ -558,9 +600,9 @@ static int launch_delta_scan(const DeltaScan& p, int n_rows, cudaStream_t stream
     const dim3 one(1, 1, 1);
     int rc = launch("delta_scan", k, dim3((unsigned)tiles * n_rows, p.H), dim3(DR_THREADS), smem, stream, one, p);
     if (rc || p.blocks == nullptr) return rc;
-    constexpr int VT = DB_THREADS / DR_DS * 2;
-    constexpr size_t bsmem = DB_STAGES * (size_t)(DB_VECS * DR_DS * dr_stride<NR>() + DB_TOK * VT + DB_SCAL) * sizeof(float);
-    auto kb = delta_block_scan_kernel<NR>;
+    constexpr int BNR = NR > 8 ? NR / 2 : NR, BDS = NR > 8 ? 2 * DR_DS : DR_DS;      // block form: fewer rows in more lanes
+    constexpr size_t bsmem = DB_STAGES * (size_t)(DB_VECS * BDS * dr_stride<BNR>() + DB_TOK * DB_VT + DB_SCAL) * sizeof(float);
+    auto kb = delta_block_scan_kernel<BNR, BDS>;
     static bool block_configured = false;
     if (!block_configured) {
         cudaError_t e = cudaFuncSetAttribute(kb, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bsmem);
@@ -569,7 +611,7 @@ static int launch_delta_scan(const DeltaScan& p, int n_rows, cudaStream_t stream
     }
     rc = launch("delta_blocks", delta_blocks_kernel, dim3((unsigned)n_rows * p.max_blocks, p.H), dim3((p.dp + 31) / 32 * 32), 0, stream, one, p);
     if (rc) return rc;
-    return launch("delta_block_scan", kb, dim3((unsigned)((p.dv + VT - 1) / VT) * n_rows, p.H), dim3(DB_THREADS), bsmem, stream, one, p);
+    return launch("delta_block_scan", kb, dim3((unsigned)((p.dv + DB_VT - 1) / DB_VT) * n_rows, p.H), dim3(BDS * DB_VT), bsmem, stream, one, p);
 }
 
 }  // namespace fd
@@ -579,7 +621,7 @@ typedef __nv_bfloat16 bf16;
 
 // dtype (0 float32, 1 bfloat16): type of proj, a2 and g2.  Columns count from the pointer.  conv_w [2 Hk d + H dv, taps]; ring
 // [slots, taps, 2 Hk d + H dv] (unused when taps == 1).  a2 [H d, R] or null with z_a [T, H d]; g2 [H dv, R2] or null (the gate's
-// pre-activation is then not made here).  Outputs: q, k [T, Hk, dp], g [T, H, dp] with dp = d rounded up to 4 (zeros after d), v
+// pre-activation is then not made here).  Outputs: q, k [T, Hk, dp], g [T, H, dp] with dp = d rounded up to 4 (zeros after d; g: log decays), v
 // [T, H, dvp], dvp = dv rounded up to 4, beta [T, H], gate_z [T, H dv]; all float.  keep: rows of a single token leave their
 // values in the ring here; longer rows need fd_conv_ring_update.
 extern "C" int fd_delta_prepare(const void* proj, int ld, int dtype, int q_col, int k_col, int v_col, int b_col, int a_col, int g_col,
@@ -619,7 +661,8 @@ extern "C" int fd_delta_prepare(const void* proj, int ld, int dtype, int q_col, 
 
 // q, k [T, Hk, dp], g [T, H, dp], v [T, H, dvp], beta [T, H] as fd_delta_prepare leaves them; state [slots, H, d, dv] and
 // out [T, H dv] float.  max_q_len: the longest row of the step; rows of more than 16 tokens take the block form and need scratch
-// memory, fd_delta_scan_scratch_floats floats (without it every row is walked token by token).
+// memory, fd_delta_scan_scratch_floats floats (without it every row is walked token by token).  short_only: rows of more
+// than 16 tokens are left out (fd_delta_chunks takes them).
 extern "C" int fd_delta_scan_single() { return DR_SINGLE; }
 extern "C" long long fd_delta_scan_scratch_floats(int T, int n_rows, int H, int d) {
     return (long long)(T / DB_TOK + n_rows + 1) * H * (DB_VECS * ((d + 3) / 4 * 4) + DB_SCAL);
@@ -627,6 +670,7 @@ extern "C" long long fd_delta_scan_scratch_floats(int T, int n_rows, int H, int 
 extern "C" int fd_delta_scan(const float* q, const float* k, const float* v, const float* g, const float* beta, float* state,
                              float* out, const int* row_slot, const int* row_q_start, const int* row_q_len, int n_rows, int H,
                              int Hk, int d, int dv, int write_state, int T, int max_q_len, float* scratch, long long scratch_floats,
+                             int short_only,
                              cudaStream_t stream) {
     if (n_rows == 0) return 0;
     FD_REQUIRE(H > 0 && Hk > 0 && H % Hk == 0 && d > 0 && d <= 256 && dv > 0, -2, "delta_scan: %d heads on %d of %d x %d (keys up to 256)", H, Hk, d, dv);
@@ -634,8 +678,8 @@ extern "C" int fd_delta_scan(const float* q, const float* k, const float* v, con
     auto al = [](const void* x) { return (uintptr_t)x % 16 == 0; };
     FD_REQUIRE(al(q) && al(k) && al(v) && al(g), -2, "delta_scan: 16-byte alignment");
     DeltaScan p = {q, k, v, g, beta, state, out, row_slot, row_q_start, row_q_len, H, Hk, d, dv, (d + 3) / 4 * 4, (dv + 3) / 4 * 4, write_state,
-                   nullptr, nullptr, 0};
-    if (scratch != nullptr && max_q_len > DR_SINGLE) {
+                   nullptr, nullptr, 0, short_only || scratch != nullptr};
+    if (scratch != nullptr && !short_only && max_q_len > DR_SINGLE) {
         FD_REQUIRE(scratch_floats >= fd_delta_scan_scratch_floats(T, n_rows, H, d) && (uintptr_t)scratch % 16 == 0, -2,
                    "delta_scan: %lld floats of scratch memory for %d tokens", scratch_floats, T);
         p.blocks = scratch;

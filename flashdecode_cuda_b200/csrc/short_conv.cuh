@@ -98,7 +98,10 @@ __device__ __forceinline__ void conv_channel(const T* __restrict__ col, int ld, 
     }
 }
 
-__device__ __forceinline__ float sc_silu(float z) { return z / (1.f + expf(-z)); }
+// z sigmoid(z); behind bfloat16 projections with the special function unit's exponential and reciprocal (a few units in the
+// last place of a float)
+template <typename T> __device__ __forceinline__ float sc_silu(float z) { return z / (1.f + expf(-z)); }
+template <> __device__ __forceinline__ float sc_silu<__nv_bfloat16>(float z) { return z * __frcp_rn(1.f + __expf(-z)); }
 __device__ __forceinline__ float sc_sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
 __device__ __forceinline__ float sc_softplus(float z) { return z > 0.f ? z + log1pf(expf(-z)) : log1pf(expf(z)); }
 

@@ -54,7 +54,7 @@ ssd_prepare_kernel(const T* __restrict__ proj, int ld, int col, int C, int dt_co
 #pragma unroll
     for (int tt = 0; tt < SC_TOK; ++tt)
         if (tt < nt && meta.slot[tt] >= 0) {
-            const float v = sc_silu(y[tt]);
+            const float v = sc_silu<T>(y[tt]);
             if (c < float_cols) xbc[(size_t)(t0 + tt) * C + c] = v;
             if (xbc16 != nullptr) xbc16[(size_t)(t0 + tt) * C + c] = __float2bfloat16_rn(v);
         }
@@ -71,10 +71,10 @@ ssd_gate_norm_kernel(const float* __restrict__ y, const float* __restrict__ xbc,
     const size_t t = blockIdx.y;
     const int c0 = blockIdx.x * part;
     float ss = 0.f;
+#pragma unroll 4
     for (int j = threadIdx.x; j < part; j += blockDim.x) {
         const int c = c0 + j;
-        const float gate = to_float(z[t * ldz + c]);
-        const float v = fmaf(D[c / dv], xbc[t * ldx + c], y[t * inner + c]) * (gate / (1.f + expf(-gate)));
+        const float v = fmaf(D[c / dv], xbc[t * ldx + c], y[t * inner + c]) * sc_silu<T>(to_float(z[t * ldz + c]));
         g_s[j] = v;
         ss = fmaf(v, v, ss);
     }
@@ -162,14 +162,28 @@ ssd_chunk_state_kernel(const SsdChunks p) {
     chunk_decays(p, tok0, n, h, cs, dts);
     __syncthreads();
     const float last = cs[SC_L - 1];
-    for (int e = threadIdx.x; e < SC_L * SC_DV / 2; e += SCH_THREADS) {
-        const int t = e / (SC_DV / 2), j = (e - t * (SC_DV / 2)) * 2;
-        const __nv_bfloat16* src = p.xbc + (size_t)(tok0 + t) * p.ld + h * p.dv + v0 + j;
-        const float w = t < n ? expf(last - cs[t]) * dts[t] : 0.f;
-        const float a = t < n && j < vw ? w * __bfloat162float(src[0]) : 0.f, b = t < n && j + 1 < vw ? w * __bfloat162float(src[1]) : 0.f;
-        const int at = swz<SC_DV>(t, j >> 3) + (j & 7) * 2;
-        *reinterpret_cast<uint32_t*>(x_s + at) = pack_bf16(a, b);
-        *reinterpret_cast<uint32_t*>(x_r + at) = pack_bf16_rest(a, b);
+    constexpr int UNR = 8;                     // loads in flight per thread
+#pragma unroll 1
+    for (int e0 = threadIdx.x; e0 < SC_L * SC_DV / 2; e0 += SCH_THREADS * UNR) {
+        float2 x[UNR];
+#pragma unroll
+        for (int k = 0; k < UNR; ++k) {
+            const int e = e0 + k * SCH_THREADS, t = e / (SC_DV / 2), j = (e - t * (SC_DV / 2)) * 2;
+            const __nv_bfloat16* src = p.xbc + (size_t)(tok0 + t) * p.ld + h * p.dv + v0 + j;
+            x[k] = make_float2(0.f, 0.f);
+            if (t < n && j < vw) {
+                if (p.aligned) x[k] = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(src));
+                else x[k] = make_float2(__bfloat162float(src[0]), j + 1 < vw ? __bfloat162float(src[1]) : 0.f);
+            }
+        }
+#pragma unroll
+        for (int k = 0; k < UNR; ++k) {
+            const int e = e0 + k * SCH_THREADS, t = e / (SC_DV / 2), j = (e - t * (SC_DV / 2)) * 2;
+            const float w = expf(last - cs[t]) * dts[t];
+            const int at = swz<SC_DV>(t, j >> 3) + (j & 7) * 2;
+            *reinterpret_cast<uint32_t*>(x_s + at) = pack_bf16(w * x[k].x, w * x[k].y);
+            *reinterpret_cast<uint32_t*>(x_r + at) = pack_bf16_rest(w * x[k].x, w * x[k].y);
+        }
     }
     cp_async_wait<0>();
     __syncthreads();
@@ -257,12 +271,26 @@ ssd_chunk_out_kernel(const SsdChunks p) {
     cp_async_commit();
     chunk_decays(p, tok0, n, h, cs, dts);
     const float* st = p.u + ((size_t)chunk_slot(q_start, r, c) * p.H + h) * p.N * p.dv + v0;
-    for (int e = threadIdx.x; e < NP * SC_DV / 2; e += SCH_THREADS) {
-        const int m = e / (SC_DV / 2), j = (e - m * (SC_DV / 2)) * 2;
-        const float a = m < p.N && j < vw ? st[(size_t)m * p.dv + j] : 0.f, b = m < p.N && j + 1 < vw ? st[(size_t)m * p.dv + j + 1] : 0.f;
-        const int at = swz<SC_DV>(m, j >> 3) + (j & 7) * 2;
-        *reinterpret_cast<uint32_t*>(s_s + at) = pack_bf16(a, b);
-        *reinterpret_cast<uint32_t*>(s_r + at) = pack_bf16_rest(a, b);
+    constexpr int UNR = 8;                     // loads in flight per thread
+#pragma unroll 1
+    for (int e0 = threadIdx.x; e0 < NP * SC_DV / 2; e0 += SCH_THREADS * UNR) {
+        float2 x[UNR];
+#pragma unroll
+        for (int k = 0; k < UNR; ++k) {
+            const int e = e0 + k * SCH_THREADS, m = e / (SC_DV / 2), j = (e - m * (SC_DV / 2)) * 2;
+            x[k] = make_float2(0.f, 0.f);
+            if (m < p.N && j < vw) {
+                if (p.aligned) x[k] = *reinterpret_cast<const float2*>(st + (size_t)m * p.dv + j);
+                else x[k] = make_float2(st[(size_t)m * p.dv + j], j + 1 < vw ? st[(size_t)m * p.dv + j + 1] : 0.f);
+            }
+        }
+#pragma unroll
+        for (int k = 0; k < UNR; ++k) {
+            const int e = e0 + k * SCH_THREADS, m = e / (SC_DV / 2), j = (e - m * (SC_DV / 2)) * 2;
+            const int at = swz<SC_DV>(m, j >> 3) + (j & 7) * 2;
+            *reinterpret_cast<uint32_t*>(s_s + at) = pack_bf16(x[k].x, x[k].y);
+            *reinterpret_cast<uint32_t*>(s_r + at) = pack_bf16_rest(x[k].x, x[k].y);
+        }
     }
     cp_async_wait<0>();
     __syncthreads();

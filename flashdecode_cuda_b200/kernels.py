@@ -108,8 +108,10 @@ def _declare(L: ctypes.CDLL) -> None:
         "fd_row_norm_gate": [P, P, P, I, P, I, I, I, F, P],
         "fd_head_norm_gate": [P, P, P, I, P, P, I, I, I, I, I, F, F, P],
         "fd_delta_prepare": [P, I, I, I, I, I, I, I, I, P, P, I, I, P, I, P, P, I, P, P, F, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, P],
-        "fd_delta_scan": [P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, P, LL, P],
+        "fd_delta_scan": [P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, P, LL, I, P],
         "fd_delta_scan_single": [],
+        "fd_delta_chunks_takes": [I],
+        "fd_delta_chunks": [P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, P, LL, P],
         "fd_conv_ring_update": [P, I, I, P, P, P, P, P, I, I, I, P],
         "fd_ssd_prepare": [P, I, I, I, I, I, P, P, P, I, I, P, P, P, P, I, P, P, P, P, P, P, I, I, P],
         "fd_ssd_chunks_takes": [I, I],
@@ -164,6 +166,8 @@ def _declare(L: ctypes.CDLL) -> None:
     L.fd_delta_scan_scratch_floats.restype = LL
     L.fd_ssd_chunks_scratch_floats.argtypes = [I, I, I, I, I]
     L.fd_ssd_chunks_scratch_floats.restype = LL
+    L.fd_delta_chunks_scratch_bytes.argtypes = [I, I, I, I]
+    L.fd_delta_chunks_scratch_bytes.restype = LL
     L.fd_sample_scratch_words.argtypes = [I, I]
     L.fd_sample_scratch_words.restype = LL
 
@@ -1053,7 +1057,7 @@ def delta_prepare(proj: torch.Tensor, cols, conv_w: torch.Tensor, ring: Optional
     """What enters the gated delta rule, as float32.  ``cols``: first columns in ``proj`` [T, ld] of q, k, v, beta's
     pre-activation, and the narrow vectors of decay and gate.  q, k, v: a causal convolution per channel (``conv_w`` float32
     [C, taps], C = 2 n_qk_heads head_dim + n_heads v_head_dim; earlier values from ``ring`` float32 [slots, taps, C]) and silu;
-    every head of q and k a unit vector, q times ``q_scale``.  g = exp(-exp(A_log[h]) softplus(z + dt_bias)) per key channel,
+    every head of q and k a unit vector, q times ``q_scale``.  g (the decay's logarithm) = -exp(A_log[h]) softplus(z + dt_bias) per key channel,
     z = ``a2`` [n_heads head_dim, R] times the narrow vector, or ``z_a`` float32 [T, n_heads head_dim].  beta = its sigmoid.
     ``gate_z`` [T, n_heads v_head_dim] <- ``g2`` times the gate's narrow vector, if g2 is given.  ``keep``: rows that bring a
     single token leave their values in the ring (longer rows: ``conv_ring_update``).  Outputs q, k [T, n_qk_heads, dp],
@@ -1084,11 +1088,12 @@ def delta_prepare(proj: torch.Tensor, cols, conv_w: torch.Tensor, ring: Optional
 
 def delta_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, g: torch.Tensor, beta: torch.Tensor, state: torch.Tensor,
                out: torch.Tensor, row_slot: torch.Tensor, row_q_start: torch.Tensor, row_q_len: torch.Tensor, n_rows: int,
-               write_state: bool, max_q_len: int = 0, scratch: Optional[torch.Tensor] = None) -> None:
-    """S <- diag(g) S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q, per sequence and head over the step's tokens, from
+               write_state: bool, max_q_len: int = 0, scratch: Optional[torch.Tensor] = None, short_only: bool = False) -> None:
+    """S <- diag(exp(g)) S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q, per sequence and head over the step's tokens, from
     ``state`` [slots, heads, d, dv] (float32, updated when ``write_state``) to ``out`` [T, heads * dv] float32.  The inputs are
     those ``delta_prepare`` leaves.  With ``scratch`` (float32, ``delta_scan_scratch_floats`` elements) and ``max_q_len`` (the longest
-    row), rows of more than ``delta_scan_single()`` tokens are walked four tokens at a time."""
+    row), rows of more than ``delta_scan_single()`` tokens are walked four tokens at a time; with ``short_only`` they are left out
+    (``delta_chunks`` takes them)."""
     H, d, dv = state.shape[1:]
     T, Hk = q.shape[:2]
     for t in (q, k, v, g, beta, state, out):
@@ -1096,7 +1101,7 @@ def delta_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, g: torch.Tenso
     assert out.shape == (T, H * dv) and k.shape == q.shape and g.shape[:2] == (T, H) and v.shape[:2] == (T, H)
     _check(lib().fd_delta_scan(_ptr(q), _ptr(k), _ptr(v), _ptr(g), _ptr(beta), _ptr(state), _ptr(out), _ptr(row_slot),
                                _ptr(row_q_start), _ptr(row_q_len), n_rows, H, Hk, d, dv, int(write_state), T, int(max_q_len), _ptr(scratch),
-                               scratch.numel() if scratch is not None else 0, _stream()))
+                               scratch.numel() if scratch is not None else 0, int(short_only), _stream()))
 
 
 def delta_scan_single() -> int:
@@ -1105,6 +1110,30 @@ def delta_scan_single() -> int:
 
 def delta_scan_scratch_floats(T: int, n_rows: int, n_heads: int, head_dim: int) -> int:
     return int(lib().fd_delta_scan_scratch_floats(T, n_rows, n_heads, head_dim))
+
+
+def delta_chunks_takes(head_dim: int) -> bool:
+    """Whether ``delta_chunks`` takes heads of this key size."""
+    return bool(lib().fd_delta_chunks_takes(head_dim))
+
+
+def delta_chunks_scratch_bytes(T: int, n_rows: int, n_heads: int, head_dim: int) -> int:
+    return int(lib().fd_delta_chunks_scratch_bytes(T, n_rows, n_heads, head_dim))
+
+
+def delta_chunks(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, g: torch.Tensor, beta: torch.Tensor, state: torch.Tensor,
+                 out: torch.Tensor, row_slot: torch.Tensor, row_q_start: torch.Tensor, row_q_len: torch.Tensor, n_rows: int,
+                 write_state: bool, max_q_len: int, scratch: torch.Tensor) -> None:
+    """``delta_scan`` of the rows with more than ``delta_scan_single()`` tokens, sixteen tokens at a time on the tensor cores;
+    ``scratch`` uint8, ``delta_chunks_scratch_bytes`` elements."""
+    H, d, dv = state.shape[1:]
+    T, Hk = q.shape[:2]
+    for t in (q, k, v, g, beta, state, out):
+        assert t.dtype == torch.float32
+    assert out.shape == (T, H * dv) and k.shape == q.shape and g.shape[:2] == (T, H) and v.shape[:2] == (T, H)
+    _check(lib().fd_delta_chunks(_ptr(q), _ptr(k), _ptr(v), _ptr(g), _ptr(beta), _ptr(state), _ptr(out), _ptr(row_slot), _ptr(row_q_start),
+                                 _ptr(row_q_len), n_rows, T, int(max_q_len), H, Hk, d, dv, int(write_state), delta_scan_single(),
+                                 _ptr(scratch), scratch.numel() * scratch.element_size(), _stream()))
 
 
 def conv_ring_update(proj: torch.Tensor, first_col: int, ring: torch.Tensor, row_slot: torch.Tensor, row_q_start: torch.Tensor,

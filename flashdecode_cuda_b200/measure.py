@@ -23,7 +23,7 @@ LAUNCHERS = ["embed", "add_rmsnorm", "silu_mul", "rope_append", "gemv_qkv_rope",
              "moe_gather", "gemm_tc_grouped", "glu_mul", "softcap", "lanes_norm", "lanes_fill", "norm_append", "head_gemm",
              "attention_ext", "attn_head_mix", "add_dyn_tanh", "quad_exp_act", "scale_", "axpy_f32", "linear_scan",
              "head_norm_gate", "row_norm_gate", "rope_heads", "post_norm", "stream_conv", "attention_dense", "add_cast", "side_gate_mul", "token_side_row", "add_row_vector", "low_rank_expand",
-             "rope_norm_append", "delta_prepare", "delta_scan", "conv_ring_update", "ssd_prepare", "ssd_chunks", "ssd_gate_norm", "relu2_cols"]
+             "rope_norm_append", "delta_prepare", "delta_scan", "delta_chunks", "conv_ring_update", "ssd_prepare", "ssd_chunks", "ssd_gate_norm", "relu2_cols"]
 
 
 class PartTimer:

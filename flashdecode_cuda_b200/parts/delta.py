@@ -127,11 +127,16 @@ class GatedDeltaRule(Mixer):
         if ring is not None and lc.writes and ctx.max_q_len > 1:
             K.conv_ring_update(proj, col0, ring, ctx.row_slot, ctx.row_q_start, ctx.row_q_len, ctx.row_ctx_len, ctx.n_rows)
         o = ws.get("scan_out", (T, H * dv), f32)
-        scratch = None
-        if ctx.max_q_len > K.delta_scan_single():
-            scratch = ws.get("delta_blocks", (K.delta_scan_scratch_floats(T, ctx.n_rows, H, d),), f32)
-        K.delta_scan(q, k, v, g, beta, lc.states["state"], o, ctx.row_slot, ctx.row_q_start, ctx.row_q_len, ctx.n_rows, lc.writes,
-                     ctx.max_q_len, scratch)
+        step = (q, k, v, g, beta, lc.states["state"], o, ctx.row_slot, ctx.row_q_start, ctx.row_q_len, ctx.n_rows, lc.writes)
+        long = ctx.max_q_len > K.delta_scan_single()
+        if long and proj.dtype == torch.bfloat16 and K.delta_chunks_takes(d):
+            if min(ctx.h_q_len, default=0) <= K.delta_scan_single():
+                K.delta_scan(*step, short_only=True)
+            n = K.delta_chunks_scratch_bytes(T, ctx.n_rows, H, d)
+            K.delta_chunks(*step, ctx.max_q_len, ws.get("delta_chunks", (n,), torch.uint8))
+        else:
+            scratch = ws.get("delta_blocks", (K.delta_scan_scratch_floats(T, ctx.n_rows, H, d),), f32) if long else None
+            K.delta_scan(*step, ctx.max_q_len, scratch)
         K.head_norm_gate(o, act, act_col, H, dv, self.eps, self.norm_w, None, 0, scale, sigmoid_gate=gate_z)
         return act
 
