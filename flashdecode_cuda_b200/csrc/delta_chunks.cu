@@ -6,8 +6,10 @@
 //     U = (T diag(beta)) (V - K~ S),      O = Q~ S + P U,      S <- exp(L_end) S + sum_j (exp(L_end - L_j) k_j) u_j^T.
 //  * delta_chunk_prepare: everything of a chunk that does not depend on the state - k~, q~, the tail-decayed keys, T diag(beta), P -
 //    for all chunks side by side.  Exponents are sums of log decays of later tokens, at most 0: nothing is divided.
-//  * delta_chunk_scan: the chunks in order.  A warp takes 16 value columns and holds S^T [16, d] as float accumulators, which
-//    are at the same time, rounded, the first operand of its own products: no state goes through memory between chunks.
+//  * delta_chunk_scan: the chunks in order.  A CTA takes 16 value columns, each of its warps 32 key channels: S^T [16, 32] as float
+//    accumulators, which are at the same time, rounded, the first operand of the warp's products, so that no state goes
+//    through memory between chunks.  The warps add up their shares of K~ S and Q~ S in shared memory, in a fixed order; that is
+//    the one barrier of a chunk.
 // State, decays, exponentials, sums and the inverse are float.  What enters a product goes in as two bfloat16 numbers, the rounded
 // one and what the rounding took away (three products: 16 bits of mantissa on both sides).
 #include <math.h>
@@ -17,8 +19,8 @@
 namespace fd {
 
 constexpr int DC_TOK = 16;
-constexpr int DC_WARPS = 2;                    // of the scan: 16 value columns each
-constexpr int DC_STAGES = 3;
+constexpr int DC_STAGES = 4;                   // chunks of the scan in flight or in use
+constexpr int DC_VLD = 20;                     // floats of a token's 16 values in shared memory
 
 struct DeltaChunks {
     const float* q; const float* k; const float* v; const float* lg; const float* beta;   // as delta_prepare leaves them
@@ -29,6 +31,8 @@ struct DeltaChunks {
 };
 // Bytes of a chunk: k~, q~, tail keys [16][DK] bfloat16, rounded and rest each; T diag(beta) and P [16][16] likewise; the whole decay [DK] float
 template <int DK> __host__ __device__ constexpr int dc_bytes() { return 6 * DC_TOK * DK * 2 + 4 * DC_TOK * DC_TOK * 2 + DK * 4; }
+// ... and of its place in the scan's shared memory: with the values of the CTA's 16 columns
+template <int DK> __host__ __device__ constexpr int dc_stage() { return dc_bytes<DK>() + DC_TOK * DC_VLD * 4; }
 __device__ __forceinline__ int dc_slot(int q_start, int r, int c) { return q_start / DC_TOK + r + c; }
 
 template <int DK>
@@ -142,26 +146,28 @@ __device__ __forceinline__ void as_operand(const float x[4], const float y[4], u
 }
 
 template <int DK>
-__global__ void __launch_bounds__(DC_WARPS * 32)
+__global__ void __launch_bounds__(DK)
 delta_chunk_scan_kernel(const DeltaChunks p) {
+    constexpr int WARPS = DK / 32, THREADS = DK;
     constexpr int CPR = DK / 8, ARR = DC_TOK * DK * 2, MATS = 6 * ARR, TAIL = 4 * DC_TOK * DC_TOK * 2 + DK * 4, BYTES = dc_bytes<DK>();
-    constexpr int THREADS = DC_WARPS * 32;
+    constexpr int STAGE = dc_stage<DK>();
     extern __shared__ __align__(128) unsigned char sm[];
-    const int tiles = (p.dv + DC_WARPS * 16 - 1) / (DC_WARPS * 16);
+    float4* red = reinterpret_cast<float4*>(sm + DC_STAGES * STAGE);       // [2][warp][X or Y][token tile][lane]
+    const int tiles = (p.dv + 15) / 16;
     const int r = blockIdx.x / tiles, tile = blockIdx.x - r * tiles, h = blockIdx.y;
     const int slot = p.row_slot[r], q_start = p.row_q_start[r], q_len = p.row_q_len[r];
     if (slot < 0 || q_len <= p.single) return;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, mi = lane >> 3;
-    const int v_a = (tile * DC_WARPS + warp) * 16 + (lane >> 2), v_b = v_a + 8;       // the thread's two value columns
+    const int v_a = tile * 16 + (lane >> 2), v_b = v_a + 8;                // the thread's two value columns
     const int c2 = (lane & 3) * 2;
     const bool in_a = v_a < p.dv, in_b = v_b < p.dv;
     float* st = p.state + ((size_t)slot * p.H + h) * p.d * p.dv;
-    float S[DK / 8][4];                        // S^T: value columns v_a, v_b by key channels 8 t + c2, + 1
+    float S[4][4];                             // S^T: value columns v_a, v_b by key channels 32 warp + 8 t + c2, + 1
 #pragma unroll
-    for (int t = 0; t < DK / 8; ++t)
+    for (int t = 0; t < 4; ++t)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-            const int ch = t * 8 + c2 + (e & 1);
+            const int ch = warp * 32 + t * 8 + c2 + (e & 1);
             S[t][e] = ch < p.d && ((e >> 1) ? in_b : in_a) ? st[(size_t)ch * p.dv + ((e >> 1) ? v_b : v_a)] : 0.f;
         }
     const int n_chunks = (q_len + DC_TOK - 1) / DC_TOK;
@@ -169,7 +175,7 @@ delta_chunk_scan_kernel(const DeltaChunks p) {
     auto issue = [&](int c) {
         if (c < n_chunks) {
             const unsigned char* src = p.chunks + ((slot0 + c) * p.H + h) * BYTES;
-            unsigned char* dst = sm + (c % DC_STAGES) * BYTES;
+            unsigned char* dst = sm + (c % DC_STAGES) * STAGE;
 #pragma unroll
             for (int e = 0; e < 6 * DC_TOK * CPR / THREADS; ++e) {
                 const int idx = tid + e * THREADS, row = idx / CPR, cc = idx % CPR;     // row: array * 16 + token
@@ -180,55 +186,76 @@ delta_chunk_scan_kernel(const DeltaChunks p) {
                 const int idx = tid + e * THREADS;
                 if (idx < TAIL / 16) cp_async16(smem_u32(dst + MATS + idx * 16), src + MATS + idx * 16, 16);
             }
+            if (tid < 64) {                    // the chunk's values of these columns, rows of DC_VLD floats
+                const int t = tid >> 2, i = (tid & 3) * 4;
+                const bool in = c * DC_TOK + t < q_len && tile * 16 + i < p.dvp;
+                cp_async16(smem_u32(dst + BYTES + (t * DC_VLD + i) * 4),
+                           in ? p.v + ((size_t)(q_start + c * DC_TOK + t) * p.H + h) * p.dvp + tile * 16 + i : p.v, in ? 16 : 0);
+            }
         }
         cp_async_commit();
     };
-    auto value = [&](int c, int e) -> float {  // v of token 8 (e >> 2) + c2 + (e & 1) of chunk c, column v_a or v_b
-        const int t = c * DC_TOK + (e >> 2) * 8 + c2 + (e & 1);
-        const bool b = (e >> 1) & 1;
-        return t < q_len && (b ? in_b : in_a) ? p.v[((size_t)(q_start + t) * p.H + h) * p.dvp + (b ? v_b : v_a)] : 0.f;
-    };
 #pragma unroll
     for (int c = 0; c < DC_STAGES - 1; ++c) issue(c);
-    float v[8];
-#pragma unroll
-    for (int e = 0; e < 8; ++e) v[e] = value(0, e);
+    cp_async_wait<DC_STAGES - 2>();
+    __syncthreads();
     for (int c = 0; c < n_chunks; ++c) {
-        cp_async_wait<DC_STAGES - 2>();
-        __syncthreads();                       // chunk c is there, and everyone is through with chunk c - 1
-        issue(c + DC_STAGES - 1);
-        const uint32_t base = smem_u32(sm + (c % DC_STAGES) * BYTES);
-        float X[3][2][4], Y[3][2][4];
+        const unsigned char* buf = sm + (c % DC_STAGES) * STAGE;
+        const uint32_t base = smem_u32(buf);
+        float4* mine = red + (c & 1) * WARPS * 128;
+        {
+            float X[3][2][4], Y[3][2][4];
 #pragma unroll
-        for (int a = 0; a < 3; ++a)
+            for (int a = 0; a < 3; ++a)
 #pragma unroll
-            for (int t = 0; t < 2; ++t)
+                for (int t = 0; t < 2; ++t)
 #pragma unroll
-                for (int e = 0; e < 4; ++e) X[a][t][e] = Y[a][t][e] = 0.f;
-        // X^T = S^T K~^T and Y^T = S^T Q~^T
+                    for (int e = 0; e < 4; ++e) X[a][t][e] = Y[a][t][e] = 0.f;
+            // the warp's share of X^T = S^T K~^T and Y^T = S^T Q~^T: its 32 key channels
 #pragma unroll
-        for (int kk = 0; kk < DK / 16; ++kk) {
-            uint32_t hi[4], lo[4];
-            as_operand(S[2 * kk], S[2 * kk + 1], hi, lo);
-            const uint32_t at = base + swz<DK>((mi >> 1) * 8 + (lane & 7), kk * 2 + (mi & 1));
-            uint32_t b[4], s[4];
-            ldmatrix_x4(at, b[0], b[1], b[2], b[3]);
-            ldmatrix_x4(at + ARR, s[0], s[1], s[2], s[3]);
-            mma3(X[0][0], X[1][0], X[2][0], hi, lo, b[0], b[1], s[0], s[1]);
-            mma3(X[0][1], X[1][1], X[2][1], hi, lo, b[2], b[3], s[2], s[3]);
-            ldmatrix_x4(at + 2 * ARR, b[0], b[1], b[2], b[3]);
-            ldmatrix_x4(at + 3 * ARR, s[0], s[1], s[2], s[3]);
-            mma3(Y[0][0], Y[1][0], Y[2][0], hi, lo, b[0], b[1], s[0], s[1]);
-            mma3(Y[0][1], Y[1][1], Y[2][1], hi, lo, b[2], b[3], s[2], s[3]);
+            for (int kk = 0; kk < 2; ++kk) {
+                uint32_t hi[4], lo[4], b[4], s[4];
+                as_operand(S[2 * kk], S[2 * kk + 1], hi, lo);
+                const uint32_t at = base + swz<DK>((mi >> 1) * 8 + (lane & 7), (warp * 2 + kk) * 2 + (mi & 1));
+                ldmatrix_x4(at, b[0], b[1], b[2], b[3]);
+                ldmatrix_x4(at + ARR, s[0], s[1], s[2], s[3]);
+                mma3(X[0][0], X[1][0], X[2][0], hi, lo, b[0], b[1], s[0], s[1]);
+                mma3(X[0][1], X[1][1], X[2][1], hi, lo, b[2], b[3], s[2], s[3]);
+                ldmatrix_x4(at + 2 * ARR, b[0], b[1], b[2], b[3]);
+                ldmatrix_x4(at + 3 * ARR, s[0], s[1], s[2], s[3]);
+                mma3(Y[0][0], Y[1][0], Y[2][0], hi, lo, b[0], b[1], s[0], s[1]);
+                mma3(Y[0][1], Y[1][1], Y[2][1], hi, lo, b[2], b[3], s[2], s[3]);
+            }
+#pragma unroll
+            for (int t = 0; t < 2; ++t) {
+                float x[4], y[4];
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    x[e] = X[0][t][e] + (X[1][t][e] + X[2][t][e]);
+                    y[e] = Y[0][t][e] + (Y[1][t][e] + Y[2][t][e]);
+                }
+                mine[(warp * 4 + t) * 32 + lane] = make_float4(x[0], x[1], x[2], x[3]);
+                mine[(warp * 4 + 2 + t) * 32 + lane] = make_float4(y[0], y[1], y[2], y[3]);
+            }
         }
+        // the one meeting of a chunk: the shares are there, the next chunk's data too, and everyone is through with the last one's
+        cp_async_wait<DC_STAGES - 3>();
+        __syncthreads();
+        issue(c + DC_STAGES - 1);
         float D[2][4];
+        const float* v_s = reinterpret_cast<const float*>(buf + BYTES);
 #pragma unroll
-        for (int t = 0; t < 2; ++t)
+        for (int t = 0; t < 2; ++t) {
+            float x[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-            for (int e = 0; e < 4; ++e) D[t][e] = v[t * 4 + e] - (X[0][t][e] + (X[1][t][e] + X[2][t][e]));
+            for (int w = 0; w < WARPS; ++w) {
+                const float4 o = mine[(w * 4 + t) * 32 + lane];
+                x[0] += o.x; x[1] += o.y; x[2] += o.z; x[3] += o.w;
+            }
 #pragma unroll
-        for (int e = 0; e < 8; ++e) v[e] = c + 1 < n_chunks ? value(c + 1, e) : 0.f;
-        // U^T = D^T (T diag(beta))^T, then O^T = Y^T + U^T P^T
+            for (int e = 0; e < 4; ++e) D[t][e] = v_s[(t * 8 + c2 + (e & 1)) * DC_VLD + (lane >> 2) + (e >> 1) * 8] - x[e];
+        }
+        // U^T = D^T (T diag(beta))^T
         uint32_t hi[4], lo[4], b[4], s[4];
         const uint32_t mat = base + MATS + ((mi >> 1) * 8 + (lane & 7)) * 32 + (mi & 1) * 16;
         float U[3][2][4];
@@ -243,50 +270,68 @@ delta_chunk_scan_kernel(const DeltaChunks p) {
         ldmatrix_x4(mat + 512, s[0], s[1], s[2], s[3]);
         mma3(U[0][0], U[1][0], U[2][0], hi, lo, b[0], b[1], s[0], s[1]);
         mma3(U[0][1], U[1][1], U[2][1], hi, lo, b[2], b[3], s[2], s[3]);
+        // the tail-decayed keys and the decay while that is under way
+        uint32_t kb[2][4], ks[2][4];
+#pragma unroll
+        for (int np = 0; np < 2; ++np) {
+            const uint32_t at = base + 4 * ARR + swz<DK>((mi & 1) * 8 + (lane & 7), (warp * 2 + np) * 2 + (mi >> 1));
+            ldmatrix_x4_trans(at, kb[np][0], kb[np][1], kb[np][2], kb[np][3]);
+            ldmatrix_x4_trans(at + ARR, ks[np][0], ks[np][1], ks[np][2], ks[np][3]);
+        }
+        const unsigned char* whole = buf + MATS + 4 * DC_TOK * DC_TOK * 2;
+#pragma unroll
+        for (int t = 0; t < 4; ++t) {
+            const float2 w = *reinterpret_cast<const float2*>(whole + (warp * 32 + t * 8 + c2) * 4);
+            S[t][0] *= w.x; S[t][1] *= w.y; S[t][2] *= w.x; S[t][3] *= w.y;
+        }
 #pragma unroll
         for (int t = 0; t < 2; ++t)
 #pragma unroll
             for (int e = 0; e < 4; ++e) U[0][t][e] += U[1][t][e] + U[2][t][e];
         as_operand(U[0][0], U[0][1], hi, lo);
         // S^T <- S^T exp(L_end) + U^T K_tail
-        const unsigned char* whole = sm + (c % DC_STAGES) * BYTES + MATS + 4 * DC_TOK * DC_TOK * 2;
 #pragma unroll
-        for (int t = 0; t < DK / 8; ++t) {
-            const float2 w = *reinterpret_cast<const float2*>(whole + (t * 8 + c2) * 4);
-            S[t][0] *= w.x; S[t][1] *= w.y; S[t][2] *= w.x; S[t][3] *= w.y;
+        for (int np = 0; np < 2; ++np) {
+            mma_bf16(S[2 * np], hi[0], hi[1], hi[2], hi[3], kb[np][0], kb[np][1]);
+            mma_bf16(S[2 * np + 1], hi[0], hi[1], hi[2], hi[3], kb[np][2], kb[np][3]);
         }
 #pragma unroll
-        for (int np = 0; np < DK / 16; ++np) {
-            const uint32_t at = base + 4 * ARR + swz<DK>((mi & 1) * 8 + (lane & 7), np * 2 + (mi >> 1));
-            uint32_t kb[4], ks[4];
-            ldmatrix_x4_trans(at, kb[0], kb[1], kb[2], kb[3]);
-            ldmatrix_x4_trans(at + ARR, ks[0], ks[1], ks[2], ks[3]);
-            mma_bf16(S[2 * np], hi[0], hi[1], hi[2], hi[3], kb[0], kb[1]);
-            mma_bf16(S[2 * np + 1], hi[0], hi[1], hi[2], hi[3], kb[2], kb[3]);
-            mma_bf16(S[2 * np], hi[0], hi[1], hi[2], hi[3], ks[0], ks[1]);
-            mma_bf16(S[2 * np + 1], hi[0], hi[1], hi[2], hi[3], ks[2], ks[3]);
-            mma_bf16(S[2 * np], lo[0], lo[1], lo[2], lo[3], kb[0], kb[1]);
-            mma_bf16(S[2 * np + 1], lo[0], lo[1], lo[2], lo[3], kb[2], kb[3]);
+        for (int np = 0; np < 2; ++np) {
+            mma_bf16(S[2 * np], hi[0], hi[1], hi[2], hi[3], ks[np][0], ks[np][1]);
+            mma_bf16(S[2 * np + 1], hi[0], hi[1], hi[2], hi[3], ks[np][2], ks[np][3]);
         }
-        ldmatrix_x4(mat + 1024, b[0], b[1], b[2], b[3]);
-        ldmatrix_x4(mat + 1536, s[0], s[1], s[2], s[3]);
-        mma3(Y[0][0], Y[1][0], Y[2][0], hi, lo, b[0], b[1], s[0], s[1]);
-        mma3(Y[0][1], Y[1][1], Y[2][1], hi, lo, b[2], b[3], s[2], s[3]);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) {
-            const int t = c * DC_TOK + (e >> 2) * 8 + c2 + (e & 1);
-            const bool bb = (e >> 1) & 1;
-            if (t < q_len && (bb ? in_b : in_a))
-                p.out[((size_t)(q_start + t) * p.H + h) * p.dv + (bb ? v_b : v_a)] = Y[0][e >> 2][e & 3] + (Y[1][e >> 2][e & 3] + Y[2][e >> 2][e & 3]);
+        for (int np = 0; np < 2; ++np) {
+            mma_bf16(S[2 * np], lo[0], lo[1], lo[2], lo[3], kb[np][0], kb[np][1]);
+            mma_bf16(S[2 * np + 1], lo[0], lo[1], lo[2], lo[3], kb[np][2], kb[np][3]);
+        }
+        // O^T = Y^T + U^T P^T: the first two warps, eight tokens each
+        if (warp < 2) {
+            float o[3][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+#pragma unroll
+            for (int w = 0; w < WARPS; ++w) {
+                const float4 y = mine[(w * 4 + 2 + warp) * 32 + lane];
+                o[0][0] += y.x; o[0][1] += y.y; o[0][2] += y.z; o[0][3] += y.w;
+            }
+            ldmatrix_x4(mat + 1024, b[0], b[1], b[2], b[3]);
+            ldmatrix_x4(mat + 1536, s[0], s[1], s[2], s[3]);
+            if (warp == 0) mma3(o[0], o[1], o[2], hi, lo, b[0], b[1], s[0], s[1]);
+            else mma3(o[0], o[1], o[2], hi, lo, b[2], b[3], s[2], s[3]);
+            const int t = c * DC_TOK + warp * 8 + c2;
+            float* out = p.out + ((size_t)(q_start + t) * p.H + h) * p.dv;
+            const size_t next = (size_t)p.H * p.dv;
+#pragma unroll
+            for (int e = 0; e < 4; ++e)
+                if (t + (e & 1) < q_len && ((e >> 1) ? in_b : in_a)) out[(e & 1) * next + ((e >> 1) ? v_b : v_a)] = o[0][e] + (o[1][e] + o[2][e]);
         }
     }
     cp_async_wait<0>();
     if (p.write_state) {
 #pragma unroll
-        for (int t = 0; t < DK / 8; ++t)
+        for (int t = 0; t < 4; ++t)
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
-                const int ch = t * 8 + c2 + (e & 1);
+                const int ch = warp * 32 + t * 8 + c2 + (e & 1);
                 if (ch < p.d && ((e >> 1) ? in_b : in_a)) st[(size_t)ch * p.dv + ((e >> 1) ? v_b : v_a)] = S[t][e];
             }
     }
@@ -294,7 +339,7 @@ delta_chunk_scan_kernel(const DeltaChunks p) {
 
 template <int DK>
 static int launch_delta_chunks(const DeltaChunks& p, int n_rows, cudaStream_t stream) {
-    constexpr int smem = DC_STAGES * dc_bytes<DK>();
+    constexpr int smem = DC_STAGES * dc_stage<DK>() + 2 * (DK / 32) * 128 * 16;
     auto k = delta_chunk_scan_kernel<DK>;
     static bool configured = false;
     if (!configured) {
@@ -305,8 +350,7 @@ static int launch_delta_chunks(const DeltaChunks& p, int n_rows, cudaStream_t st
     const dim3 one(1, 1, 1);
     int rc = launch("delta_chunk_prepare", delta_chunk_prepare_kernel<DK>, dim3((unsigned)n_rows * p.max_chunks, p.H), dim3(256), 0, stream, one, p);
     if (rc) return rc;
-    const int tiles = (p.dv + DC_WARPS * 16 - 1) / (DC_WARPS * 16);
-    return launch("delta_chunk_scan", k, dim3((unsigned)tiles * n_rows, p.H), dim3(DC_WARPS * 32), smem, stream, one, p);
+    return launch("delta_chunk_scan", k, dim3((unsigned)((p.dv + 15) / 16) * n_rows, p.H), dim3(DK), smem, stream, one, p);
 }
 
 }  // namespace fd
