@@ -103,14 +103,15 @@ delta_prepare_kernel(const DeltaParams p) {
     const int nqk = p.Hk * p.d, C = 2 * nqk + p.H * p.dv;
     conv_meta(meta, t0, nt, p.tok_row, p.tok_pos, p.row_slot, p.row_q_start, p.row_q_len);
     if (u < 2 * p.Hk) {                                     // a head of q or k
-        __syncthreads();
         const bool is_q = u < p.Hk;
         const int h = is_q ? u : u - p.Hk;
         const bool active = tid < p.d;
         const int c = (is_q ? 0 : nqk) + h * p.d + (active ? tid : 0);
-        float y[SC_TOK];
-        conv_channel<T>(proj + (is_q ? p.q_col : p.k_col) + h * p.d + (active ? tid : 0), p.ld, p.conv_w + (size_t)c * p.taps, 0.f, p.taps,
-                        p.ring, c, C, meta, t0, nt, p.keep && active, y);
+        const T* col = proj + (is_q ? p.q_col : p.k_col) + h * p.d + (active ? tid : 0);
+        float x[SC_VALS], y[SC_TOK];
+        if (p.tpc > 1) conv_load<T>(col, p.ld, t0, nt, x);
+        __syncthreads();
+        conv_channel<T>(col, p.ld, p.conv_w + (size_t)c * p.taps, 0.f, p.taps, p.ring, c, C, meta, t0, nt, p.keep && active, x, y);
 #pragma unroll
         for (int tt = 0; tt < SC_TOK; ++tt) {
             if (tt >= nt) continue;
@@ -139,9 +140,10 @@ delta_prepare_kernel(const DeltaParams p) {
         for (int j = tid; j < p.dvp; j += blockDim.x) {
             const bool active = j < p.dv;
             const int c = 2 * nqk + u * p.dv + (active ? j : 0);
-            float y[SC_TOK];
-            conv_channel<T>(proj + p.v_col + u * p.dv + (active ? j : 0), p.ld, p.conv_w + (size_t)c * p.taps, 0.f, p.taps, p.ring, c, C,
-                            meta, t0, nt, p.keep && active, y);
+            const T* col = proj + p.v_col + u * p.dv + (active ? j : 0);
+            float x[SC_VALS], y[SC_TOK];
+            if (p.tpc > 1) conv_load<T>(col, p.ld, t0, nt, x);
+            conv_channel<T>(col, p.ld, p.conv_w + (size_t)c * p.taps, 0.f, p.taps, p.ring, c, C, meta, t0, nt, p.keep && active, x, y);
 #pragma unroll
             for (int tt = 0; tt < SC_TOK; ++tt)
                 if (tt < nt && meta.slot[tt] >= 0)

@@ -69,6 +69,10 @@ struct GsParams {
     int n_tiles;           // tiles of 128 rows of W
     unsigned long long wait_ns;
     int skip_last;         // tests only: the producer leaves out its very last copy
+    // mode 1: rows of W from tail_from (a multiple of 16) on are a feed-forward's that reads the same x: max(., 0)^2 of their
+    // outputs goes to tail_out, rows of tail_ld elements, instead of out (null: there are none)
+    __nv_bfloat16* tail_out;
+    int tail_from, tail_ld;
 };
 
 // Named barrier 1 of the 128 epilogue threads, plain and with an AND over a flag of every thread.
@@ -171,6 +175,14 @@ __device__ __forceinline__ void gs_finish(const GsParams& p, const TcRope& ra, c
             if (vec_ok) {
                 add_bias16(p, n_tile, v);
                 if (p.mode == 1) {
+                    if (p.tail_out != nullptr && n_tile >= p.tail_from) {
+#pragma unroll
+                        for (int j = 0; j < 16; ++j) { const float a = fmaxf(v[j], 0.f); v[j] = a * a; }
+                        uint4* o = reinterpret_cast<uint4*>(p.tail_out + (size_t)m * p.tail_ld + (n_tile - p.tail_from));
+                        o[0] = make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7]));
+                        o[1] = make_uint4(pack_bf16(v[8], v[9]), pack_bf16(v[10], v[11]), pack_bf16(v[12], v[13]), pack_bf16(v[14], v[15]));
+                        continue;
+                    }
                     uint4* o = reinterpret_cast<uint4*>(static_cast<__nv_bfloat16*>(p.out) + (size_t)m * p.N + n_tile);
                     o[0] = make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7]));
                     o[1] = make_uint4(pack_bf16(v[8], v[9]), pack_bf16(v[10], v[11]), pack_bf16(v[12], v[13]), pack_bf16(v[14], v[15]));
@@ -621,10 +633,15 @@ extern "C" int fd_gemm_stream_splits(int M, int N, int K) {
 }
 
 // mode 1: out bf16 [M, N] (+ bias); 2: out float [M, N] (+ bias); 3: W rows in tiles of 8 gate + 8 up
-// rows, out bf16 [M, N / 2] = silu(gate) * up (N a multiple of 16).  splits 0: chosen by the launcher.
+// rows, out bf16 [M, N / 2] = silu(gate) * up (N a multiple of 16).  splits 0: chosen by the launcher.  tail_out (optional, mode
+// 1): the outputs of the rows of W from tail_from on go there, in rows of tail_ld elements, as max(., 0)^2.
 extern "C" int fd_gemm_stream(const void* x, const void* w, const void* bias, int bias_f32, void* out, int mode,
-                              int M, int N, int K, int splits, int* status, cudaStream_t stream) {
+                              int M, int N, int K, int splits, int* status, void* tail_out, int tail_from, int tail_ld,
+                              cudaStream_t stream) {
     if (M == 0 || N == 0) return 0;
+    FD_REQUIRE(tail_out == nullptr || (mode == 1 && tail_from >= 0 && tail_from % 16 == 0 && N % 16 == 0 && tail_ld % 8 == 0 &&
+               tail_ld >= N - tail_from && (uintptr_t)tail_out % 16 == 0), -2,
+               "gemm_stream: a feed-forward's rows from %d of %d on to rows of %d (multiples of 16, 16 and 8)", tail_from, N, tail_ld);
     int act = 0;
     if (mode == 6) { mode = 3; act = 1; }           // gated with the tanh form of GELU
     FD_REQUIRE(mode >= 1 && mode <= 3, -2, "gemm_stream: mode %d", mode);
@@ -634,6 +651,7 @@ extern "C" int fd_gemm_stream(const void* x, const void* w, const void* bias, in
     GsParams p = {};
     p.bias = bias; p.out = out; p.status = status; p.M = M; p.N = N; p.K = K; p.mode = mode; p.bias_f32 = bias_f32;
     p.act = act;
+    p.tail_out = (__nv_bfloat16*)tail_out; p.tail_from = tail_from; p.tail_ld = tail_ld;
     TcRope ra = {};
     return launch_gs(x, w, p, ra, splits, stream, "gemm_stream");
 }

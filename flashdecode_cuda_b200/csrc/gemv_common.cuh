@@ -41,6 +41,10 @@ struct GemvParams {
     // 27.5 MB of the down projection from the gate/up kernel made the step 1.2 % slower.
     const unsigned char* pf_ptr;
     unsigned long long pf_bytes;
+    // mode 1: rows of W from tail_from on are a feed-forward's that reads the same x: max(., 0)^2 of their outputs goes to
+    // tail_out [M] rows of tail_ld elements instead of out (tail_from >= N: there are none)
+    __nv_bfloat16* tail_out;
+    int tail_from, tail_ld;
 };
 
 // Mode 4.  W rows are the q heads, then the k heads, then the v heads.  Inside a
@@ -201,7 +205,10 @@ __device__ __forceinline__ void gemv_epilogue(const GemvParams& p, const RopeArg
                 const float v = acc[nt][h * 2 + e] + bias;
                 if (p.mode == 0)
                     static_cast<float*>(p.out)[((size_t)split * p.M + m) * p.N + n] = v;
-                else if (p.mode == 1)
+                else if (p.mode == 1 && n >= p.tail_from) {
+                    const float a = fmaxf(v, 0.f);
+                    p.tail_out[(size_t)m * p.tail_ld + (n - p.tail_from)] = __float2bfloat16_rn(a * a);
+                } else if (p.mode == 1)
                     static_cast<__nv_bfloat16*>(p.out)[(size_t)m * p.N + n] = __float2bfloat16_rn(v);
                 else
                     static_cast<float*>(p.out)[(size_t)m * p.N + n] = v;

@@ -279,11 +279,14 @@ extern "C" int fd_gemv_splits(int M, int N, int K, int target_ctas, int allow_sp
 // mode 0: out = float partial sums [n_splits, M, N]; 1: bf16 [M, N]; 2: float [M, N] (both with
 // up to 8 splits added inside a cluster); 3: gated (rows of W in tiles of 8 gate + 8 up):
 // bf16 [M, N / 2], n_splits == 1.  prefetch / prefetch_bytes (optional, 16-byte aligned): memory that a
-// later kernel streams, which this kernel asks L2 for once its own loads are through.
+// later kernel streams, which this kernel asks L2 for once its own loads are through.  tail_out (optional, mode 1): the outputs
+// of the rows of W from tail_from on go there, in rows of tail_ld elements, as max(., 0)^2.
 extern "C" int fd_gemv(const void* x, const void* w, const void* bias, int bias_f32, void* out, int mode,
                        int M, int N, int K, int n_splits, const void* prefetch, unsigned long long prefetch_bytes,
-                       cudaStream_t stream) {
+                       void* tail_out, int tail_from, int tail_ld, cudaStream_t stream) {
     if (M == 0 || N == 0) return 0;
+    FD_REQUIRE(tail_out == nullptr || (mode == 1 && tail_from >= 0 && tail_ld >= N - tail_from), -2,
+               "gemv: a feed-forward's rows from %d of %d on to rows of %d", tail_from, N, tail_ld);
     FD_REQUIRE((uintptr_t)prefetch % 16 == 0, -2, "gemv: the memory to prefetch must be 16-byte aligned");
     FD_REQUIRE(M >= 1 && M <= 64, -2, "gemv: %d rows of x; this kernel takes 1..64", M);
     FD_REQUIRE(K >= 32 && K % 32 == 0, -2, "gemv: K=%d must be a positive multiple of 32", K);
@@ -297,6 +300,7 @@ extern "C" int fd_gemv(const void* x, const void* w, const void* bias, int bias_
     GemvParams p;
     p.x = (const __nv_bfloat16*)x; p.w = (const __nv_bfloat16*)w; p.bias = bias; p.out = out;
     p.M = M; p.N = N; p.K = K; p.n_splits = n_splits; p.mode = mode; p.bias_f32 = bias_f32; p.act = act;
+    p.tail_out = (__nv_bfloat16*)tail_out; p.tail_from = tail_out ? tail_from : 0x7fffffff; p.tail_ld = tail_ld;
     p.pf_ptr = (const unsigned char*)prefetch; p.pf_bytes = prefetch ? prefetch_bytes : 0;
     RopeArgs ra = {};
     return run_gemv(p, ra, stream);
@@ -324,6 +328,7 @@ extern "C" int fd_gemv_qkv_rope(const void* x, const void* w, const void* bias, 
     GemvParams p;
     p.x = (const __nv_bfloat16*)x; p.w = (const __nv_bfloat16*)w; p.bias = bias; p.out = q_out;
     p.M = M; p.N = (n_q + 2 * n_kv) * d; p.K = K; p.n_splits = n_splits; p.mode = 4; p.bias_f32 = bias_f32; p.act = 0;
+    p.tail_out = nullptr; p.tail_from = 0x7fffffff; p.tail_ld = 0;
     p.pf_ptr = (const unsigned char*)prefetch; p.pf_bytes = prefetch ? prefetch_bytes : 0;
     RopeArgs ra;
     ra.cos_t = cos_t; ra.sin_t = sin_t; ra.tok_row = tok_row; ra.tok_pos = tok_pos; ra.row_slot = row_slot;

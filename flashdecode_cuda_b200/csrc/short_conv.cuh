@@ -17,7 +17,7 @@ constexpr int SC_TAPS = 4;            // more taps than this take the plain loop
 
 struct ConvMeta {                     // what the tokens of a tile need to know, in shared memory
     int slot[SC_TOK], i[SC_TOK], pos[SC_TOK], single[SC_TOK];     // slot -1: padding row; i: place in its row's new tokens
-    int one_row;                      // the tile's tokens all belong to one row (and none is padding)
+    int one_row;                      // the tile has several tokens, all of one row (and none is padding)
 };
 
 // threads 0 .. nt - 1 fill the tile's entries; the caller synchronises
@@ -29,31 +29,43 @@ __device__ __forceinline__ void conv_meta(ConvMeta& m, int t0, int nt, const int
         m.i[threadIdx.x] = t - row_q_start[r];
         m.pos[threadIdx.x] = tok_pos[t];
         m.single[threadIdx.x] = row_q_len[r] == 1;
-        if (threadIdx.x == 0) m.one_row = m.slot[0] >= 0 && tok_row[t0 + nt - 1] == r;
+        if (threadIdx.x == 0) m.one_row = nt > 1 && m.slot[0] >= 0 && tok_row[t0 + nt - 1] == r;
     }
 }
 
-// The nt <= SC_TOK tokens from t0 on of channel c of C (column `col` points at it in token 0's row, rows of ld elements);
+constexpr int SC_VALS = SC_TOK + SC_TAPS - 1;      // values the taps of a tile's tokens see; place SC_TAPS - 1 + j is token t0 + j
+
+// The values of a tile as they lie in the step's rows, before anything is known of its tokens: so the loads pass beside those of the
+// tile's ConvMeta.  Those before the row's first token are wrong yet; conv_channel puts the ring's in their place.
+template <typename T>
+__device__ __forceinline__ void conv_load(const T* __restrict__ col, int ld, int t0, int nt, float u[SC_VALS]) {
+#pragma unroll
+    for (int e = 0; e < SC_VALS; ++e) {
+        const int j = e - (SC_TAPS - 1);
+        u[e] = j < nt && t0 + j >= 0 ? to_float(col[(size_t)(t0 + j) * ld]) : 0.f;
+    }
+}
+
+// The nt <= SC_TOK tokens from t0 on of channel c of C (column `col` points at it in token 0's row, rows of ld elements; u: what
+// conv_load made of it, looked at only in tiles of one row);
 // rows that bring a single token leave their value in the ring when `keep` is set.
 template <typename T>
 __device__ __forceinline__ void conv_channel(const T* __restrict__ col, int ld, const float* __restrict__ w, float bias, int taps,
                                              float* ring, int c, int C, const ConvMeta& m, int t0, int nt, bool keep,
-                                             float y[SC_TOK]) {
+                                             float u[SC_VALS], float y[SC_TOK]) {
     float wk[SC_TAPS];
 #pragma unroll
     for (int k = 0; k < SC_TAPS; ++k) wk[k] = k < taps ? w[k] : 0.f;
     if (m.one_row && !m.single[0] && taps <= SC_TAPS) {
-        // consecutive tokens of one row: every value once, all loads under way together; place SC_TAPS - 1 + j is token t0 + j
-        float u[SC_TOK + SC_TAPS - 1];
+        // consecutive tokens of one row
         const int i0 = m.i[0], pos0 = m.pos[0];
         const float* rg = ring + (size_t)m.slot[0] * taps * C + c;
+        if (i0 < taps - 1) {
 #pragma unroll
-        for (int e = 0; e < SC_TOK + SC_TAPS - 1; ++e) {
-            const int j = e - (SC_TAPS - 1);
-            u[e] = 0.f;
-            if (j >= nt || -j >= taps) continue;
-            if (i0 + j >= 0) u[e] = to_float(col[(size_t)(t0 + j) * ld]);
-            else if (pos0 + j >= 0) u[e] = rg[(size_t)((pos0 + j) % taps) * C];
+            for (int e = 0; e < SC_TAPS - 1; ++e) {
+                const int j = e - (SC_TAPS - 1);
+                if (i0 + j < 0) u[e] = -j < taps && pos0 + j >= 0 ? rg[(size_t)((pos0 + j) % taps) * C] : 0.f;
+            }
         }
         // the weights moved to the end, so that tap k of `taps` meets the place it would meet below
         float we[SC_TAPS];
@@ -85,11 +97,11 @@ __device__ __forceinline__ void conv_channel(const T* __restrict__ col, int ld, 
         float a = bias;
         const float cur = value(0);
         if (taps <= SC_TAPS) {
-            float u[SC_TAPS];
+            float x[SC_TAPS];
 #pragma unroll
-            for (int k = 0; k < SC_TAPS; ++k) u[k] = k < taps - 1 ? value(taps - 1 - k) : (k == taps - 1 ? cur : 0.f);
+            for (int k = 0; k < SC_TAPS; ++k) x[k] = k < taps - 1 ? value(taps - 1 - k) : (k == taps - 1 ? cur : 0.f);
 #pragma unroll
-            for (int k = 0; k < SC_TAPS; ++k) if (k < taps) a = fmaf(wk[k], u[k], a);
+            for (int k = 0; k < SC_TAPS; ++k) if (k < taps) a = fmaf(wk[k], x[k], a);
         } else {
             for (int k = 0; k < taps; ++k) a = fmaf(w[k], value(taps - 1 - k), a);
         }

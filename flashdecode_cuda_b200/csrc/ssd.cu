@@ -38,6 +38,9 @@ ssd_prepare_kernel(const T* __restrict__ proj, int ld, int col, int C, int dt_co
     __shared__ ConvMeta meta;
     const int t0 = blockIdx.x * tpc, nt = min(tpc, n_tok - t0);
     conv_meta(meta, t0, nt, tok_row, tok_pos, row_slot, row_q_start, row_q_len);
+    const int c = blockIdx.y * SSD_THREADS + threadIdx.x;
+    float u[SC_VALS];
+    if (tpc > 1 && c < C) conv_load<T>(proj + col + c, ld, t0, nt, u);
     __syncthreads();
     if (blockIdx.y == gridDim.y - 1) {                       // step sizes and decays
         for (int e = threadIdx.x; e < nt * H; e += blockDim.x) {
@@ -47,10 +50,9 @@ ssd_prepare_kernel(const T* __restrict__ proj, int ld, int col, int C, int dt_co
         }
         return;
     }
-    const int c = blockIdx.y * SSD_THREADS + threadIdx.x;
     if (c >= C) return;
     float y[SC_TOK];
-    conv_channel<T>(proj + col + c, ld, conv_w + (size_t)c * taps, conv_b[c], taps, ring, c, C, meta, t0, nt, keep, y);
+    conv_channel<T>(proj + col + c, ld, conv_w + (size_t)c * taps, conv_b[c], taps, ring, c, C, meta, t0, nt, keep, u, y);
 #pragma unroll
     for (int tt = 0; tt < SC_TOK; ++tt)
         if (tt < nt && meta.slot[tt] >= 0) {

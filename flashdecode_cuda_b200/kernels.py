@@ -85,11 +85,11 @@ def _declare(L: ctypes.CDLL) -> None:
         "fd_gemm_stream_force_2d": [I],
         "fd_gemm_stream_set_pdl": [I],
         "fd_gemm_stream_last_map3d": [],
-        "fd_gemm_stream": [P, P, P, I, P, I, I, I, I, I, P, P],
+        "fd_gemm_stream": [P, P, P, I, P, I, I, I, I, I, P, P, I, I, P],
         "fd_gemm_stream_qkv_rope": [P, P, P, I, P, I, I, I, P, P, I, P, P, P, P, P, P, I, I, I, I, I, I, I, P, P],
         "fd_tc_test_hook": [LL, I],
         "fd_gemv_splits": [I, I, I, I, I],
-        "fd_gemv": [P, P, P, I, P, I, I, I, I, I, P, c_ulonglong, P],
+        "fd_gemv": [P, P, P, I, P, I, I, I, I, I, P, c_ulonglong, P, I, I, P],
         "fd_gemm_simt": [P, P, P, P, I, I, I, I, I, I, P],
         "fd_attn_simt_qt": [I],
         "fd_attn_decode_group": [I, I, I],
@@ -615,11 +615,12 @@ def gemm_stream_splits(M: int, N: int, K: int) -> int:
 
 
 def gemm_stream(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out: torch.Tensor, gated: bool = False,
-                splits: int = 0, status: Optional[torch.Tensor] = None) -> None:
+                splits: int = 0, status: Optional[torch.Tensor] = None, tail=None) -> None:
     """Weight-streaming product for up to 128 rows of x on the tcgen05 tensor cores (W tiles as the
     M side, the rows of x as the N side, K split over a thread-block cluster for narrow W):
     out = x w^T (+ bias), bfloat16 or float32 [M, N], or with ``gated`` (w rows in tiles of 8 gate +
-    8 up) bfloat16 [M, N / 2] = silu(gate) * up.  ``splits`` 0: chosen by the launcher."""
+    8 up) bfloat16 [M, N / 2] = silu(gate) * up.  ``splits`` 0: chosen by the launcher.  ``tail`` (row, out2, col): as for ``gemv``;
+    row, N, col and out2's columns multiples of 16."""
     M, K = x.shape
     N = w.shape[0]
     assert x.dtype == w.dtype == torch.bfloat16 and w.shape[1] == K
@@ -630,7 +631,7 @@ def gemm_stream(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], 
         assert out.shape == (M, N) and out.dtype in (torch.bfloat16, torch.float32)
         mode = GEMV_BF16 if out.dtype == torch.bfloat16 else GEMV_F32
     _check(lib().fd_gemm_stream(_ptr(x), _ptr(w), _ptr(bias), int(bias is not None and bias.dtype == torch.float32),
-                                _ptr(out), mode, M, N, K, splits, _ptr(status), _stream()))
+                                _ptr(out), mode, M, N, K, splits, _ptr(status), *_tail_args(tail, M, N, mode), _stream()))
 
 
 def gemm_stream_qkv_rope(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], q_out: torch.Tensor,
@@ -690,14 +691,25 @@ def _prefetch_args(t: Optional[torch.Tensor], limit: int):
     return t.data_ptr(), min(int(limit), t.numel() * t.element_size()) & ~15
 
 
+def _tail_args(tail, M: int, N: int, mode: int):
+    if tail is None:
+        return None, 0, 0
+    row, out2, col = tail
+    assert mode == GEMV_BF16 and out2.dtype == torch.bfloat16 and out2.shape[0] == M and 0 <= row < N
+    assert col + N - row <= out2.shape[1]
+    return _col_ptr(out2, col), row, out2.shape[1]
+
+
 def gemv(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out: torch.Tensor, mode: int,
-         n_splits: int = 1, prefetch: Optional[torch.Tensor] = None, prefetch_bytes: int = 1 << 62) -> None:
+         n_splits: int = 1, prefetch: Optional[torch.Tensor] = None, prefetch_bytes: int = 1 << 62, tail=None) -> None:
     """Weight-streaming product for M <= 64 rows (bfloat16): out = x w^T.
     mode GEMV_PARTIAL: out float32 [n_splits, M, N]; GEMV_BF16 / GEMV_F32: out
     [M, N] (+ bias), with ``n_splits`` <= 8 splits of K added inside a
     thread-block cluster; GEMV_GATED: w rows in tiles of 8 gate + 8 up, out
     bfloat16 [M, N / 2] = silu(gate) * up.  ``prefetch``: a tensor that a later kernel
-    streams; the kernel asks L2 for its first ``prefetch_bytes`` once its own loads are through."""
+    streams; the kernel asks L2 for its first ``prefetch_bytes`` once its own loads are through.  ``tail`` (GEMV_BF16)
+    (row, out2, col): the outputs of w's rows from ``row`` on are a feed-forward's; max(., 0)^2 of them goes to the columns of
+    ``out2`` [M, *] from ``col`` on instead of to ``out``."""
     M, K = x.shape
     N = w.shape[0]
     assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and w.shape[1] == K
@@ -706,7 +718,8 @@ def gemv(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out: to
             GEMV_GATED_GELU: (torch.bfloat16, M * N // 2)}[mode]
     assert out.dtype == want[0] and out.numel() == want[1], (out.dtype, out.shape, mode)
     _check(lib().fd_gemv(_ptr(x), _ptr(w), _ptr(bias), int(bias is not None and bias.dtype == torch.float32),
-                         _ptr(out), mode, M, N, K, n_splits, *_prefetch_args(prefetch, prefetch_bytes), _stream()))
+                         _ptr(out), mode, M, N, K, n_splits, *_prefetch_args(prefetch, prefetch_bytes),
+                         *_tail_args(tail, M, N, mode), _stream()))
 
 
 def gemm_simt(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out: torch.Tensor) -> None:

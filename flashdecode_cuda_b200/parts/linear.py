@@ -54,9 +54,18 @@ def fused_prompt_gemm(M: int, N: int, Kd: int) -> bool:
     return PROMPT_GEMM == "tcgen05" or M >= 128
 
 
+def takes_tail(M: int, N: int, Kd: int, dtype: torch.dtype, row: int, out2_cols: int, col: int) -> bool:
+    """Whether ``matmul`` of M rows can finish the outputs from ``row`` on as a feed-forward's (``tail``)."""
+    if dtype != torch.bfloat16:
+        return False
+    if M <= GEMV_MAX_ROWS and K.gemv_splits(M, N, Kd, 0, allow_split=False) >= 1:
+        return True
+    return stream_gemm(M, N, Kd) and row % 16 == 0 and N % 16 == 0 and out2_cols % 8 == 0 and col % 8 == 0
+
+
 def matmul(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out: torch.Tensor,
            target_ctas: int = 0, parts: Optional[torch.Tensor] = None,
-           status: Optional[torch.Tensor] = None, upcoming: Optional[torch.Tensor] = None) -> torch.Tensor:
+           status: Optional[torch.Tensor] = None, upcoming: Optional[torch.Tensor] = None, tail=None) -> torch.Tensor:
     """x [M, K], w [N, K], bias [N] or None, out [M, N] (dtype of x, or
     float32 for logits).  ``target_ctas``: how many CTAs a decode product
     should spread over (it splits K to get there).  ``parts``: float32 memory
@@ -65,7 +74,8 @@ def matmul(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out: 
     consumer to add up in order (the next norm does), instead of being added
     inside a thread-block cluster, whose launch and barriers cost more.
     ``status``: the status word for the kernels with bounded waits.  ``upcoming``: what the step
-    streams after this product; a decode product asks L2 for its first ``UPCOMING_BYTES``."""
+    streams after this product; a decode product asks L2 for its first ``UPCOMING_BYTES``.  ``tail`` (row, out2, col): see
+    ``kernels.gemv``; given only where ``takes_tail`` says so."""
     if x.dtype == torch.float32:
         K.gemm_simt(x, w, bias, out)
         return out
@@ -78,10 +88,10 @@ def matmul(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out: 
             return view
         if splits >= 1:
             K.gemv(x, w, bias, out, K.GEMV_F32 if out.dtype == torch.float32 else K.GEMV_BF16, splits,
-                   prefetch=upcoming, prefetch_bytes=UPCOMING_BYTES)
+                   prefetch=upcoming, prefetch_bytes=UPCOMING_BYTES, tail=tail)
             return out
     if stream_gemm(M, w.shape[0], Kd):
-        K.gemm_stream(x, w, bias, out, status=status)
+        K.gemm_stream(x, w, bias, out, status=status, tail=tail)
         return out
     if PROMPT_GEMM == "tcgen05" and K.gemm_tc_supported(M, w.shape[0], Kd):
         K.gemm_tc(x, w, bias, out)

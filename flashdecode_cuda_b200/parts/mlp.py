@@ -190,6 +190,10 @@ class DenseActMLP(FeedForward):
     def shares_products(self) -> bool:
         return self.activation == "relu2"
 
+    @property
+    def epilogue_act(self) -> str:
+        return self.activation
+
     def kv_request(self):
         return None
 

@@ -11,7 +11,7 @@ from ..cache.paged import StateSpec
 from ..registry import register_part
 from ..weights.spec import TensorSpec
 from .base import KVRequest, LayerCache, Mixer, Runtime
-from .linear import matmul
+from .linear import matmul, takes_tail
 
 
 @register_part("mixer", "parallel")
@@ -24,7 +24,7 @@ class ParallelMixers(Mixer):
     output product over the branches' activations laid side by side with the stacked output matrices:
     sum_b scale_b W_b a_b = [W_1 | W_2 | ...] [scale_1 a_1 ; scale_2 a_2 ; ...].  The scale enters each branch's
     activations in float32 before their one rounding.  A feed-forward that reads the same input as the mixers is one more
-    such branch.  A branch's activations start at a multiple of 8 columns, and the row's length is a multiple of 32 (columns
+    such branch; as the last one, its activation is taken in the input product's epilogue in steps of up to 128 tokens.  A branch's activations start at a multiple of 8 columns, and the row's length is a multiple of 32 (columns
     of zeros fill up).  Other branches run whole, and the weighted sum of the outputs is taken in float32.  At most one branch may keep keys; every branch's per-sequence state is kept under
     ``<name>.<its own name>``."""
 
@@ -63,6 +63,14 @@ class ParallelMixers(Mixer):
         if not self.fused:
             return
         ins = [b.in_proj() for b in self.branches]
+        # a feed-forward whose activation the product's epilogue can take comes last, its rows at a multiple of 16
+        self.tail = len(ins) - 1 if getattr(self.branches[-1], "epilogue_act", None) == "relu2" and self.scales[-1] == 1.0 else None
+        if self.tail is not None and rt.dtype == torch.bfloat16 and len(ins) > 1:
+            fill = -sum(w.shape[0] for w, _ in ins[:-1]) % 16
+            w, bias = ins[-2]
+            if fill:
+                ins[-2] = (torch.cat([w, w.new_zeros((fill, w.shape[1]))], dim=0),
+                           None if bias is None else torch.cat([bias, bias.new_zeros(fill)]))
         self.w_in = torch.cat([w for w, _ in ins], dim=0).contiguous()
         self.b_in = None
         if any(bias is not None for _, bias in ins):
@@ -112,12 +120,16 @@ class ParallelMixers(Mixer):
     def forward(self, ctx, x: torch.Tensor, lc: LayerCache) -> torch.Tensor:
         T, ws, rt = ctx.T, ctx.ws, self.rt
         if self.fused:
-            proj = ws.get("par_proj", (T, self.w_in.shape[0]), x.dtype)
-            matmul(x, self.w_in, self.b_in, proj, status=rt.status)
+            N, Kd = self.w_in.shape
+            proj = ws.get("par_proj", (T, N), x.dtype)
             act = ws.get("par_act", (T, self.n_act), x.dtype)
+            tail, branches = None, list(enumerate(self.branches))
+            if self.tail is not None and takes_tail(T, N, Kd, x.dtype, self.in_cols[-1], self.n_act, self.act_cols[-1]):
+                tail, branches = (self.in_cols[-1], act, self.act_cols[-1]), branches[:-1]
+            matmul(x, self.w_in, self.b_in, proj, status=rt.status, tail=tail)
             for lo, hi in self.gaps:
                 act[:, lo:hi].zero_()
-            for i, b in enumerate(self.branches):
+            for i, b in branches:
                 b.inner(ctx, proj, self.in_cols[i], self._sub(lc, i), act, self.act_cols[i], self.scales[i])
             out = ws.get("mixer_out", (T, self.hidden_size), x.dtype)
             return matmul(act, self.w_o, None, out, target_ctas=4 * rt.sm_count, status=rt.status, upcoming=ctx.upcoming)

@@ -467,6 +467,31 @@ def test_relu_squared_between_columns(dtype, T, C, xc, oc):
     assert bool((out[:, :oc] == 0).all()) and bool((out[:, oc + C:] == 0).all())
 
 
+@pytest.mark.parametrize("M", [1, 3, 8, 16, 17, 40, 128])
+@pytest.mark.parametrize("N,row,Kd", [(1168, 144, 256), (400, 16, 2048), (4096, 2048, 512)])
+@pytest.mark.parametrize("biased", [False, True])
+def test_products_whose_last_rows_are_a_feed_forwards(M, N, row, Kd, biased):
+    """The streaming products' epilogue: rows from ``row`` on leave max(., 0)^2 in another buffer's columns, the others are as
+    they are without it, and nothing else of either buffer changes."""
+    from flashdecode_cuda_b200.parts.linear import matmul, takes_tail
+    torch.manual_seed(M + N)
+    x, w = torch.randn(M, Kd).bfloat16(), (torch.randn(N, Kd) / Kd ** 0.5).bfloat16()
+    b = torch.randn(N).bfloat16() if biased else None
+    col, ld = 8, 8 + N - row + 24
+    assert takes_tail(M, N, Kd, torch.bfloat16, row, ld, col)
+    out, out2 = torch.full((M, N), 7.0, dtype=torch.bfloat16, device=DEV), torch.full((M, ld), 7.0, dtype=torch.bfloat16, device=DEV)
+    plain = torch.zeros_like(out)
+    status = new_status()
+    bd = b.to(DEV) if biased else None
+    matmul(x.to(DEV), w.to(DEV), bd, plain, status=status)
+    matmul(x.to(DEV), w.to(DEV), bd, out, status=status, tail=(row, out2, col))
+    assert int(status) == 0
+    assert torch.equal(out[:, :row], plain[:, :row]) and bool((out[:, row:] == 7).all())
+    want = P.relu_squared((x.double() @ w.double().t() + (b.double() if biased else 0))[:, row:])
+    assert rel_err(out2[:, col:col + N - row], want) < 1e-2
+    assert bool((out2[:, :col] == 7).all()) and bool((out2[:, col + N - row:] == 7).all())
+
+
 # ---------------------------------------------------------------- whole models
 @pytest.fixture(scope="module")
 def folders(tmp_path_factory):
