@@ -130,6 +130,7 @@ class GatedDeltaRule(Mixer):
         step = (q, k, v, g, beta, lc.states["state"], o, ctx.row_slot, ctx.row_q_start, ctx.row_q_len, ctx.n_rows, lc.writes)
         long = ctx.max_q_len > K.delta_scan_single()
         if long and proj.dtype == torch.bfloat16 and K.delta_chunks_takes(d):
+            # (the rows' lengths on the host: a step with a long row is never replayed from a graph)
             if min(ctx.h_q_len, default=0) <= K.delta_scan_single():
                 K.delta_scan(*step, short_only=True)
             n = K.delta_chunks_scratch_bytes(T, ctx.n_rows, H, d)
