@@ -1,6 +1,6 @@
 // The gated delta rule with a decay per head and key channel, for prompts and decode steps:
 //
-//   S <- diag(g_t) S;  u_t = beta_t (v_t - S^T k_t);  S <- S + k_t u_t^T;  o_t = S^T q_t        S [d, dv] per sequence and head
+//   F_t = diag(g_t) S_(t-1);  S_t = F_t + k_t u_t^T, u_t = beta_t (v_t - F_t^T k_t);  o_t = S_t^T q_t    S [d, dv] per sequence and head
 //
 //  * delta_prepare: everything that enters the recurrence, as floats.  q, k and v pass a short causal convolution over time
 //    per channel (short_conv.cuh) and silu; every head of q and k becomes a unit vector, x / sqrt(sum x^2 + 1e-6), and q is

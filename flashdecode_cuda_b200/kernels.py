@@ -1102,7 +1102,7 @@ def delta_prepare(proj: torch.Tensor, cols, conv_w: torch.Tensor, ring: Optional
 def delta_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, g: torch.Tensor, beta: torch.Tensor, state: torch.Tensor,
                out: torch.Tensor, row_slot: torch.Tensor, row_q_start: torch.Tensor, row_q_len: torch.Tensor, n_rows: int,
                write_state: bool, max_q_len: int = 0, scratch: Optional[torch.Tensor] = None, short_only: bool = False) -> None:
-    """S <- diag(exp(g)) S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q, per sequence and head over the step's tokens, from
+    """S_t = F + k_t (beta_t (v_t - F^T k_t))^T with F = diag(exp(g_t)) S_(t-1), o_t = S_t^T q_t, per sequence and head, from
     ``state`` [slots, heads, d, dv] (float32, updated when ``write_state``) to ``out`` [T, heads * dv] float32.  The inputs are
     those ``delta_prepare`` leaves.  With ``scratch`` (float32, ``delta_scan_scratch_floats`` elements) and ``max_q_len`` (the longest
     row), rows of more than ``delta_scan_single()`` tokens are walked four tokens at a time; with ``short_only`` they are left out

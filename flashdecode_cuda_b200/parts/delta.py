@@ -25,7 +25,8 @@ class GatedDeltaRule(Mixer):
         q, k    = x / sqrt(sum x^2 + 1e-6) per head;  q times head_dim^(-1/2)
         beta    = sigmoid(W_b h)                                              per head
         g       = exp(-exp(A_h) softplus(W_a2 (W_a1 h) + b))                  per head and key channel
-        S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q    S [head_dim, v_head_dim] per head
+        F_t     = diag(g_t) S_(t-1)                                           what the state keeps, [head_dim, v_head_dim] per head
+        S_t     = F_t + k_t (beta_t (v_t - F_t^T k_t))^T;   o_t = S_t^T q_t
         out     = W_o ( concat_h o / rms(o) * w * sigmoid(W_g2 (W_g1 h)) )    rms per head over v_head_dim, w [v_head_dim]
 
     The state starts at zero and is carried in float32 per cache slot, and so are the last projected values (a ring of ``taps``

@@ -14,8 +14,8 @@ Three kinds of mixer:
   softmax attention with biased projections, q and k RMS-normed over the whole
   projection and then rotated (pairs i, i + dims/2).  The right one is the gated
   delta rule with a decay per key channel: q, k, v convolved and passed through
-  silu, q and k made unit vectors, S <- diag(g) S, u = beta (v - S^T k),
-  S <- S + k u^T, o = S^T q; each head's o RMS-normed, weighted, gated by a sigmoid.
+  silu, q and k made unit vectors, S_t = F + beta k (v - F^T k)^T with
+  F = diag(g) S_(t-1), o = S_t^T q; each head's o RMS-normed, weighted, gated by a sigmoid.
 * ``attention``: grouped-head softmax attention, rotation first, then an RMS norm
   per head without a weight, tanh-capped scores, a sliding window, one extra
   learned term per head in the softmax denominator, and values mixed with those of
@@ -101,8 +101,8 @@ def gated_part_norm(y: torch.Tensor, z: torch.Tensor, w: torch.Tensor, parts: in
 
 
 def delta_recurrence(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, g: torch.Tensor, beta: torch.Tensor) -> torch.Tensor:
-    """q, k [S, G, d], v [S, H, dv], g [S, H, d], beta [S, H]: S <- diag(g) S; u = beta (v - S^T k); S <- S + k u^T;
-    o = S^T q; head h reads q/k head h // (H / G)."""
+    """q, k [S, G, d], v [S, H, dv], g [S, H, d], beta [S, H]: F = diag(g_t) S_(t-1);
+    S_t = F + beta_t k_t (v_t - F^T k_t)^T; o_t = S_t^T q_t; head h reads q/k head h // (H / G)."""
     S, H, dv = v.shape
     rep = H // q.shape[1]
     q, k = q.repeat_interleave(rep, dim=1), k.repeat_interleave(rep, dim=1)
